@@ -139,9 +139,11 @@ def allocate_cache(
     device: str | torch.device = "cuda",
     max_step_tokens: int | None = None,
     embedding_state: StateSpec | None = None,
+    block_states: list[StateSpec | None] | None = None,
 ) -> CacheLayout:
     """``max_step_tokens`` (the token budget of a step) bounds what a group with a window can
-    hold; without it such a group is sized like one that keeps every key."""
+    hold; without it such a group is sized like one that keeps every key.  ``block_states``: per
+    execution entry the state that the layer's block keeps beside its mixer's."""
     specs, group_of = plan_groups(needs)
     pages = [
         pages_of_group(s, num_blocks, block_size, max_num_seqs, max_step_tokens) if max_step_tokens else num_blocks
@@ -182,6 +184,10 @@ def allocate_cache(
         if state is not None:
             slot_groups.append(SlotGroupSpec(f"state{entry}:{'x'.join(map(str, state.shape))}"))
             view.state = torch.zeros((max_num_seqs + 1, *state.shape), dtype=state.dtype, device=device)
+        block_state = block_states[entry] if block_states is not None else None
+        if block_state is not None:
+            slot_groups.append(SlotGroupSpec(f"block{entry}:{'x'.join(map(str, block_state.shape))}"))
+            view.block_state = torch.zeros((max_num_seqs + 1, *block_state.shape), dtype=block_state.dtype, device=device)
         views.append(view)
     per_token = sum(len(e) * s.kv_heads * (s.head_dim + s.v_dim) * element for s, e in zip(specs, owners))
     first_state = None

@@ -14,6 +14,7 @@ from mini_engine_b200.config.registry import (
     register_architecture,
     registered_architectures,
 )
+from mini_engine_b200.config.tobadra import TobadraConfig
 
 __all__ = [
     "Architecture",
@@ -27,6 +28,7 @@ __all__ = [
     "MolotarConfig",
     "PimezenConfig",
     "Qwen3Config",
+    "TobadraConfig",
     "architecture_for",
     "load_model_config",
     "register_architecture",

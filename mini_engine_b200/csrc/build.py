@@ -38,6 +38,8 @@ LIBRARIES = {
     "latent_attention_tcgen05": "latent_attention_tcgen05.cu",
     "linear_attention": "linear_attention.cu",
     "hyper_connections": "hyper_connections.cu",
+    "sandwich": "sandwich.cu",
+    "delta_rule": "delta_rule.cu",
     "recurrent": "recurrent.cu",
     "routing": "routing.cu",
     "gemm_tcgen05": "gemm_tcgen05.cu",

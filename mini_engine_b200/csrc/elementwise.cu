@@ -830,6 +830,29 @@ ME_EXPORT int me_rope_table(const float* inv_freq, const int* positions, float* 
                          reinterpret_cast<float2*>(out), tokens, half);
 }
 
+// The same with the angle formed, and reduced to one turn, in double precision.
+__global__ void rope_table_double_kernel(const double* __restrict__ inv_freq, const int* __restrict__ positions,
+                                         float2* __restrict__ out, int tokens, int half) {
+    pdl_trigger();
+    pdl_wait();
+    const int idx = blockIdx.x * blockDim.x + threadIdx.x;
+    if (idx >= tokens * half) return;
+    const int token = idx / half, i = idx % half;
+    constexpr double TURN = 6.283185307179586476925;
+    const double angle = static_cast<double>(positions[token]) * inv_freq[i];
+    float sine, cosine;
+    sincosf(static_cast<float>(angle - TURN * rint(angle / TURN)), &sine, &cosine);
+    out[idx] = make_float2(cosine, sine);
+}
+
+ME_EXPORT int me_rope_table_double(const double* inv_freq, const int* positions, float* out, int tokens, int half,
+                                   cudaStream_t stream) {
+    if (tokens <= 0) return 0;
+    const int total = tokens * half;
+    return launch_kernel(rope_table_double_kernel, (total + 255) / 256, 256, 0, stream, inv_freq, positions,
+                         reinterpret_cast<float2*>(out), tokens, half);
+}
+
 ME_EXPORT int me_qk_norm_rope_store(const float* qkv, int splits, long long split_stride, const float* q_weight,
                                     const float* k_weight, float eps, const float* cos_sin,
                                     const int* positions, const int* slot_mapping, void* q_out, void* k_pages,
@@ -1232,60 +1255,67 @@ ME_EXPORT int me_qk_wide_norm_rope_store(const float* qkv, int splits, long long
 // ------------------------------------------------------ an activation on a product's partial sums
 
 // out[t][i] = act(sum_s partial[s][t][i]) in the compute dtype, for a feed-forward without a gate.
-// 0: relu(z)^2, 1: z * sigmoid(z), 2: the tanh form of GELU, 3: relu(z).
-enum : int { ACT_RELU_SQUARED = 0, ACT_SILU = 1, ACT_GELU_TANH = 2, ACT_RELU = 3 };
+// 0: relu(z)^2, 1: z * sigmoid(z), 2: the tanh form of GELU, 3: relu(z), 4: GELU, 0.5 z (1 + erf(z / sqrt 2)).  With
+// `group_weight [tokens][groups]` the features form `groups` equal runs (routed units side by side) and feature i of
+// token t is multiplied by group_weight[t][i / group_size].
+enum : int { ACT_RELU_SQUARED = 0, ACT_SILU = 1, ACT_GELU_TANH = 2, ACT_RELU = 3, ACT_GELU_ERF = 4 };
 
 __device__ __forceinline__ float plain_activation(float z, int activation) {
     if (activation == ACT_RELU_SQUARED) { const float r = fmaxf(z, 0.0f); return r * r; }
     if (activation == ACT_SILU) return z / (1.0f + expf(-z));
     if (activation == ACT_GELU_TANH) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    if (activation == ACT_GELU_ERF) return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));
     return fmaxf(z, 0.0f);
 }
 
 template <typename OutT, int V>  // V consecutive elements per thread: 4 (16-byte loads) or 1
 __global__ void activation_kernel(const float* __restrict__ partial, int splits, size_t split_stride,
-                                  OutT* __restrict__ out, size_t total, int activation) {
+                                  OutT* __restrict__ out, size_t total, int activation, const float* __restrict__ group_weight,
+                                  int width, int group_size) {
     pdl_trigger();
     pdl_wait();
     for (size_t idx = (blockIdx.x * static_cast<size_t>(blockDim.x) + threadIdx.x) * V; idx < total;
          idx += static_cast<size_t>(gridDim.x) * blockDim.x * V) {
+        float weight = 1.0f;
+        if (group_weight != nullptr) weight = group_weight[idx / width * (width / group_size) + idx % width / group_size];
         if constexpr (V == 4) {
             float4 z = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
             for (int s = 0; s < splits; ++s) add4(z, *reinterpret_cast<const float4*>(partial + s * split_stride + idx));
-            store4(out + idx, make_float4(plain_activation(z.x, activation), plain_activation(z.y, activation),
-                                          plain_activation(z.z, activation), plain_activation(z.w, activation)));
+            store4(out + idx, make_float4(weight * plain_activation(z.x, activation), weight * plain_activation(z.y, activation),
+                                          weight * plain_activation(z.z, activation), weight * plain_activation(z.w, activation)));
         } else {
             float z = 0.0f;
             for (int s = 0; s < splits; ++s) z += partial[s * split_stride + idx];
-            out[idx] = from_float<OutT>(plain_activation(z, activation));
+            out[idx] = from_float<OutT>(weight * plain_activation(z, activation));
         }
     }
 }
 
 ME_EXPORT int me_activation(const float* partial, int splits, long long split_stride, void* out, int out_type,
-                            int tokens, int width, int activation, cudaStream_t stream) {
+                            int tokens, int width, int activation, const float* group_weight, int group_size, cudaStream_t stream) {
     if (tokens <= 0) return 0;
-    if (activation < ACT_RELU_SQUARED || activation > ACT_RELU) return ME_ERR_ARGUMENT;
+    if (activation < ACT_RELU_SQUARED || activation > ACT_GELU_ERF) return ME_ERR_ARGUMENT;
+    if (group_weight != nullptr && (group_size < 1 || width % group_size)) return ME_ERR_ARGUMENT;
     const size_t total = static_cast<size_t>(tokens) * width;
-    const bool vec = width % 4 == 0 && split_stride % 4 == 0 && aligned16(partial) && aligned16(out);
+    const bool vec = width % 4 == 0 && split_stride % 4 == 0 && aligned16(partial) && aligned16(out) && (group_weight == nullptr || group_size % 4 == 0);
     const int threads = 256;
     const int blocks = static_cast<int>(std::min<size_t>((total / (vec ? 4 : 1) + threads - 1) / threads, 148 * 32));
     const size_t stride = static_cast<size_t>(split_stride);
     if (out_type == ME_BF16) {
         auto* o = static_cast<__nv_bfloat16*>(out);
-        return vec ? launch_kernel(activation_kernel<__nv_bfloat16, 4>, blocks, threads, 0, stream, partial, splits, stride, o, total, activation)
-                   : launch_kernel(activation_kernel<__nv_bfloat16, 1>, blocks, threads, 0, stream, partial, splits, stride, o, total, activation);
+        return vec ? launch_kernel(activation_kernel<__nv_bfloat16, 4>, blocks, threads, 0, stream, partial, splits, stride, o, total, activation, group_weight, width, group_size)
+                   : launch_kernel(activation_kernel<__nv_bfloat16, 1>, blocks, threads, 0, stream, partial, splits, stride, o, total, activation, group_weight, width, group_size);
     }
     auto* o = static_cast<float*>(out);
-    return vec ? launch_kernel(activation_kernel<float, 4>, blocks, threads, 0, stream, partial, splits, stride, o, total, activation)
-               : launch_kernel(activation_kernel<float, 1>, blocks, threads, 0, stream, partial, splits, stride, o, total, activation);
+    return vec ? launch_kernel(activation_kernel<float, 4>, blocks, threads, 0, stream, partial, splits, stride, o, total, activation, group_weight, width, group_size)
+               : launch_kernel(activation_kernel<float, 1>, blocks, threads, 0, stream, partial, splits, stride, o, total, activation, group_weight, width, group_size);
 }
 
 // --------------------------------------- bias + rotary + unit norm behind the rotation + cache write
 
 // One warp per (token, head) over the columns of qkv = [q heads | k heads | v heads]: the partial sums and the
 // bias are added, the first rotary_dim elements of a q or k head are rotated (element e pairs with e +
-// rotary_dim / 2), and then, with `unit_norm`, the rotated head is divided by its root mean square over head_dim
+// rotary_dim / 2; a value head is rotated too, over its whole width, when it has a table of its own), and then, with `unit_norm`, the rotated head is divided by its root mean square over head_dim
 // (eps inside the root, no weight).  q goes to q_out, k and v to the token's cache slot (or to dense buffers).
 // Lane l holds elements l, l + 32, ... and adds their squares in ascending order; the lanes meet in a butterfly.
 struct UnitQkvArgs {
@@ -1303,6 +1333,7 @@ struct UnitQkvArgs {
     void* v_dense;
     float eps;
     int tokens, heads, kv_heads, head_dim, value_dim, page_size, rotary_dim, unit_norm;
+    const float2* value_cos_sin;  // [tokens][value_dim / 2]: a rotation over the whole value head, or null
 };
 
 constexpr int UNIT_WARPS = 4;
@@ -1334,14 +1365,16 @@ __global__ void __launch_bounds__(UNIT_WARPS * 32) qkv_rope_unit_store_kernel(Un
     __syncwarp();
     float value[UNIT_MAX_PER_LANE];
     float sum_sq = 0.0f;
-    const int half = a.rotary_dim / 2;
-    const float2* angles = (a.cos_sin && (is_q || is_k)) ? a.cos_sin + static_cast<size_t>(token) * half : nullptr;
+    const int rotary_dim = (is_q || is_k) ? a.rotary_dim : a.value_dim;
+    const int half = rotary_dim / 2;
+    const float2* table = (is_q || is_k) ? a.cos_sin : a.value_cos_sin;
+    const float2* angles = table ? table + static_cast<size_t>(token) * half : nullptr;
 #pragma unroll
     for (int j = 0; j < UNIT_MAX_PER_LANE; ++j) {
         const int e = lane + 32 * j;
         if (e >= d) break;
         float v = mine[e];
-        if (angles && e < a.rotary_dim) {
+        if (angles && e < rotary_dim) {
             const float other = mine[e < half ? e + half : e - half];
             const float2 angle = angles[e < half ? e : e - half];
             v = e < half ? v * angle.x - other * angle.y : v * angle.x + other * angle.y;
@@ -1374,7 +1407,7 @@ ME_EXPORT int me_qkv_rope_unit_store(const float* qkv, int splits, long long spl
                                      const float* bias, const float* cos_sin, const int* slot_mapping, void* q_out,
                                      void* k_pages, void* v_pages, void* k_dense, void* v_dense, float eps, int out_type,
                                      int tokens, int heads, int kv_heads, int head_dim, int value_dim, int page_size,
-                                     int rotary_dim, int unit_norm, cudaStream_t stream) {
+                                     int rotary_dim, int unit_norm, const float* value_cos_sin, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (rotary_dim < 0 || rotary_dim > head_dim || rotary_dim % 2) return ME_ERR_ARGUMENT;
     if (row_width < (heads + kv_heads) * head_dim + kv_heads * value_dim) return ME_ERR_ARGUMENT;
@@ -1382,10 +1415,69 @@ ME_EXPORT int me_qkv_rope_unit_store(const float* qkv, int splits, long long spl
         return ME_ERR_UNSUPPORTED;
     UnitQkvArgs a{qkv, splits, (size_t)split_stride, row_width, bias, reinterpret_cast<const float2*>(cos_sin), slot_mapping,
                   q_out, k_pages, v_pages, k_dense, v_dense, eps, tokens, heads, kv_heads, head_dim, value_dim, page_size,
-                  rotary_dim, unit_norm};
+                  rotary_dim, unit_norm, reinterpret_cast<const float2*>(value_cos_sin)};
+    if (value_cos_sin != nullptr && value_dim % 2) return ME_ERR_ARGUMENT;
     const long long items = static_cast<long long>(tokens) * (heads + 2 * kv_heads);
     const int blocks = static_cast<int>((items + UNIT_WARPS - 1) / UNIT_WARPS);
     const size_t smem = static_cast<size_t>(UNIT_WARPS) * std::max(head_dim, value_dim) * sizeof(float);
     if (out_type == ME_BF16) return launch_kernel(qkv_rope_unit_store_kernel<__nv_bfloat16>, blocks, UNIT_WARPS * 32, smem, stream, a);
     return launch_kernel(qkv_rope_unit_store_kernel<float>, blocks, UNIT_WARPS * 32, smem, stream, a);
+}
+
+// ------------------------------------------------------------- attention outputs, turned back
+
+// In place on x [tokens][heads][dim]: the rotation of a whole head by the negative of the token's angles (pairs (m, m + dim /
+// 2)): (u, v) becomes (u cos a + v sin a, v cos a - u sin a).  V pairs per thread.
+template <typename T, int V>
+__global__ void __launch_bounds__(256) turn_heads_back_kernel(T* __restrict__ x, const float2* __restrict__ cos_sin, size_t total, int heads, int dim) {
+    pdl_trigger();
+    pdl_wait();
+    const int half = dim / 2;
+    for (size_t idx = (blockIdx.x * static_cast<size_t>(256) + threadIdx.x) * V; idx < total; idx += static_cast<size_t>(gridDim.x) * 256 * V) {
+        const size_t row = idx / half;  // (token, head)
+        const int m = static_cast<int>(idx % half);
+        T* u_at = x + row * dim + m;
+        const float2* angles = cos_sin + row / heads * half + m;
+        if constexpr (V == 4) {
+            float u[4], v[4];
+            if constexpr (sizeof(T) == 2) {
+                const uint2 raw_u = *reinterpret_cast<const uint2*>(u_at), raw_v = *reinterpret_cast<const uint2*>(u_at + half);
+                const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw_u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw_u.y));
+                const float2 c = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw_v.x)), d = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw_v.y));
+                u[0] = a.x, u[1] = a.y, u[2] = b.x, u[3] = b.y, v[0] = c.x, v[1] = c.y, v[2] = d.x, v[3] = d.y;
+            } else {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) u[i] = to_float(u_at[i]), v[i] = to_float(u_at[half + i]);
+            }
+            const float4 first = *reinterpret_cast<const float4*>(angles), second = *reinterpret_cast<const float4*>(angles + 2);
+            const float cosine[4] = {first.x, first.z, second.x, second.z}, sine[4] = {first.y, first.w, second.y, second.w};
+            float nu[4], nv[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) nu[i] = u[i] * cosine[i] + v[i] * sine[i], nv[i] = v[i] * cosine[i] - u[i] * sine[i];
+            store4(u_at, make_float4(nu[0], nu[1], nu[2], nu[3]));
+            store4(u_at + half, make_float4(nv[0], nv[1], nv[2], nv[3]));
+        } else {
+            const float u = to_float(u_at[0]), v = to_float(u_at[half]);
+            const float2 angle = angles[0];
+            u_at[0] = from_float<T>(u * angle.x + v * angle.y);
+            u_at[half] = from_float<T>(v * angle.x - u * angle.y);
+        }
+    }
+}
+
+ME_EXPORT int me_turn_heads_back(void* x, int type, const float* cos_sin, int tokens, int heads, int dim, cudaStream_t stream) {
+    if (tokens <= 0 || heads <= 0) return 0;
+    if (dim < 2 || dim % 2) return ME_ERR_ARGUMENT;
+    const bool vec = dim % 8 == 0 && aligned16(x) && aligned16(cos_sin);
+    const size_t total = static_cast<size_t>(tokens) * heads * (dim / 2);
+    const int blocks = static_cast<int>(std::min<size_t>((total / (vec ? 4 : 1) + 255) / 256, 148 * 32));
+    const auto* angles = reinterpret_cast<const float2*>(cos_sin);
+    if (type == ME_BF16) {
+        auto* p = static_cast<__nv_bfloat16*>(x);
+        return vec ? launch_kernel(turn_heads_back_kernel<__nv_bfloat16, 4>, blocks, 256, 0, stream, p, angles, total, heads, dim)
+                   : launch_kernel(turn_heads_back_kernel<__nv_bfloat16, 1>, blocks, 256, 0, stream, p, angles, total, heads, dim);
+    }
+    auto* p = static_cast<float*>(x);
+    return vec ? launch_kernel(turn_heads_back_kernel<float, 4>, blocks, 256, 0, stream, p, angles, total, heads, dim)
+               : launch_kernel(turn_heads_back_kernel<float, 1>, blocks, 256, 0, stream, p, angles, total, heads, dim);
 }

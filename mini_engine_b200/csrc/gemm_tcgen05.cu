@@ -73,6 +73,8 @@ struct GemmParams {
     // The gated epilogue: g * sigmoid(slope * g) * (u + offset) with g = min(gate, limit), u = clamp(up, +-limit)
     // when limit > 0.  The defaults are SwiGLU.
     float act_slope = 1.0f, act_limit = 0.0f, act_offset = 0.0f;
+    // A product without a gate: what its sums pass before they are stored, as bfloat16 (PLAIN_*); negative: nothing, float32.
+    int plain_act = -1;
     int act_gelu = 0;  // 1: the gate is the tanh form of GELU, g * sigmoid(2 sqrt(2 / pi) (g + 0.044715 g^3))
 };
 
@@ -82,6 +84,23 @@ struct GemmParams {
 __device__ __forceinline__ float gate_activation(float g, float slope, int gelu) {
     const float inside = gelu ? 1.5957691216057308f * g * fmaf(0.044715f * g, g, 1.0f) : slope * g;
     return __fdividef(g, 1.0f + __expf(-inside));
+}
+
+// Activations of a product without a gate, numbered as in elementwise.cu: relu(z)^2, z sigmoid(z), the tanh form of GELU,
+// relu(z), GELU.
+enum : int { PLAIN_RELU_SQUARED = 0, PLAIN_SILU = 1, PLAIN_GELU_TANH = 2, PLAIN_RELU = 3, PLAIN_GELU_ERF = 4 };
+
+__device__ __forceinline__ float plain_activation(float z, int act) {
+    if (act == PLAIN_GELU_ERF) return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));
+    if (act == PLAIN_GELU_TANH || act == PLAIN_SILU) return gate_activation(z, 1.0f, act == PLAIN_GELU_TANH);
+    const float r = fmaxf(z, 0.0f);
+    return act == PLAIN_RELU_SQUARED ? r * r : r;
+}
+
+// One sum of a product without a gate at element `at` of the output.
+__device__ __forceinline__ void store_sum(const GemmParams& p, size_t at, float v) {
+    if (p.plain_act >= 0) static_cast<__nv_bfloat16*>(p.out)[at] = __float2bfloat16_rn(plain_activation(v, p.plain_act));
+    else static_cast<float*>(p.out)[at] = v;
 }
 
 template <int BLOCK_T, bool DUAL>
@@ -198,7 +217,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
         if (ok && iterations > 0) {
             const uint32_t lane_base = tmem_base + (static_cast<uint32_t>(quarter * 32) << 16);
             if (!DUAL) {
-                float* out = static_cast<float*>(p.out) + static_cast<size_t>(split) * p.tokens * p.outs;
+                const size_t base = static_cast<size_t>(split) * p.tokens * p.outs;  // an activation comes with one split only
 #pragma unroll 1
                 for (int c0 = 0; c0 < BLOCK_T; c0 += 16) {
                     if (t0 + c0 >= p.tokens) break;  // uniform: the rest of the tile is padding
@@ -208,7 +227,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
 #pragma unroll
                         for (int c = 0; c < 16; ++c) {
                             const int t = t0 + c0 + c;
-                            if (t < p.tokens) out[static_cast<size_t>(t) * p.outs + n] = v[c];
+                            if (t < p.tokens) store_sum(p, base + static_cast<size_t>(t) * p.outs + n, v[c]);
                         }
                     }
                 }
@@ -574,10 +593,10 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid
                     float v[16];
                     tcgen05_ld16(lane_base + c0, v);
                     if (n < p.outs) {
-                        float* out = static_cast<float*>(p.out) + static_cast<size_t>(split) * p.tokens * p.outs;
+                        const size_t base = static_cast<size_t>(split) * p.tokens * p.outs;
 #pragma unroll
                         for (int c = 0; c < 16; ++c)
-                            if (t0 + c0 + c < p.tokens) out[static_cast<size_t>(t0 + c0 + c) * p.outs + n] = v[c];
+                            if (t0 + c0 + c < p.tokens) store_sum(p, base + static_cast<size_t>(t0 + c0 + c) * p.outs + n, v[c]);
                     }
                 } else {
                     float gate[16], up[16];
@@ -784,10 +803,9 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const 
                     float v[16];
                     tcgen05_ld16(lane_base + c0, v);
                     if (n < p.outs) {
-                        float* out = static_cast<float*>(p.out);
 #pragma unroll
                         for (int c = 0; c < 16; ++c)
-                            if (t0 + c0 + c < p.tokens) out[static_cast<size_t>(t0 + c0 + c) * p.outs + n] = v[c];
+                            if (t0 + c0 + c < p.tokens) store_sum(p, static_cast<size_t>(t0 + c0 + c) * p.outs + n, v[c]);
                     }
                 } else {
                     float gate[16], up[16];
@@ -887,11 +905,12 @@ ME_EXPORT int me_gemm_tcgen05(const void* map_w, const void* map_x, float* out, 
 
 // Grouped product over rows that are sorted by group (see GemmParams): out[t][n] = x[t] . w[group(t) * group_rows + n]
 // for n < outs, float32 [rows][outs]; or, with dual_row_offset > 0, the gated unit of rows n and dual_row_offset + n
-// of the row's group, bfloat16 [rows][outs].  `group_pad` must be a multiple of the token tile (128).
+// of the row's group, bfloat16 [rows][outs]; or, with plain_act >= 0, the activation of the sums, bfloat16 [rows][outs].  `group_pad` must be a multiple of the token tile (128).
 ME_EXPORT int me_gemm_tcgen05_grouped(const void* map_w, const void* map_x, void* out, int rows, int outs, int inner,
                                       const int* group_of_block, int group_pad, int group_rows, int dual_row_offset,
-                                      float slope, float limit, float offset, cudaStream_t stream) {
+                                      float slope, float limit, float offset, int plain_act, cudaStream_t stream) {
     if (rows <= 0 || outs <= 0) return 0;
+    if (plain_act > PLAIN_GELU_ERF || (plain_act >= 0 && dual_row_offset > 0)) return ME_ERR_ARGUMENT;
     if (group_of_block == nullptr || group_pad < 128 || group_pad % 128 || rows % group_pad || group_rows < outs)
         return ME_ERR_ARGUMENT;
     alignas(64) CUtensorMap w, x;
@@ -903,6 +922,7 @@ ME_EXPORT int me_gemm_tcgen05_grouped(const void* map_w, const void* map_x, void
     p.group_pad = group_pad;
     p.group_rows = group_rows;
     p.act_slope = slope, p.act_limit = limit, p.act_offset = offset;
+    p.plain_act = plain_act;
     return dual_row_offset > 0 ? launch<128, true>(w, x, p, 1, stream) : launch<128, false>(w, x, p, 1, stream);
 }
 
@@ -1001,15 +1021,17 @@ static int launch_persistent(const CUtensorMap& map_w, const CUtensorMap& map_x,
     return static_cast<int>(cudaLaunchKernelEx(&config, kernel, map_w, map_x, q));
 }
 
-// out[t][n] (float32) = x[t] . w[n] by persistent CTA pairs.  Weight and activation maps have
-// boxes of 128 rows.
-ME_EXPORT int me_gemm_tcgen05_persistent(const void* map_w, const void* map_x, float* out, int tokens, int outs,
-                                         int inner, int group, cudaStream_t stream) {
+// out[t][n] (float32) = x[t] . w[n] by persistent CTA pairs; with plain_act >= 0 the activation of the sums, bfloat16.
+// Weight and activation maps have boxes of 128 rows.
+ME_EXPORT int me_gemm_tcgen05_persistent(const void* map_w, const void* map_x, void* out, int tokens, int outs,
+                                         int inner, int group, int plain_act, cudaStream_t stream) {
     if (tokens <= 0 || outs <= 0) return 0;
+    if (plain_act > PLAIN_GELU_ERF) return ME_ERR_ARGUMENT;
     alignas(64) CUtensorMap w, x;
     memcpy(&w, map_w, sizeof(w));
     memcpy(&x, map_x, sizeof(x));
     GemmParams p{out, tokens, outs, (inner + BLOCK_K - 1) / BLOCK_K, 0, 0, 0, 0, 1, 0, 0, 0};
+    p.plain_act = plain_act;
     return launch_persistent<false>(w, x, p, group, stream);
 }
 

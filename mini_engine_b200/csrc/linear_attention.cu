@@ -15,7 +15,8 @@
 // over warps, and a token's output depends on the tokens before it only through the state: the bits are
 // the same for a whole prompt, its portions and single decoded tokens.
 //
-// Finish kernel: one warp per (token, head): unit norm, weight, gate.
+// Finish kernel: one warp per (token, head): unit norm, weight, gate (silu or sigmoid).  With the norm over all heads of a
+// token together, one block per token.
 #include "common.cuh"
 
 #include <algorithm>
@@ -105,9 +106,12 @@ struct ScanArgs {
     float* out;              // [tokens][heads][vdim] float32: o_t before the norm
     int heads, dim, vdim;
     int max_count = 0;       // > 0: entries with more tokens than this are left to the chunked kernels
+    int silu = 0;            // 1: the value sums pass silu
 };
 
 constexpr int SCAN_CHUNK = 16;
+
+__device__ __forceinline__ float silu_of(float z) { return z / (1.0f + expf(-z)); }
 
 __device__ __forceinline__ void copy_async_16(float* shared_dst, const float* global_src) {
     const uint32_t dst = static_cast<uint32_t>(__cvta_generic_to_shared(shared_dst));
@@ -172,6 +176,7 @@ __global__ void __launch_bounds__(32) gla_scan_kernel(ScanArgs a) {
             if (live && t < count) {
                 const float* src = a.proj + static_cast<size_t>(chunk + t) * a.width + a.v_col + head * a.vdim + column;
                 for (int p = 0; p < a.splits; ++p) v[t] += src[p * a.split_stride];
+                if (a.silu) v[t] = silu_of(v[t]);
             }
         }
     };
@@ -269,6 +274,7 @@ ME_EXPORT int me_gla_scan(const float* proj, int splits, long long split_stride,
     if (dim <= 64) return launch_scan<64>(a, entries, stream);
     if (dim <= 128) return launch_scan<128>(a, entries, stream);
     if (dim <= 192) return launch_scan<192>(a, entries, stream);
+    if (dim <= 256) return launch_scan<256>(a, entries, stream);  // more state than registers: a part of it lives in local memory
     return ME_ERR_UNSUPPORTED;
 }
 
@@ -281,7 +287,8 @@ ME_EXPORT int me_gla_scan(const float* proj, int splits, long long split_stride,
 //
 // Its prepare kernel fills the scan's input: the sums of the product's partial sums, the rotation of the first
 // rotary_dim elements of every head (element e pairs with e + rotary_dim / 2, angles from the step's table), the
-// key scale and the head's decay for every channel, float32.  The scan kernel above then walks the tokens.
+// key scale and the head's decay for every channel, float32.  The scan kernel above then walks the tokens.  With `silu`
+// (lightning attention) the sums of q, k and v are activated, in the place of a rotation.
 struct RetentionPrepArgs {
     const float* proj;  // [splits][tokens][width]
     int splits;
@@ -292,7 +299,7 @@ struct RetentionPrepArgs {
     const float* decay;     // [heads]
     float* prepared;        // [tokens][heads][3][dim]
     float k_scale;
-    int tokens, heads, dim, rotary_dim;
+    int tokens, heads, dim, rotary_dim, silu;
 };
 
 __global__ void __launch_bounds__(256) retention_prepare_kernel(RetentionPrepArgs a) {
@@ -322,6 +329,7 @@ __global__ void __launch_bounds__(256) retention_prepare_kernel(RetentionPrepArg
             q = d < half ? q * angle.x - q_other * angle.y : q * angle.x + q_other * angle.y;
             k = d < half ? k * angle.x - k_other * angle.y : k * angle.x + k_other * angle.y;
         }
+        if (a.silu) q = silu_of(q), k = silu_of(k);
         float* dst = a.prepared + ((token * a.heads + head) * 3) * a.dim + d;
         dst[0] = q;
         dst[a.dim] = k * a.k_scale;
@@ -361,6 +369,7 @@ struct ChunkArgs {
     float* out;          // [tokens][heads][vdim]
     float* chunk_state;  // [chunks][heads][dim][vdim]: first every chunk's own sum, then the state in front of it
     int entries, heads, dim, vdim, min_count;
+    int silu;  // 1: the value sums pass silu
 };
 
 // The entry that chunk number `chunk` belongs to (entries of at least min_count tokens, cut in order).
@@ -384,7 +393,7 @@ __device__ __forceinline__ float value_sum(const ChunkArgs& a, int token, int he
     const float* src = a.proj + static_cast<size_t>(token) * a.width + a.v_col + head * a.vdim + e;
     float v = 0.0f;
     for (int p = 0; p < a.splits; ++p) v += src[p * a.split_stride];
-    return v;
+    return a.silu ? silu_of(v) : v;
 }
 
 // (1) chunk_state[chunk][head] = sum_j a^(n - 1 - j) k_j v_j^T.  One block per (chunk, head).
@@ -622,11 +631,12 @@ ME_EXPORT int me_retention_scan(const float* proj, int splits, long long split_s
                                 int v_col, const float* cos_sin, int rotary_dim, const float* decay, float k_scale,
                                 const int* cu_tokens, const int* state_slots, const int* fresh, float* state, float* out,
                                 float* prepared, int tokens, int entries, int heads, int dim, int vdim, int chunk_min,
-                                float* chunk_state, int max_chunks, cudaStream_t stream) {
+                                float* chunk_state, int max_chunks, int silu, cudaStream_t stream) {
     if (entries <= 0 || tokens <= 0) return 0;
     if (dim < 1 || vdim < 1 || heads < 1 || rotary_dim < 0 || rotary_dim > dim || rotary_dim % 2) return ME_ERR_ARGUMENT;
+    if (silu && cos_sin != nullptr) return ME_ERR_ARGUMENT;
     RetentionPrepArgs p{proj, splits, static_cast<size_t>(split_stride), width, q_col, k_col,
-                        reinterpret_cast<const float2*>(cos_sin), decay, prepared, k_scale, tokens, heads, dim, rotary_dim};
+                        reinterpret_cast<const float2*>(cos_sin), decay, prepared, k_scale, tokens, heads, dim, rotary_dim, silu};
     const size_t total = static_cast<size_t>(tokens) * heads * dim;
     const int blocks = static_cast<int>(std::min<size_t>((total + 255) / 256, 148 * 16));
     int code = launch_kernel(retention_prepare_kernel, blocks, 256, 0, stream, p);
@@ -634,7 +644,7 @@ ME_EXPORT int me_retention_scan(const float* proj, int splits, long long split_s
     if (chunk_min > 0) {
         if (!me_retention_chunked_supports(dim, vdim) || chunk_state == nullptr || max_chunks < 1) return ME_ERR_ARGUMENT;
         ChunkArgs c{proj, splits, static_cast<size_t>(split_stride), width, v_col, prepared, decay, cu_tokens, state_slots,
-                    fresh, state, out, chunk_state, entries, heads, dim, vdim, chunk_min};
+                    fresh, state, out, chunk_state, entries, heads, dim, vdim, chunk_min, silu};
         static SharedMemoryOptIn state_opt_in, output_opt_in;
         const size_t state_smem = static_cast<size_t>(RC) * ((dim + 4) + (vdim + 4)) * sizeof(float);
         const size_t output_smem = chunk_output_smem(dim, vdim);
@@ -647,21 +657,29 @@ ME_EXPORT int me_retention_scan(const float* proj, int splits, long long split_s
         if ((code = launch_kernel_in_order(retention_chunk_output_kernel, dim3(max_chunks, heads), 256, output_smem, stream, c))) return code;
     }
     ScanArgs a{proj, splits, static_cast<size_t>(split_stride), width, v_col, prepared, cu_tokens, state_slots,
-               fresh, state, out, heads, dim, vdim, chunk_min > 0 ? chunk_min - 1 : 0};
+               fresh, state, out, heads, dim, vdim, chunk_min > 0 ? chunk_min - 1 : 0, silu};
     if (dim <= 16) return launch_scan<16>(a, entries, stream);
     if (dim <= 32) return launch_scan<32>(a, entries, stream);
     if (dim <= 64) return launch_scan<64>(a, entries, stream);
     if (dim <= 128) return launch_scan<128>(a, entries, stream);
     if (dim <= 192) return launch_scan<192>(a, entries, stream);
+    if (dim <= 256) return launch_scan<256>(a, entries, stream);  // more state than registers: a part of it lives in local memory
     return ME_ERR_UNSUPPORTED;
 }
 
-// out[t][h][e] = weight[e] * o[t][h][e] * rsqrt(mean_e(o^2) + eps) * silu(gate[t][h][e]); a null weight is all ones.
+// out[t][h][e] = weight[e] * o[t][h][e] * rsqrt(mean_e(o^2) + eps) * gate(g[t][h][e]); a null weight is all ones.  The gate
+// is silu or the sigmoid.
+enum : int { FINISH_SILU = 0, FINISH_SIGMOID = 1 };
+
+__device__ __forceinline__ float finish_gate(float g, int kind) {
+    return (kind == FINISH_SIGMOID ? 1.0f : g) / (1.0f + expf(-g));
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128) gla_finish_kernel(const float* __restrict__ o, const float* __restrict__ proj,
                                                          int splits, size_t split_stride, int width, int g_col,
                                                          const float* __restrict__ weight, float eps,
-                                                         T* __restrict__ out, int tokens, int heads, int vdim) {
+                                                         T* __restrict__ out, int tokens, int heads, int vdim, int gate_kind) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long item = static_cast<long long>(blockIdx.x) * 4 + warp;
     pdl_trigger();
@@ -679,21 +697,58 @@ __global__ void __launch_bounds__(128) gla_finish_kernel(const float* __restrict
     for (int e = lane; e < vdim; e += 32) {
         float gate = 0.0f;
         for (int p = 0; p < splits; ++p) gate += gate_row[p * split_stride + e];
-        const float activated = gate / (1.0f + expf(-gate));
-        dst[e] = from_float<T>((weight ? weight[e] : 1.0f) * (row[e] * inv) * activated);
+        dst[e] = from_float<T>((weight ? weight[e] : 1.0f) * (row[e] * inv) * finish_gate(gate, gate_kind));
+    }
+}
+
+// The same with the root mean square over all `count` columns of a token (every head together) and a weight of that size.
+// One block per token; column i's square goes to the partial sum of thread i % 256 in ascending order.
+template <typename T>
+__global__ void __launch_bounds__(256) projection_finish_kernel(const float* __restrict__ o, const float* __restrict__ proj,
+                                                                int splits, size_t split_stride, int width, int g_col,
+                                                                const float* __restrict__ weight, float eps,
+                                                                T* __restrict__ out, int count, int gate_kind) {
+    __shared__ float partial[8];
+    const size_t token = blockIdx.x;
+    pdl_trigger();
+    pdl_wait();
+    const float* row = o + token * count;
+    float sum_sq = 0.0f;
+    for (int i = threadIdx.x; i < count; i += 256) sum_sq = fmaf(row[i], row[i], sum_sq);
+    sum_sq = warp_sum(sum_sq);
+    if ((threadIdx.x & 31) == 0) partial[threadIdx.x >> 5] = sum_sq;
+    __syncthreads();
+    float total = 0.0f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) total += partial[w];
+    const float inv = rsqrtf(total / static_cast<float>(count) + eps);
+    const float* gate_row = proj + token * width + g_col;
+    T* dst = out + token * count;
+    for (int i = threadIdx.x; i < count; i += 256) {
+        float gate = 0.0f;
+        for (int p = 0; p < splits; ++p) gate += gate_row[p * split_stride + i];
+        dst[i] = from_float<T>((weight ? weight[i] : 1.0f) * (row[i] * inv) * finish_gate(gate, gate_kind));
     }
 }
 
 ME_EXPORT int me_gla_finish(const float* o, const float* proj, int splits, long long split_stride, int width,
                             int g_col, const float* weight, float eps, void* out, int type, int tokens, int heads,
-                            int vdim, cudaStream_t stream) {
+                            int vdim, int gate_kind, int whole_projection, cudaStream_t stream) {
     if (tokens <= 0) return 0;
+    if (gate_kind != FINISH_SILU && gate_kind != FINISH_SIGMOID) return ME_ERR_ARGUMENT;
+    if (whole_projection) {
+        if (type == ME_BF16)
+            return launch_kernel(projection_finish_kernel<__nv_bfloat16>, tokens, 256, 0, stream, o, proj, splits, (size_t)split_stride,
+                                 width, g_col, weight, eps, static_cast<__nv_bfloat16*>(out), heads * vdim, gate_kind);
+        return launch_kernel(projection_finish_kernel<float>, tokens, 256, 0, stream, o, proj, splits, (size_t)split_stride, width,
+                             g_col, weight, eps, static_cast<float*>(out), heads * vdim, gate_kind);
+    }
     const long long items = static_cast<long long>(tokens) * heads;
     const int blocks = static_cast<int>((items + 3) / 4);
     if (type == ME_BF16)
         return launch_kernel(gla_finish_kernel<__nv_bfloat16>, blocks, 128, 0, stream, o, proj, splits,
                              (size_t)split_stride, width, g_col, weight, eps, static_cast<__nv_bfloat16*>(out), tokens,
-                             heads, vdim);
+                             heads, vdim, gate_kind);
     return launch_kernel(gla_finish_kernel<float>, blocks, 128, 0, stream, o, proj, splits, (size_t)split_stride, width,
-                         g_col, weight, eps, static_cast<float*>(out), tokens, heads, vdim);
+                         g_col, weight, eps, static_cast<float*>(out), tokens, heads, vdim, gate_kind);
 }

@@ -399,12 +399,14 @@ def qk_norm_rope_store(
 
 
 def rope_table(inv_freq: torch.Tensor, positions: torch.Tensor, out: torch.Tensor) -> None:
-    """``out[t, i] = (cos, sin)(positions[t] * inv_freq[i])`` in float32, ``[T, rotary_dim / 2, 2]``."""
-    _need(inv_freq, torch.float32, "inv_freq"), _need(positions, torch.int32, "positions"), _need(out, torch.float32, "out")
+    """``out[t, i] = (cos, sin)(positions[t] * inv_freq[i])`` in float32, ``[T, rotary_dim / 2, 2]``.  With float64
+    frequencies the angle is formed, and reduced to one turn, in double precision."""
+    double = inv_freq.dtype == torch.float64
+    _need(inv_freq, torch.float64 if double else torch.float32, "inv_freq"), _need(positions, torch.int32, "positions"), _need(out, torch.float32, "out")
     tokens, half = positions.shape[0], inv_freq.shape[0]
     if tuple(out.shape) != (tokens, half, 2):
         raise KernelError(f"rope_table: out {tuple(out.shape)} is not [{tokens}, {half}, 2]")
-    fn = _fn("elementwise", "me_rope_table", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p])
+    fn = _fn("elementwise", "me_rope_table_double" if double else "me_rope_table", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p])
     _check(fn(_ptr(inv_freq), _ptr(positions), _ptr(out), tokens, half, _stream()), "rope_table")
 
 
@@ -452,6 +454,10 @@ def GemmPlan(weight: torch.Tensor, dual_rows: int | None = None):  # noqa: N802 
 
 def gemm_tensor_core(plan, x: torch.Tensor, out: torch.Tensor, splits: int) -> None:
     tensor_core.gemm(plan, x, out, splits)
+
+
+def gemm_tensor_core_activated(plan, x: torch.Tensor, act: torch.Tensor, activation: str) -> None:
+    tensor_core.gemm_activated(plan, x, act, PLAIN_ACTIVATIONS[activation])
 
 
 def gemm_tensor_core_swiglu(plan, x: torch.Tensor, act: torch.Tensor, activation: str = "silu") -> None:
@@ -845,24 +851,33 @@ def gla_scan(
     _check(code, "gla_scan")
 
 
+FINISH_GATES = {"silu": 0, "sigmoid": 1}
+RETENTION_MAX_DIM = 256  # key channels per head that the walking kernel takes
+
+
 def gla_finish(
     *, o: torch.Tensor, proj: torch.Tensor, gate_column: int, weight: torch.Tensor | None, eps: float, out: torch.Tensor,
-    heads: int, vdim: int,
+    heads: int, vdim: int, gate: str = "silu", scope: str = "head",
 ) -> None:  # fmt: skip
     """``out = weight * o / rms(o) * silu(gate)`` per (token, head); the gate is a column range of ``proj``;
-    ``weight=None`` is a weight of ones."""
+    ``weight=None`` is a weight of ones.  ``gate="sigmoid"`` multiplies by the gate's sigmoid; ``scope="projection"`` takes
+    the root mean square over all heads of a token together, with a weight ``[heads * vdim]``."""
+    if gate not in FINISH_GATES or scope not in ("head", "projection"):
+        raise KernelError("gla_finish: the gate is 'silu' or 'sigmoid', the scope 'head' or 'projection'")
     _need(o, torch.float32, "o"), _need(proj, torch.float32, "proj"), _need(out, None, "out")
     if weight is not None:
         _need(weight, torch.float32, "weight")
+        if weight.shape != (vdim if scope == "head" else heads * vdim,):
+            raise KernelError("gla_finish: the weight does not fit the scope of the norm")
     tokens = o.shape[0]
     fn = _fn(
         "linear_attention",
         "me_gla_finish",
-        [c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_void_p, c_float, c_void_p] + [c_int] * 4 + [c_void_p],
+        [c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_void_p, c_float, c_void_p] + [c_int] * 6 + [c_void_p],
     )
     code = fn(
         _ptr(o), _ptr(proj), proj.shape[0], proj.stride(0), proj.shape[2], gate_column, _ptr(weight), float(eps), _ptr(out),
-        _type_code(out.dtype), tokens, heads, vdim, _stream(),
+        _type_code(out.dtype), tokens, heads, vdim, FINISH_GATES[gate], 1 if scope == "projection" else 0, _stream(),
     )  # fmt: skip
     _check(code, "gla_finish")
 
@@ -880,7 +895,7 @@ def retention_chunked_supports(dim: int, vdim: int) -> bool:
 def retention_scan(
     *, proj: torch.Tensor, columns: dict[str, int], cos_sin: torch.Tensor | None, decay: torch.Tensor, k_scale: float, ctx,
     state: torch.Tensor, out: torch.Tensor, prepared: torch.Tensor, heads: int, dim: int, vdim: int,
-    chunk_min: int = 0, chunk_state: torch.Tensor | None = None,
+    chunk_min: int = 0, chunk_state: torch.Tensor | None = None, silu: bool = False,
 ) -> None:  # fmt: skip
     """The recurrence ``S_t = decay_h S_(t-1) + k_t v_t^T``, ``o_t = S_t^T q_t`` over the batch's tokens, entry by entry,
     from and into each request's state slot.  ``proj`` is ``[S, T, width]`` float32 partial sums whose ``columns`` ``q, k,
@@ -889,7 +904,8 @@ def retention_scan(
     ``out`` is float32 ``[T, heads, vdim]``; ``prepared`` is float32 scratch of ``T * heads * 3 * dim`` values.
     ``chunk_min`` > 0: entries of at least that many tokens run in chunks of ``RETENTION_CHUNK`` tokens whose blocks work
     side by side (the closed form of the recurrence over a chunk), with ``chunk_state [chunks, heads, dim, vdim]`` float32 as
-    scratch for at least ``sum ceil(tokens / RETENTION_CHUNK)`` chunks; the other entries walk token by token."""
+    scratch for at least ``sum ceil(tokens / RETENTION_CHUNK)`` chunks; the other entries walk token by token.  ``silu``: the sums
+    of q, k and v pass silu first (without a rotation)."""
     _need(proj, torch.float32, "proj"), _need(decay, torch.float32, "decay"), _need(state, torch.float32, "state")
     max_chunks = 0
     if chunk_min:
@@ -913,13 +929,13 @@ def retention_scan(
         "linear_attention",
         "me_retention_scan",
         [c_void_p, c_int, c_longlong] + [c_int] * 4 + [c_void_p, c_int, c_void_p, c_float] + [c_void_p] * 6 + [c_int] * 6
-        + [c_void_p, c_int, c_void_p],
+        + [c_void_p, c_int, c_int, c_void_p],
     )
     code = fn(
         _ptr(proj), proj.shape[0], proj.stride(0), proj.shape[2], columns["q"], columns["k"], columns["v"], _ptr(cos_sin),
         rotary_dim, _ptr(decay), float(k_scale), _ptr(ctx.cu_tokens), _ptr(ctx.state_slots), _ptr(ctx.fresh), _ptr(state),
         _ptr(out), _ptr(prepared), tokens, ctx.num_entries, heads, dim, vdim, int(chunk_min), _ptr(chunk_state), max_chunks,
-        _stream(),
+        1 if silu else 0, _stream(),
     )  # fmt: skip
     _check(code, "retention_scan")
 
@@ -998,21 +1014,28 @@ def hyper_sum(
     _check(code, "hyper_sum")
 
 
-PLAIN_ACTIVATIONS = {"relu_squared": 0, "silu": 1, "gelu_tanh": 2, "relu": 3}
+PLAIN_ACTIVATIONS = {"relu_squared": 0, "silu": 1, "gelu_tanh": 2, "relu": 3, "gelu_erf": 4}
 
 
-def activation(partials: torch.Tensor, out: torch.Tensor, kind: str) -> None:
+def activation(partials: torch.Tensor, out: torch.Tensor, kind: str, group_weight: torch.Tensor | None = None) -> None:
     """``out = act(sum_s partials[s])`` in the dtype of ``out``: ``relu_squared`` (``max(z, 0)^2``), ``silu``,
-    ``gelu_tanh`` or ``relu``, for a feed-forward without a gate."""
+    ``gelu_tanh``, ``relu`` or ``gelu_erf`` (``0.5 z (1 + erf(z / sqrt 2))``), for a feed-forward without a gate.  With
+    ``group_weight`` (float32 ``[T, groups]``) the features form ``groups`` equal runs, multiplied by their run's weight."""
     if kind not in PLAIN_ACTIVATIONS:
         raise KernelError(f"activation: kind must be one of {sorted(PLAIN_ACTIVATIONS)}, got {kind!r}")
     _need(partials, torch.float32, "partials"), _need(out, None, "out")
     splits, tokens, width = partials.shape
     if out.shape != (tokens, width):
         raise KernelError(f"activation: out {tuple(out.shape)} does not fit partials {tuple(partials.shape)}")
-    fn = _fn("elementwise", "me_activation", [c_void_p, c_int, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    group_size = 0
+    if group_weight is not None:
+        _need(group_weight, torch.float32, "group_weight")
+        if group_weight.dim() != 2 or group_weight.shape[0] != tokens or width % group_weight.shape[1]:
+            raise KernelError(f"activation: group_weight {tuple(group_weight.shape)} does not fit {tokens} tokens of {width} features")
+        group_size = width // group_weight.shape[1]
+    fn = _fn("elementwise", "me_activation", [c_void_p, c_int, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p])
     code = fn(_ptr(partials), splits, partials.stride(0), _ptr(out), _type_code(out.dtype), tokens, width,
-              PLAIN_ACTIVATIONS[kind], _stream())  # fmt: skip
+              PLAIN_ACTIVATIONS[kind], _ptr(group_weight), group_size, _stream())  # fmt: skip
     _check(code, "activation")
 
 
@@ -1020,12 +1043,13 @@ def qkv_rope_unit_store(
     *, qkv: torch.Tensor, heads: int, kv_heads: int, head_dim: int, value_dim: int, bias: torch.Tensor | None,
     cos_sin: torch.Tensor | None, unit_norm_eps: float | None, q_out: torch.Tensor, page_size: int,
     slot_mapping: torch.Tensor | None = None, k_pages: torch.Tensor | None = None, v_pages: torch.Tensor | None = None,
-    k_dense: torch.Tensor | None = None, v_dense: torch.Tensor | None = None,
+    k_dense: torch.Tensor | None = None, v_dense: torch.Tensor | None = None, value_cos_sin: torch.Tensor | None = None,
 ) -> None:  # fmt: skip
     """``qkv [S, T, width]`` float32 partial sums with the columns ``[q | k | v]``: add ``bias`` (float32 ``[width]``),
     rotate the first ``rotary_dim`` elements of every q and k head by ``cos_sin [T, rotary_dim / 2, 2]``, then (with
     ``unit_norm_eps``) divide every rotated q and k head by its root mean square over ``head_dim``, eps inside the root;
-    q goes to ``q_out``, k and v to their cache slots (or dense buffers)."""
+    q goes to ``q_out``, k and v to their cache slots (or dense buffers).  ``value_cos_sin [T, value_dim / 2, 2]`` rotates the
+    value heads, over their whole width."""
     _need(qkv, torch.float32, "qkv"), _need(q_out, None, "q_out")
     splits, tokens, width = qkv.shape
     if width != (heads + kv_heads) * head_dim + kv_heads * value_dim:
@@ -1048,14 +1072,161 @@ def qkv_rope_unit_store(
         _need(bias, torch.float32, "bias")
         if bias.shape != (width,):
             raise KernelError(f"bias {tuple(bias.shape)} does not fit the {width} columns of qkv")
+    if value_cos_sin is not None:
+        _need(value_cos_sin, torch.float32, "value_cos_sin")
+        if tuple(value_cos_sin.shape) != (tokens, value_dim // 2, 2) or value_dim % 2:
+            raise KernelError(f"value_cos_sin {tuple(value_cos_sin.shape)} is not [tokens, value_dim / 2, 2]")
     fn = _fn("elementwise", "me_qkv_rope_unit_store",
-             [c_void_p, c_int, c_longlong, c_int] + [c_void_p] * 8 + [c_float] + [c_int] * 9 + [c_void_p])  # fmt: skip
+             [c_void_p, c_int, c_longlong, c_int] + [c_void_p] * 8 + [c_float] + [c_int] * 9 + [c_void_p, c_void_p])  # fmt: skip
     code = fn(
         _ptr(qkv), splits, qkv.stride(0), width, _ptr(bias), _ptr(cos_sin), _ptr(slot_mapping), _ptr(q_out), _ptr(k_pages),
         _ptr(v_pages), _ptr(k_dense), _ptr(v_dense), float(unit_norm_eps or 0.0), _type_code(q_out.dtype), tokens, heads,
-        kv_heads, head_dim, value_dim, page_size, rotary_dim, 1 if unit_norm_eps is not None else 0, _stream(),
+        kv_heads, head_dim, value_dim, page_size, rotary_dim, 1 if unit_norm_eps is not None else 0,
+        _ptr(value_cos_sin), _stream(),
     )  # fmt: skip
     _check(code, "qkv_rope_unit_store")
+
+
+def turn_heads_back(x: torch.Tensor, cos_sin: torch.Tensor, heads: int) -> None:
+    """In place on ``x [T, heads * dim]``: every head rotated (rotate-half, over its whole width) by the negative of its
+    token's angles ``cos_sin [T, dim / 2, 2]``."""
+    _need(x, None, "x"), _need(cos_sin, torch.float32, "cos_sin")
+    tokens, width = x.shape
+    if width % (2 * heads) or tuple(cos_sin.shape) != (tokens, width // heads // 2, 2):
+        raise KernelError(f"turn_heads_back: {tuple(cos_sin.shape)} does not fit {heads} heads of {tuple(x.shape)}")
+    fn = _fn("elementwise", "me_turn_heads_back", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p])
+    _check(fn(_ptr(x), _type_code(x.dtype), _ptr(cos_sin), tokens, heads, width // heads, _stream()), "turn_heads_back")
+
+
+# -------------------------------------------------- sublayers between two norms, and the delta rule
+
+
+MAX_CONV_TAPS = 16  # taps of a short convolution over time
+DELTA_MAX_DIM = 512  # key channels per head of the delta rule
+
+
+def sandwich_norm(
+    *, x: torch.Tensor, pending: torch.Tensor, bias: torch.Tensor | None, gate: torch.Tensor | None, gate_bias: torch.Tensor | None,
+    out_weight: torch.Tensor, out_eps: float, weight: torch.Tensor, eps: float, out: torch.Tensor, rows: torch.Tensor | None = None,
+) -> None:  # fmt: skip
+    """``y = (sum_s pending[s] + bias) * sigmoid(sum_s gate[s] + gate_bias)``, ``x += out_weight * y / rms(y)`` (in place,
+    float32) and ``out = weight * x / rms(x)``.  With ``rows`` (int32) only these rows are produced and ``x`` is left as it
+    was."""
+    _need(x, torch.float32, "x"), _need(pending, torch.float32, "pending"), _need(out, None, "out")
+    tokens, hidden = x.shape
+    for name, sums in (("pending", pending), ("gate", gate)):
+        if sums is not None:
+            _need(sums, torch.float32, name)
+            if sums.dim() != 3 or sums.shape[1:] != (tokens, hidden):
+                raise KernelError(f"sandwich_norm: {name} {tuple(sums.shape)} does not fit x {tuple(x.shape)}")
+    for name, vector in (("bias", bias), ("gate_bias", gate_bias), ("out_weight", out_weight), ("weight", weight)):
+        if vector is not None:
+            _need(vector, torch.float32, name)
+            if vector.shape != (hidden,):
+                raise KernelError(f"sandwich_norm: {name} must have one value per column")
+    if rows is not None:
+        _need(rows, torch.int32, "rows")
+    count = tokens if rows is None else rows.shape[0]
+    if out.shape != (count, hidden):
+        raise KernelError("sandwich_norm: out does not fit")
+    fn = _fn("sandwich", "me_sandwich_norm",
+             [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_float,
+              c_void_p, c_int, c_void_p, c_int, c_int, c_void_p])  # fmt: skip
+    code = fn(
+        _ptr(x), _ptr(pending), pending.shape[0], pending.stride(0), _ptr(bias), _ptr(gate), 0 if gate is None else gate.shape[0],
+        0 if gate is None else gate.stride(0), _ptr(gate_bias), _ptr(out_weight), float(out_eps), _ptr(weight), float(eps),
+        _ptr(out), _type_code(out.dtype), _ptr(rows), count, hidden, _stream(),
+    )  # fmt: skip
+    _check(code, "sandwich_norm")
+
+
+def input_convolution(*, h: torch.Tensor, taps: torch.Tensor, ctx, state: torch.Tensor | None, out: torch.Tensor) -> None:
+    """``out_t = h_t + sum_j taps[j] * h_(t - K + 1 + j)`` per channel within every entry's request (``taps [K, width]``
+    float32), from and into ``state [slots + 1, K - 1, width]`` (float32: the request's last ``K - 1`` inputs; ``None`` for
+    one tap)."""
+    _need(h, None, "h"), _need(out, h.dtype, "out"), _need(taps, torch.float32, "taps")
+    tokens, width = h.shape
+    count = taps.shape[0]
+    if taps.shape != (count, width) or out.shape != h.shape or (state is None) != (count == 1):
+        raise KernelError("input_convolution: taps, state or out do not fit")
+    if state is not None:
+        _need(state, torch.float32, "state")
+        if state.shape[1:] != (count - 1, width):
+            raise KernelError(f"input_convolution: state {tuple(state.shape)} is not [slots + 1, {count - 1}, {width}]")
+    fn = _fn("sandwich", "me_input_convolution", [c_void_p, c_int] + [c_void_p] * 7 + [c_int] * 3 + [c_void_p])
+    code = fn(
+        _ptr(h), _type_code(h.dtype), _ptr(taps), _ptr(ctx.entry_of_token), _ptr(ctx.cu_tokens), _ptr(ctx.state_slots),
+        _ptr(ctx.fresh), _ptr(state), _ptr(out), tokens, width, count, _stream(),
+    )  # fmt: skip
+    _check(code, "input_convolution")
+
+
+def split_halves(proj: torch.Tensor, column: int, count: int, out: torch.Tensor) -> None:
+    """The columns ``column .. column + count`` of ``sum_s proj[s]``: rounded to bfloat16, and behind them what the rounding
+    left, rounded to bfloat16 (``out [T, 2 * count]``); with a float32 ``out [T, count]`` the sums themselves."""
+    _need(proj, torch.float32, "proj"), _need(out, None, "out")
+    splits, tokens, width = proj.shape
+    if out.shape != (tokens, count * (2 if out.dtype == torch.bfloat16 else 1)) or column + count > width:
+        raise KernelError("split_halves: out or the columns do not fit")
+    fn = _fn("delta_rule", "me_split_halves", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p])
+    code = fn(_ptr(proj), splits, proj.stride(0), width, column, count, _ptr(out), _type_code(out.dtype), tokens, _stream())
+    _check(code, "split_halves")
+
+
+def delta_prepare(
+    *, proj: torch.Tensor, columns: dict[str, int], second: torch.Tensor, conv: torch.Tensor, a_log: torch.Tensor,
+    dt_bias: torch.Tensor, ctx, state: torch.Tensor, matrix: int, qk: torch.Tensor, gv: torch.Tensor, scalars: torch.Tensor,
+    q_scale: float, unit_eps: float, heads: int, qk_heads: int, dim: int, vdim: int,
+) -> None:  # fmt: skip
+    """What the delta rule's recurrence takes, for all tokens of the batch, in float32: from the partial sums ``proj [S, T,
+    width]`` (``columns`` says where ``q``, ``k``, ``v`` and ``beta`` start; q, k and v are its first columns) the short
+    convolutions (``conv [K, channels]``) with silu, unit q (times ``q_scale``) and k and their dot product, ``beta``; from
+    ``second [S', T, heads * dim + ...]`` the decays ``exp(-exp(a_log) * softplus(second + dt_bias))``.  ``state`` is ``[slots +
+    1, floats]``: behind ``matrix`` floats of matrix states it holds the convolution's last ``K - 1`` inputs ``[K - 1,
+    channels]``, read and replaced here.  Outputs: ``qk [T, qk_heads, 2, dim]``, ``gv [T, heads, dim + vdim]`` (decays, then
+    values), ``scalars [T, heads, 2]`` (beta, q . k)."""
+    for name, t in (("proj", proj), ("second", second), ("conv", conv), ("a_log", a_log), ("dt_bias", dt_bias), ("state", state),
+                    ("qk", qk), ("gv", gv), ("scalars", scalars)):  # fmt: skip
+        _need(t, torch.float32, name)
+    splits, tokens, width = proj.shape
+    taps, channels = conv.shape
+    if second.shape[1] != tokens or second.shape[2] < heads * dim or a_log.shape != (heads,) or dt_bias.shape != (heads * dim,):
+        raise KernelError("delta_prepare: the decay's logits or constants do not fit heads and dim")
+    if channels != 2 * qk_heads * dim + heads * vdim or columns["v"] + heads * vdim > width or columns["beta"] + heads > width:
+        raise KernelError("delta_prepare: the projection's columns do not fit the head sizes")
+    if state.dim() != 2 or state.shape[1] < matrix + (taps - 1) * channels:
+        raise KernelError("delta_prepare: the state does not hold the convolution's past")
+    if qk.numel() < tokens * qk_heads * 2 * dim or gv.numel() < tokens * heads * (dim + vdim) or scalars.numel() < tokens * heads * 2:
+        raise KernelError("delta_prepare: outputs too small")
+    fn = _fn("delta_rule", "me_delta_prepare",
+             [c_void_p, c_int, c_longlong] + [c_int] * 5 + [c_void_p, c_int, c_longlong, c_int] + [c_void_p] * 8 + [c_longlong, c_longlong]
+             + [c_void_p] * 3 + [c_float, c_float] + [c_int] * 7 + [c_void_p])  # fmt: skip
+    code = fn(
+        _ptr(proj), splits, proj.stride(0), width, columns["q"], columns["k"], columns["v"], columns["beta"], _ptr(second),
+        second.shape[0], second.stride(0), second.shape[2], _ptr(conv), _ptr(a_log), _ptr(dt_bias), _ptr(ctx.entry_of_token),
+        _ptr(ctx.cu_tokens), _ptr(ctx.state_slots), _ptr(ctx.fresh), _ptr(state), state.shape[1], int(matrix), _ptr(qk), _ptr(gv),
+        _ptr(scalars), float(q_scale), float(unit_eps), tokens, heads, qk_heads, dim, vdim, taps, channels, _stream(),
+    )  # fmt: skip
+    _check(code, "delta_prepare")
+
+
+def delta_scan(
+    *, qk: torch.Tensor, gv: torch.Tensor, scalars: torch.Tensor, ctx, state: torch.Tensor, out: torch.Tensor, heads: int,
+    qk_heads: int, dim: int, vdim: int,
+) -> None:  # fmt: skip
+    """The recurrence of the gated delta rule over the batch's tokens, entry by entry, from and into each request's state
+    slot (``state [slots + 1, floats]``, a slot starts with ``[heads, vdim, dim]``), on what :func:`delta_prepare` made;
+    ``out`` is float32 ``[T, heads, vdim]``."""
+    for name, t in (("qk", qk), ("gv", gv), ("scalars", scalars), ("state", state), ("out", out)):
+        _need(t, torch.float32, name)
+    if state.dim() != 2 or state.shape[1] < heads * dim * vdim:
+        raise KernelError("delta_scan: the state does not hold the matrix states")
+    fn = _fn("delta_rule", "me_delta_scan", [c_void_p] * 7 + [c_longlong, c_void_p] + [c_int] * 5 + [c_void_p])
+    code = fn(
+        _ptr(qk), _ptr(gv), _ptr(scalars), _ptr(ctx.cu_tokens), _ptr(ctx.state_slots), _ptr(ctx.fresh), _ptr(state),
+        state.shape[1], _ptr(out), ctx.num_entries, heads, qk_heads, dim, vdim, _stream(),
+    )  # fmt: skip
+    _check(code, "delta_scan")
 
 
 def pair_embedding(
@@ -1191,43 +1362,55 @@ def rglru(
     _check(code, "rglru")
 
 
-ROUTE_SCORINGS = {"sigmoid": 0, "softmax_chosen": 1}
+ROUTE_SCORINGS = {"sigmoid": 0, "softmax_chosen": 1, "softmax_all": 2}
 
 
 def route(
     *, h: torch.Tensor, router: torch.Tensor, weights: torch.Tensor, chosen: torch.Tensor, chosen_weight: torch.Tensor,
     top: int, group_count: int, group_keep: int, weight_scale: float, bias: torch.Tensor | None = None,
-    scoring: str = "sigmoid",
+    scoring: str = "sigmoid", correction: torch.Tensor | None = None, identity_weight: torch.Tensor | None = None,
+    shared_gate: torch.Tensor | None = None,
 ) -> None:  # fmt: skip
     """Per token the ``top`` units with the largest ``sigmoid(router h)`` among the units of the ``group_keep`` best
     of ``group_count`` equal groups of neighbours (a group's value: the sum of its two largest scores); weights are
     the chosen scores over their sum, times ``weight_scale``.  ``weights [T, units]`` float32 gets them densely (zero
     elsewhere), ``chosen`` (int32) and ``chosen_weight`` (float32) ``[T, top]`` as lists.  ``bias`` (float32 ``[units]``)
     is added to ``router h``.  ``scoring="softmax_chosen"``: the units with the largest logits are chosen and their weights
-    are the softmax over the chosen logits only (times ``weight_scale``)."""
+    are the softmax over the chosen logits only (times ``weight_scale``).  ``scoring="softmax_all"``: the choice is made by the
+    softmax over all units plus ``correction`` (float32 ``[units]``), a group's value is its largest one, and the weights
+    are the softmax times ``weight_scale``.  Units of ``router`` behind the columns of ``weights`` have no tensors: the sum of
+    their weights goes to ``identity_weight [T]``.  ``shared_gate [T]``: the router's last row is no unit, its sigmoid goes
+    there."""
     if scoring not in ROUTE_SCORINGS:
         raise KernelError(f"route: scoring must be one of {sorted(ROUTE_SCORINGS)}, got {scoring!r}")
-    if bias is not None:
-        _need(bias, torch.float32, "bias")
-        if bias.shape != (router.shape[0],):
-            raise KernelError("route: one bias per unit")
+    units = router.shape[0] - (0 if shared_gate is None else 1)
+    tensorless = units - weights.shape[1]
+    for name, vector, length in (("bias", bias, units), ("correction", correction, units),
+                                 ("identity_weight", identity_weight, h.shape[0]), ("shared_gate", shared_gate, h.shape[0])):  # fmt: skip
+        if vector is not None:
+            _need(vector, torch.float32, name)
+            if vector.shape != (length,):
+                raise KernelError(f"route: {name} must hold {length} values")
+    if tensorless < 0 or (tensorless > 0) != (identity_weight is not None):
+        raise KernelError("route: units without tensors and identity_weight come together")
     _need(h, None, "h"), _need(router, torch.float32, "router"), _need(weights, torch.float32, "weights")
     _need(chosen, torch.int32, "chosen"), _need(chosen_weight, torch.float32, "chosen_weight")
     tokens, hidden = h.shape
-    units = router.shape[0]
-    if router.shape != (units, hidden) or weights.shape != (tokens, units) or chosen.shape != (tokens, top) or chosen_weight.shape != (tokens, top):
+    if router.shape[1] != hidden or weights.shape[0] != tokens or chosen.shape != (tokens, top) or chosen_weight.shape != (tokens, top):
         raise KernelError("route: shapes do not fit")
-    fn = _fn("routing", "me_route", [c_void_p, c_int, c_void_p, c_void_p, c_int] + [c_void_p] * 3 + [c_int] * 6 + [c_float, c_void_p])
+    fn = _fn("routing", "me_route", [c_void_p, c_int, c_void_p, c_void_p, c_int] + [c_void_p] * 3 + [c_int] * 6 + [c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p])
     code = fn(
         _ptr(h), _type_code(h.dtype), _ptr(router), _ptr(bias), ROUTE_SCORINGS[scoring], _ptr(weights), _ptr(chosen), _ptr(chosen_weight), tokens, hidden,
-        units, int(top), int(group_count), int(group_keep), float(weight_scale), _stream(),
+        units, int(top), int(group_count), int(group_keep), float(weight_scale), _ptr(correction), tensorless, _ptr(identity_weight),
+        _ptr(shared_gate), _stream(),
     )  # fmt: skip
     _check(code, "route")
 
 
 def sort_by_unit(*, chosen: torch.Tensor, units: int, pad: int, row_of: torch.Tensor, token_of: torch.Tensor,
                  unit_of_block: torch.Tensor) -> None:  # fmt: skip
-    """Rows sorted by unit for grouped products: every (token, choice) of ``chosen [T, top]`` gets a row, each unit's
+    """Rows sorted by unit for grouped products: every (token, choice) of ``chosen [T, top]`` gets a row (choices outside
+    ``[0, units)`` get none: -1), each unit's
     run padded to a multiple of ``pad``.  ``row_of [T, top]``, ``token_of [capacity]`` (-1: no token) and
     ``unit_of_block [capacity / pad]`` (-1: no rows) are int32 outputs; ``capacity >= T * top + units * (pad - 1)``."""
     for name, t in (("chosen", chosen), ("row_of", row_of), ("token_of", token_of), ("unit_of_block", unit_of_block)):
@@ -1261,8 +1444,53 @@ def combine_rows(sorted_out: torch.Tensor, row_of: torch.Tensor, weight: torch.T
     _check(fn(_ptr(sorted_out), _ptr(row_of), _ptr(weight), _ptr(out), tokens, top, out.shape[1], _stream()), "combine_rows")
 
 
-def gemm_tensor_core_grouped(plan, x, out, group_of_block, group_rows, outs, dual_rows=0, slope=1.0, limit=None, offset=0.0) -> None:
-    tensor_core.gemm_grouped(plan, x, out, group_of_block, group_rows, outs, dual_rows, slope, limit, offset)
+def moe_finish(
+    *, out: torch.Tensor, routed: torch.Tensor | None = None, sorted_out: torch.Tensor | None = None, row_of: torch.Tensor | None = None,
+    weight: torch.Tensor | None = None, h: torch.Tensor | None = None, identity_weight: torch.Tensor | None = None,
+    shared: torch.Tensor | None = None, shared_gate: torch.Tensor | None = None,
+) -> None:  # fmt: skip
+    """``out [T, width]`` (float32) ``= routed + identity_weight * h + shared_gate * sum_s shared[s]``.  The first term is
+    ``sum_s routed[s]`` (``[S, T, width]``), or the rows of ``sorted_out`` joined as in :func:`combine_rows`; the second and the
+    third may be absent, and a shared output without a gate has weight one."""
+    _need(out, torch.float32, "out")
+    tokens, width = out.shape
+    top = 0
+    if (routed is None) == (sorted_out is None):
+        raise KernelError("moe_finish: either partial sums or sorted rows")
+    if sorted_out is not None:
+        _need(sorted_out, torch.float32, "sorted_out"), _need(row_of, torch.int32, "row_of"), _need(weight, torch.float32, "weight")
+        top = row_of.shape[1]
+        if row_of.shape != (tokens, top) or weight.shape != row_of.shape or sorted_out.shape[1] != width:
+            raise KernelError("moe_finish: the sorted rows do not fit")
+    for name, sums in (("routed", routed), ("shared", shared)):
+        if sums is not None:
+            _need(sums, torch.float32, name)
+            if sums.dim() != 3 or sums.shape[1:] != (tokens, width):
+                raise KernelError(f"moe_finish: {name} {tuple(sums.shape)} does not fit out {tuple(out.shape)}")
+    for name, vector in (("identity_weight", identity_weight), ("shared_gate", shared_gate)):
+        if vector is not None:
+            _need(vector, torch.float32, name)
+            if vector.shape != (tokens,):
+                raise KernelError(f"moe_finish: {name} must hold one value per token")
+    if identity_weight is not None and (h is None or h.shape != (tokens, width) or not h.is_contiguous()):
+        raise KernelError("moe_finish: identity units need the input rows")
+    first = routed if routed is not None else sorted_out
+    fn = _fn("routing", "me_moe_finish",
+             [c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_longlong, c_void_p,
+              c_void_p, c_int, c_int, c_void_p])  # fmt: skip
+    code = fn(
+        _ptr(first), 0 if routed is None else routed.shape[0], 0 if routed is None else routed.stride(0),
+        _ptr(row_of if sorted_out is not None else None), _ptr(weight if sorted_out is not None else None), top, _ptr(h),
+        F32 if h is None else _type_code(h.dtype), _ptr(identity_weight), _ptr(shared), 0 if shared is None else shared.shape[0],
+        0 if shared is None else shared.stride(0), _ptr(shared_gate), _ptr(out), tokens, width, _stream(),
+    )  # fmt: skip
+    _check(code, "moe_finish")
+
+
+def gemm_tensor_core_grouped(plan, x, out, group_of_block, group_rows, outs, dual_rows=0, slope=1.0, limit=None, offset=0.0,
+                             activation: str | None = None) -> None:  # fmt: skip
+    tensor_core.gemm_grouped(plan, x, out, group_of_block, group_rows, outs, dual_rows, slope, limit, offset,
+                             None if activation is None else PLAIN_ACTIVATIONS[activation])  # fmt: skip
 
 
 GROUP_PAD = 128  # rows of a run of sorted rows (tensor_core.GROUP_PAD)

@@ -62,14 +62,14 @@ def _library():
         lib.me_gemm_tcgen05_swiglu.restype = c_int
         lib.me_gemm_tcgen05_pair_split.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
         lib.me_gemm_tcgen05_pair_split.restype = c_int
-        lib.me_gemm_tcgen05_persistent.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
+        lib.me_gemm_tcgen05_persistent.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]
         lib.me_gemm_tcgen05_persistent.restype = c_int
         lib.me_gemm_tcgen05_persistent_swiglu.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
         lib.me_gemm_tcgen05_persistent_swiglu.restype = c_int
         lib.me_gemm_tcgen05_stacked_swiglu.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
         lib.me_gemm_tcgen05_stacked_swiglu.restype = c_int
         lib.me_gemm_tcgen05_grouped.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int,
-                                                ctypes.c_float, ctypes.c_float, ctypes.c_float, c_void_p]
+                                                ctypes.c_float, ctypes.c_float, ctypes.c_float, c_int, c_void_p]
         lib.me_gemm_tcgen05_grouped.restype = c_int
         lib.me_gemm_wait_probe.argtypes = [c_int, c_void_p, c_void_p]
         lib.me_gemm_wait_probe.restype = c_int
@@ -163,7 +163,7 @@ def gemm(plan: GemmPlan, x: torch.Tensor, out: torch.Tensor, splits: int, group:
     if tokens > PAIR_MIN_TOKENS and splits == 1:
         code = _library().me_gemm_tcgen05_persistent(
             plan.map, _activation_map(x, 128), out.data_ptr(), tokens, plan.rows, plan.inner,
-            PAIR_GROUP_TOKEN_TILES if group is None else group, stream,
+            PAIR_GROUP_TOKEN_TILES if group is None else group, -1, stream,
         )  # fmt: skip
     elif tokens > PAIR_MIN_TOKENS and -(-plan.inner // BLOCK_K) >= PAIR_SPLIT_MIN_K_BLOCKS * splits:
         code = _library().me_gemm_tcgen05_pair_split(
@@ -176,6 +176,24 @@ def gemm(plan: GemmPlan, x: torch.Tensor, out: torch.Tensor, splits: int, group:
     _count_launch()
     if code != 0:
         raise RuntimeError(f"tensor-core product failed to launch (code {code})")
+
+
+def gemm_activated(plan: GemmPlan, x: torch.Tensor, act: torch.Tensor, activation: int) -> None:
+    """``act = a(x @ weight^T)`` in bfloat16 with an activation of :data:`ops.PLAIN_ACTIVATIONS` in the epilogue, for
+    products of more than ``PAIR_MIN_TOKENS`` tokens."""
+    _check_x(plan, x)
+    tokens = x.shape[0]
+    if tokens <= PAIR_MIN_TOKENS:
+        raise RuntimeError(f"the product with a plain activation takes more than {PAIR_MIN_TOKENS} tokens")
+    if act.dtype != torch.bfloat16 or tuple(act.shape) != (tokens, plan.rows) or not act.is_contiguous():
+        raise RuntimeError(f"activation output {tuple(act.shape)} does not fit [{tokens}, {plan.rows}] bfloat16")
+    code = _library().me_gemm_tcgen05_persistent(
+        plan.map, _activation_map(x, 128), act.data_ptr(), tokens, plan.rows, plan.inner, PAIR_GROUP_TOKEN_TILES, activation,
+        _ops_stream(),
+    )  # fmt: skip
+    _count_launch()
+    if code != 0:
+        raise RuntimeError(f"activated tensor-core product failed to launch (code {code})")
 
 
 def gemm_swiglu(
@@ -223,23 +241,25 @@ GROUP_PAD = 128  # rows of a run of the sorted rows that belongs to one group: t
 
 def gemm_grouped(
     plan: GemmPlan, x: torch.Tensor, out: torch.Tensor, group_of_block: torch.Tensor, group_rows: int, outs: int,
-    dual_rows: int = 0, slope: float = 1.0, limit: float | None = None, offset: float = 0.0,
+    dual_rows: int = 0, slope: float = 1.0, limit: float | None = None, offset: float = 0.0, activation: int | None = None,
 ) -> None:  # fmt: skip
     """A product over rows that are sorted by group: the plan's weight holds ``group_rows`` rows per group, run
     ``b`` of ``GROUP_PAD`` rows of ``x`` belongs to group ``group_of_block[b]`` (int32 on the device; negative: no
     rows there).  ``out [rows, outs]`` float32 is ``x[t] . w[group * group_rows + n]``; with ``dual_rows`` it is
     bfloat16 and holds the gated unit of rows ``n`` and ``dual_rows + n`` of the row's group with the constants of
-    :func:`ops.swiglu`."""
+    :func:`ops.swiglu`; with ``activation`` (a number of :data:`ops.PLAIN_ACTIVATIONS`) it is bfloat16 and holds the
+    activated sums."""
     _check_x(plan, x)
     rows = x.shape[0]
-    want = torch.bfloat16 if dual_rows else torch.float32
+    want = torch.bfloat16 if dual_rows or activation is not None else torch.float32
     if out.dtype != want or tuple(out.shape) != (rows, outs) or not out.is_contiguous():
         raise RuntimeError(f"output {tuple(out.shape)} {out.dtype} does not fit [{rows}, {outs}] {want}")
     if rows % GROUP_PAD or group_of_block.dtype != torch.int32 or group_of_block.numel() < rows // GROUP_PAD:
         raise RuntimeError("the rows of a grouped product come in runs of GROUP_PAD with one int32 group each")
     code = _library().me_gemm_tcgen05_grouped(
         plan.map, _activation_map(x, GROUP_PAD), out.data_ptr(), rows, outs, plan.inner, group_of_block.data_ptr(),
-        GROUP_PAD, group_rows, dual_rows, float(slope), float(limit or 0.0), float(offset), _ops_stream(),
+        GROUP_PAD, group_rows, dual_rows, float(slope), float(limit or 0.0), float(offset),
+        -1 if activation is None else activation, _ops_stream(),
     )  # fmt: skip
     _count_launch()
     if code != 0:

@@ -81,6 +81,7 @@ class ModelRunner:
             model.cache_needs(), num_blocks, block_size, max_num_seqs, dtype, self.device,
             max_step_tokens=max_request_tokens or max_num_batched_tokens,
             embedding_state=model.embedding_state(),
+            block_states=model.block_states(),
         )  # fmt: skip
         self.num_groups = len(self.layout.groups)
         self.workspace = Workspace(max_num_batched_tokens, self.device)

@@ -41,6 +41,11 @@ And two for designs that normalise behind the rotation and bound their scores: `
 k head, *after* its rotation, by its root mean square over ``head_dim`` (eps inside the root, no weight), in the
 kernel that adds the biases, rotates and writes the cache; ``score_softcap`` replaces a scaled score ``s`` by ``cap *
 tanh(s / cap)``.  They combine with ``qkv_bias``, ``value_dim``, ``scale``, a partial rotation and either sink.
+
+And one for designs that put positions into the values as well: ``value_encoding`` names a rotation over the whole value
+head.  The value of position ``j`` is cached turned by ``j``; a head's output, the weighted sum of turned values, is turned
+back by the query's position ``i``, so that what leaves the head is the sum of values turned by ``j - i``.  It combines with
+``qkv_bias``, ``o_bias``, ``value_dim``, ``scale``, ``window`` and a partial rotation of q and k.
 """
 
 from __future__ import annotations
@@ -94,6 +99,7 @@ class GroupedQueryAttention(Mixer):
         linear_bias_span: float = 8.0,
         unit_norm_eps: float | None = None,
         score_softcap: float | None = None,
+        value_encoding: PartSpec | None = None,
     ):
         if num_heads % kv_heads:
             raise ValueError(f"num_heads ({num_heads}) must be a multiple of kv_heads ({kv_heads})")
@@ -120,9 +126,9 @@ class GroupedQueryAttention(Mixer):
             raise ValueError(f"score_softcap must be positive, got {score_softcap}")
         # The kernel that adds biases, rotates, then divides by the root mean square: it stands where the other
         # stores would, in front of the attention kernels that know a sink and a cap.
-        self.unit_store = self.unit_norm_eps is not None or bool(self.softcap)
-        if self.unit_store and (qk_norm_eps is not None or head_gate or element_gate or distance_bias or talking_heads or keep_first or reads_shared_cache or o_bias):
-            raise ValueError("unit_norm_eps and score_softcap do not combine with q/k norm weights, gates, distance biases, talking heads, keep_first, an output bias or a shared cache")
+        self.unit_store = self.unit_norm_eps is not None or bool(self.softcap) or value_encoding is not None
+        if self.unit_store and (qk_norm_eps is not None or head_gate or element_gate or distance_bias or talking_heads or keep_first or reads_shared_cache):
+            raise ValueError("unit_norm_eps, score_softcap and value_encoding do not combine with q/k norm weights, gates, distance biases, talking heads, keep_first or a shared cache")
         # Whether q, k, v (and the gates) leave the fused product through the kernel that normalises whole projections.
         self.wide_store = self.wide_norm or self.head_gate or self.element_gate or self.linear_bias
         if (self.head_gate or self.element_gate or self.linear_bias) and qk_norm_eps is not None and not self.wide_norm:
@@ -177,6 +183,9 @@ class GroupedQueryAttention(Mixer):
         self.position = None
         if position_encoding is not None:
             self.position = build_part("position_encoding", position_encoding, prefix, hidden_size)
+        self.value_position = None
+        if value_encoding is not None:
+            self.value_position = build_part("position_encoding", value_encoding, prefix, hidden_size)
         self.r1 = self.r2 = self.talk = None
         self.gates = num_heads if self.head_gate else num_heads * self.value_dim if self.element_gate else 0
         self.slopes: torch.Tensor | None = None
@@ -329,14 +338,19 @@ class GroupedQueryAttention(Mixer):
         return self.out.forward(out, ctx, "attn.o")
 
     def _forward_unit(self, qkv, q, table, slots, ctx: StepContext, cache: LayerCache) -> torch.Tensor:
-        """The step with q and k normalised behind their rotation and (or) capped scores."""
+        """The step with q and k normalised behind their rotation, capped scores, rotated values, or several of these."""
         tokens = q.shape[0]
         if self.position is not None and table is None:
             raise ValueError("these attention options take a rotation that the fused kernel applies, or none")
+        value_table = None
+        if self.value_position is not None:
+            value_table = self.value_position.step_angles(ctx)
+            if value_table is None or value_table.shape[1] * 2 != self.value_dim:
+                raise ValueError("value_encoding takes a rotation over the whole value head")
         ops.qkv_rope_unit_store(
             qkv=qkv, heads=self.heads, kv_heads=self.kv_heads, head_dim=self.head_dim, value_dim=self.value_dim,
             bias=self.bias, cos_sin=table, unit_norm_eps=self.unit_norm_eps, q_out=q, page_size=ctx.page_size,
-            slot_mapping=slots, k_pages=cache.k, v_pages=cache.v,
+            slot_mapping=slots, k_pages=cache.k, v_pages=cache.v, value_cos_sin=value_table,
         )  # fmt: skip
         out = ctx.buffer("attn.out", (tokens, self.heads * self.value_dim), ctx.dtype)
         ops.paged_attention(
@@ -344,6 +358,8 @@ class GroupedQueryAttention(Mixer):
             heads=self.heads, kv_heads=self.kv_heads, head_dim=self.head_dim, scale=self.scale, window=self.window or 0,
             value_dim=self.value_dim, sink=self.sink, sink_values=self.sink_values, softcap=self.softcap,
         )  # fmt: skip
+        if value_table is not None:
+            ops.turn_heads_back(out, value_table, self.heads)
         return self.out.forward(out, ctx, "attn.o")
 
     def _forward_gated(self, qkv, q, table, slots, ctx: StepContext, cache: LayerCache) -> torch.Tensor:

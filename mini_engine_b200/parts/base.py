@@ -86,6 +86,10 @@ class Residual:
     streams, ``(mix [N, N], share [N], mult)``: ``x_t = sum_s mix[s, t] x_s + mult * share[t] * pending``;
     ``stream_read [N]`` are the weights of the sum that the next norm normalises (``None``: all ones, the model's
     end).  The norm applies the update, writes the streams back and reads them in one kernel.
+
+    ``pending_gate`` (partial sums ``[S'', T, hidden]``) with ``pending_gate_bias`` (float32 ``[hidden]``) says that the
+    pending output (with its bias) is first multiplied by ``sigmoid(gate + gate_bias)``, and ``pending_norm = (weight, eps)``
+    that it is then RMS-normed before it is added to ``x`` (a sublayer between two norms).
     """
 
     x: torch.Tensor
@@ -98,6 +102,9 @@ class Residual:
     streams_unwritten: bool = False
     stream_update: tuple | None = None
     stream_read: torch.Tensor | None = None
+    pending_gate: torch.Tensor | None = None
+    pending_gate_bias: torch.Tensor | None = None
+    pending_norm: tuple[torch.Tensor, float] | None = None
 
     def add(self, delta: torch.Tensor, scale: torch.Tensor | None = None, bias: torch.Tensor | None = None) -> None:
         if self.pending is not None:
@@ -115,6 +122,7 @@ class Residual:
     def clear(self) -> None:
         self.pending = self.pending_scale = self.pending_bias = self.pending_more = None
         self.stream_update = self.stream_read = None
+        self.pending_gate = self.pending_gate_bias = self.pending_norm = None
 
 
 @dataclass
@@ -124,7 +132,8 @@ class LayerCache:
     ``k`` and ``v`` are the page arrays of this entry, ``[pages + 1, kv_heads, page_size,
     head_dim]`` (the last page is a spare that no request owns); ``group`` indexes the
     per-group arrays of :class:`StepContext`; ``writes`` is False when the entry reads
-    another entry's cache.  ``state`` is ``[slots + 1, *StateSpec.shape]`` or ``None``.
+    another entry's cache.  ``state`` is ``[slots + 1, *StateSpec.shape]`` or ``None``, ``block_state``
+    the same for the state that the layer's block keeps beside its mixer's.
     """
 
     group: int | None = None
@@ -132,6 +141,7 @@ class LayerCache:
     v: torch.Tensor | None = None
     writes: bool = True
     state: torch.Tensor | None = None
+    block_state: torch.Tensor | None = None
 
 
 @dataclass
@@ -303,6 +313,11 @@ class Block(Part):
     @property
     def feed_forward_norm(self) -> Norm:
         return self.norms["feed_forward"]
+
+    def state(self) -> StateSpec | None:
+        """Per-request state of fixed size that the arrangement itself keeps beside its mixer's (``LayerCache.block_state``,
+        one per execution of the layer), or ``None``."""
+        return None
 
     def parts(self) -> list[Part]:
         whole = [self.mixer, self.feed_forward, *(self.norms[name] for name in self.NORMS)]

@@ -5,7 +5,8 @@ from __future__ import annotations
 import torch
 
 from mini_engine_b200.csrc import ops
-from mini_engine_b200.parts.base import Block, LayerCache, Residual, StepContext, register
+from mini_engine_b200.parts.base import Block, LayerCache, Residual, StateSpec, StepContext, register
+from mini_engine_b200.parts.linear import Linear
 from mini_engine_b200.weights.loader import WeightSpec
 
 
@@ -234,3 +235,76 @@ class ParallelBlock(Block):
         state.add(self.mixer.forward(h, ctx, cache), bias=self.mixer.output_bias)
         if self.feed_forward is not None:
             state.add_beside(self.feed_forward.forward(h, ctx))
+
+
+@register("block", "gated_sandwich")
+class GatedSandwichBlock(Block):
+    """Sublayers between two norms and behind a gate, with a short convolution in front of the mixer::
+
+        h = norm_in(x)        x <- x + norm_out(sigmoid(W_r h + b_r) * sublayer(h'))
+
+    For the mixer ``h'`` is ``h + conv(h)``, a causal convolution over time per channel (``taps`` columns, the last one the
+    current token's, zeros in front of the sequence); for the feed-forward ``h'`` is ``h``.  The gate reads ``h`` in both.
+    The convolution's last ``taps - 1`` inputs are a per-request state of the block.  Gate, bias of the mixer's output
+    projection, the norm behind the sublayer, the residual sum and the next norm are one kernel, in 32-bit."""
+
+    capturable = True
+    adds_output_bias = True
+    NORMS = ("mixer", "mixer_out", "feed_forward", "feed_forward_out")
+
+    def __init__(self, mixer, feed_forward, norms, *, prefix: str, hidden_size: int, gates, conv: str, taps: int, unused_names=()):
+        """``gates``: for ``"mixer"`` (and ``"feed_forward"``) the names of the gate's weight and bias behind the layer's
+        prefix; ``conv``: the convolution's tensor ``[hidden, taps]``.  ``unused_names``: tensors of the layer that a
+        checkpoint may carry although the layer has no use for them."""
+        super().__init__(mixer, feed_forward, norms)
+        wanted = {"mixer"} if feed_forward is None else {"mixer", "feed_forward"}
+        if set(gates) != wanted:
+            raise ValueError(f"gated_sandwich wants the gates' names for {sorted(wanted)}, got {sorted(gates)}")
+        if not 1 <= taps <= ops.MAX_CONV_TAPS:
+            raise ValueError(f"gated_sandwich takes a convolution of 1 to {ops.MAX_CONV_TAPS} taps, got {taps}")
+        self.hidden, self.taps = hidden_size, int(taps)
+        self.gate_names = {sub: tuple(prefix + name for name in pair) for sub, pair in gates.items()}
+        self.conv_name = prefix + conv
+        self.unused = [prefix + name for name in unused_names]
+        self.gates: dict[str, tuple[Linear, torch.Tensor]] = {}
+        self.conv: torch.Tensor | None = None
+
+    def state(self) -> StateSpec | None:
+        return StateSpec((self.taps - 1, self.hidden), torch.float32) if self.taps > 1 else None
+
+    def weight_specs(self) -> list[WeightSpec]:
+        specs = super().weight_specs()
+        for weight, bias in self.gate_names.values():
+            specs.append(WeightSpec(weight, (self.hidden, self.hidden)))
+            specs.append(WeightSpec(bias, (self.hidden,), role="vector", init="small_normal"))
+        specs.append(WeightSpec(self.conv_name, (self.hidden, self.taps), role="vector", init="small_normal"))
+        return specs + [WeightSpec(name, (), role="vector", optional=True) for name in self.unused]
+
+    def load(self, tensors) -> None:
+        super().load(tensors)
+        self.gates = {sub: (Linear(tensors[weight]), tensors[bias]) for sub, (weight, bias) in self.gate_names.items()}
+        self.conv = tensors[self.conv_name].t().contiguous()  # [taps, hidden]: the kernel reads it along the channels
+
+    def _add(self, which: str, state: Residual, gate: torch.Tensor, out: torch.Tensor, bias: torch.Tensor | None = None) -> None:
+        norm = self.norms[which + "_out"]
+        state.add(out, bias=bias)
+        state.pending_gate, state.pending_gate_bias = gate, self.gates[which][1]
+        state.pending_norm = (norm.weight, norm.eps)
+
+    def forward(self, state: Residual, ctx: StepContext, cache: LayerCache) -> None:
+        h = self.norms["mixer"].forward(state, ctx, ctx.dtype)
+        gate = self.gates["mixer"][0].forward(h, ctx, "block.gate")
+        mixed_in = ctx.buffer("block.convolved", tuple(h.shape), h.dtype)
+        ops.input_convolution(h=h, taps=self.conv, ctx=ctx, state=cache.block_state, out=mixed_in)
+        self._add("mixer", state, gate, self.mixer.forward(mixed_in, ctx, cache), self.mixer.output_bias)
+        if self.feed_forward is not None:
+            h = self.norms["feed_forward"].forward(state, ctx, ctx.dtype)
+            gate = self.gates["feed_forward"][0].forward(h, ctx, "block.gate")
+            self._add("feed_forward", state, gate, self.feed_forward.forward(h, ctx))
+
+
+@register("block", "gated_sandwich_mixer_only")
+class GatedSandwichMixerOnlyBlock(GatedSandwichBlock):
+    """The same arrangement for a layer without a feed-forward: two norms, one gate."""
+
+    NORMS = ("mixer", "mixer_out")

@@ -1,0 +1,155 @@
+"""The gated delta rule with a decay per key channel as a mixer part: a matrix state per head that is corrected, not
+only added to.
+
+From the layer's input ``h``: ``q, k`` (``qk_heads`` heads of ``dim``), ``v`` (``heads`` heads of ``vdim``) pass a short causal
+convolution per channel (``taps`` columns, the last one the current token's, zeros in front of the sequence) and silu; q
+and k become unit vectors per head, ``x / sqrt(sum x^2 + unit_eps)``, and q is multiplied by ``query_scale``.  Head ``h``
+uses q/k head ``h // (heads / qk_heads)``.  With ``beta = sigmoid(W_b h)`` (one per head) and ``g = exp(-exp(A_h) *
+softplus(W_a2 (W_a1 h) + dt_bias))`` (one per head and key channel)::
+
+    S <- diag(g) S        u = beta (v - S^T k)        S <- S + k u^T        o = S^T q
+
+Each head's ``o`` is divided by its root mean square over ``vdim``, multiplied by a weight ``[vdim]`` shared by the heads
+and by ``sigmoid(W_g2 (W_g1 h))``, and the concatenated heads are projected by ``W_o``.
+
+A request's state is one float32 row in its slot of the cache manager: the matrix states, head by head with the key
+channels of a value column side by side (``[heads, vdim, dim]``), then the convolution's last ``taps - 1`` inputs.  Decays,
+unit norms, gates of the recurrence and the recurrence are computed in 32-bit from the 32-bit sums of the projections.
+
+Products: all projections of ``h`` run as one product on the row-concatenated weight (q, k, v, both low-rank first
+factors, beta); the two second factors run as one product on a block-diagonal weight.  In bfloat16 the low-rank sums
+enter it as two bfloat16 halves each (the sum rounded, and what rounding left), side by side on the reduction axis against
+the same weight twice, so that the decay is formed from the 32-bit sums up to 2^-16.
+"""
+
+from __future__ import annotations
+
+from typing import Mapping
+
+import torch
+
+from mini_engine_b200.csrc import ops
+from mini_engine_b200.parts.base import LayerCache, Mixer, StateSpec, StepContext, register
+from mini_engine_b200.parts.linear import Linear
+from mini_engine_b200.weights.loader import WeightSpec
+
+
+@register("mixer", "gated_delta_rule")
+class GatedDeltaRule(Mixer):
+    capturable = True
+    # A walk over the tokens is one long kernel per layer, like the scan of the gated linear attention, with which
+    # prompt steps launched as programmatic dependents were seen to stall; this mixer's steps run in plain stream order too.
+    programmatic_launch = False
+
+    def __init__(
+        self,
+        prefix: str,
+        hidden_size: int,
+        *,
+        num_heads: int,
+        qk_heads: int,
+        head_dim: int,
+        value_dim: int,
+        taps: int,
+        decay_rank: int,
+        gate_rank: int,
+        norm_eps: float,
+        unit_eps: float = 1e-6,
+        query_scale: float | None = None,
+        names: Mapping[str, str] | None = None,
+    ):
+        if min(num_heads, qk_heads, head_dim, value_dim, taps, decay_rank, gate_rank) < 1 or num_heads % qk_heads:
+            raise ValueError("gated_delta_rule: sizes must be positive and num_heads a multiple of qk_heads")
+        if head_dim > ops.DELTA_MAX_DIM or taps > ops.MAX_CONV_TAPS:
+            raise ValueError(f"gated_delta_rule takes up to {ops.DELTA_MAX_DIM} key channels per head and {ops.MAX_CONV_TAPS} taps, got {head_dim} and {taps}")
+        self.hidden, self.heads, self.qk_heads, self.dim, self.vdim = hidden_size, num_heads, qk_heads, head_dim, value_dim
+        self.taps, self.ranks = taps, (decay_rank, gate_rank)
+        self.eps, self.unit_eps = float(norm_eps), float(unit_eps)
+        self.q_scale = float(query_scale) if query_scale is not None else head_dim**-0.5
+        defaults = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "q_conv": "q_conv.weight",
+                    "k_conv": "k_conv.weight", "v_conv": "v_conv.weight", "beta": "b_proj.weight", "a_log": "A_log",
+                    "a1": "decay_down.weight", "a2": "decay_up.weight", "dt_bias": "dt_bias", "norm": "norm.weight",
+                    "g1": "gate_down.weight", "g2": "gate_up.weight", "o": "o_proj.weight"}  # fmt: skip
+        self.names = {key: prefix + (names or {}).get(key, value) for key, value in defaults.items()}
+        # Columns of the fused input projection, in this order.
+        widths = {"q": qk_heads * head_dim, "k": qk_heads * head_dim, "v": num_heads * value_dim, "a1": decay_rank,
+                  "g1": gate_rank, "beta": num_heads}  # fmt: skip
+        self.columns, column = {}, 0
+        for key, width in widths.items():
+            self.columns[key] = column
+            column += width
+        self.channels = self.columns["a1"]  # of the convolution: q, k and v
+        self.matrix = num_heads * head_dim * value_dim  # floats of a request's matrix states
+        self.proj: Linear | None = None
+        self.second: Linear | None = None  # both second factors, block-diagonal
+        self.out: Linear | None = None
+        self.conv: torch.Tensor | None = None
+        self.norm_weight = self.a_log = self.dt_bias = None
+
+    def state(self) -> StateSpec:
+        return StateSpec((self.matrix + (self.taps - 1) * self.channels,), torch.float32)
+
+    def weight_specs(self) -> list[WeightSpec]:
+        n, keys, inner, outer = self.names, self.qk_heads * self.dim, self.heads * self.dim, self.heads * self.vdim
+        small = dict(role="vector", init="small_normal")
+        return [
+            WeightSpec(n["q"], (keys, self.hidden)),
+            WeightSpec(n["q_conv"], (keys, self.taps), **small),
+            WeightSpec(n["k"], (keys, self.hidden)),
+            WeightSpec(n["k_conv"], (keys, self.taps), **small),
+            WeightSpec(n["v"], (outer, self.hidden)),
+            WeightSpec(n["v_conv"], (outer, self.taps), **small),
+            WeightSpec(n["beta"], (self.heads, self.hidden)),
+            WeightSpec(n["a_log"], (self.heads,), **small),
+            WeightSpec(n["a1"], (self.ranks[0], self.hidden)),
+            WeightSpec(n["a2"], (inner, self.ranks[0])),
+            WeightSpec(n["dt_bias"], (inner,), **small),
+            WeightSpec(n["norm"], (self.vdim,), role="vector", init="ones_normal"),
+            WeightSpec(n["g1"], (self.ranks[1], self.hidden)),
+            WeightSpec(n["g2"], (outer, self.ranks[1])),
+            WeightSpec(n["o"], (self.hidden, outer)),
+        ]
+
+    def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        n, (decay_rank, gate_rank) = self.names, self.ranks
+        rows = [tensors[n[key]] for key in ("q", "k", "v", "a1", "g1", "beta")]
+        count = sum(r.shape[0] for r in rows)
+        if count % 4:  # rows of zeros: the sums of a token then start on 16 bytes
+            rows.append(torch.zeros(4 - count % 4, self.hidden, dtype=rows[0].dtype, device=rows[0].device))
+        self.proj = Linear(torch.cat(rows, dim=0).contiguous())
+        a2, g2 = tensors[n["a2"]], tensors[n["g2"]]
+        self.halves = 2 if a2.dtype == torch.bfloat16 else 1
+        inner, outer = a2.shape[0], g2.shape[0]
+        second = torch.zeros(inner + outer, self.halves * (decay_rank + gate_rank), dtype=a2.dtype, device=a2.device)
+        for half in range(self.halves):
+            first = half * (decay_rank + gate_rank)
+            second[:inner, first : first + decay_rank] = a2
+            second[inner:, first + decay_rank : first + decay_rank + gate_rank] = g2
+        self.second = Linear(second)
+        self.out = Linear(tensors[n["o"]])
+        self.conv = torch.cat([tensors[n[key]] for key in ("q_conv", "k_conv", "v_conv")], dim=0).t().contiguous()  # [taps, channels]
+        self.norm_weight, self.a_log, self.dt_bias = tensors[n["norm"]], tensors[n["a_log"]], tensors[n["dt_bias"]]
+
+    def forward(self, h: torch.Tensor, ctx: StepContext, cache: LayerCache) -> torch.Tensor:
+        tokens, heads, dim, vdim = h.shape[0], self.heads, self.dim, self.vdim
+        proj = self.proj.forward(h, ctx, "delta.proj")
+        low = ctx.buffer("delta.low", (tokens, self.halves * sum(self.ranks)), h.dtype)
+        ops.split_halves(proj, self.columns["a1"], sum(self.ranks), low)
+        second = self.second.forward(low, ctx, "delta.second")  # [decay logits | gate logits]
+        qk = ctx.buffer("delta.qk", (tokens, self.qk_heads * 2 * dim), torch.float32)
+        gv = ctx.buffer("delta.gv", (tokens, heads * (dim + vdim)), torch.float32)
+        scalars = ctx.buffer("delta.scalars", (tokens, heads * 2), torch.float32)
+        sizes = dict(heads=heads, qk_heads=self.qk_heads, dim=dim, vdim=vdim)
+        ops.delta_prepare(
+            proj=proj, columns=self.columns, second=second, conv=self.conv, a_log=self.a_log, dt_bias=self.dt_bias, ctx=ctx,
+            state=cache.state, matrix=self.matrix, qk=qk, gv=gv, scalars=scalars, q_scale=self.q_scale, unit_eps=self.unit_eps,
+            **sizes,
+        )  # fmt: skip
+        raw = ctx.buffer("delta.raw", (tokens, heads * vdim), torch.float32)
+        ops.delta_scan(qk=qk, gv=gv, scalars=scalars, ctx=ctx, state=cache.state, out=raw, **sizes)
+        gated = ctx.buffer("delta.out", (tokens, heads * vdim), ctx.dtype)
+        ops.gla_finish(
+            o=raw, proj=second, gate_column=heads * dim, weight=self.norm_weight, eps=self.eps, out=gated, heads=heads,
+            vdim=vdim, gate="sigmoid",
+        )  # fmt: skip
+        return self.out.forward(gated, ctx, "delta.o")

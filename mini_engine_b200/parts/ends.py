@@ -30,20 +30,36 @@ from mini_engine_b200.weights.loader import WeightSpec
 class TokenEmbedding(Embedding):
     capturable = True
 
-    def __init__(self, vocab_size: int, hidden_size: int, *, weight: str, multiplier: float | None = None):
+    def __init__(
+        self, vocab_size: int, hidden_size: int, *, weight: str, multiplier: float | None = None, norm: str | None = None,
+        norm_eps: float = 0.0,
+    ):  # fmt: skip
+        """``norm``: the weight of an RMS norm (``norm_eps`` inside the root) that the rows pass before they become the
+        residual stream, in 32-bit; by default there is none."""
         self.vocab, self.hidden = vocab_size, hidden_size
-        self.weight_name = weight
+        self.weight_name, self.norm_name, self.norm_eps = weight, norm, float(norm_eps)
         self.multiplier = 1.0 if multiplier is None else float(multiplier)
         self.table: torch.Tensor | None = None
+        self.norm_weight: torch.Tensor | None = None
 
     def weight_specs(self) -> list[WeightSpec]:
-        return [WeightSpec(self.weight_name, (self.vocab, self.hidden))]
+        specs = [WeightSpec(self.weight_name, (self.vocab, self.hidden))]
+        if self.norm_name is not None:
+            specs.append(WeightSpec(self.norm_name, (self.hidden,), role="vector", init="ones_normal"))
+        return specs
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         self.table = tensors[self.weight_name]
+        if self.norm_name is not None:
+            self.norm_weight = tensors[self.norm_name]
 
-    def forward(self, token_ids: torch.Tensor, ctx: StepContext, out: torch.Tensor) -> None:
+    def forward(self, token_ids: torch.Tensor, ctx: StepContext, out: torch.Tensor) -> torch.Tensor | None:
         ops.embedding(self.table, token_ids, out, self.multiplier)
+        if self.norm_weight is None:
+            return None
+        rounded = ctx.buffer("embedding.rounded", tuple(out.shape), ctx.dtype)
+        ops.add_rmsnorm(out, None, self.norm_weight, self.norm_eps, rounded, keep_normed=True)
+        return rounded
 
 
 @register("embedding", "pair_hash_embedding")

@@ -38,6 +38,9 @@ GATED_FUSED_MIN_TOKENS = 4
 # is faster (intermediate size 3,072: a decode step of 28 layers takes 1.11 ms that way against
 # 1.15 ms at batch 8, 2.07 against 2.13 ms at batch 32; at 12,288 features the stacked kernel wins).
 GATED_STACKED_MIN_FEATURES = 128 * 64
+# A product with a plain activation carries it in its epilogue from this many tokens on: the steps whose products are not
+# split (a split product's sums meet in the activation kernel instead).
+ACTIVATED_FUSED_MIN_TOKENS = 1025
 
 
 def partial_rows(max_tokens: int) -> int:
@@ -105,4 +108,22 @@ class GatedLinear:
             return act
         both = self.linear.forward(x, ctx, name + ".gate_up")
         ops.swiglu(both, act, self.slope, self.limit, self.offset, activation=self.activation)
+        return act
+
+
+class ActivatedLinear:
+    """``act(x W^T)`` in the compute dtype with an activation of :data:`ops.PLAIN_ACTIVATIONS`: from ``ACTIVATED_FUSED_MIN_TOKENS``
+    tokens on in the tensor-core product's epilogue, below as a kernel on the product's partial sums."""
+
+    def __init__(self, weight: torch.Tensor, activation: str):
+        self.linear, self.activation = Linear(weight), activation
+        self.out_features = weight.shape[0]
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, name: str) -> torch.Tensor:
+        """``x [T, in]`` -> activated ``[T, out]`` in the compute dtype."""
+        act = ctx.buffer(name + ".act", (x.shape[0], self.out_features), x.dtype)
+        if self.linear.tensor_core and x.shape[0] >= ACTIVATED_FUSED_MIN_TOKENS:
+            ops.gemm_tensor_core_activated(self.linear.plan, x, act, self.activation)
+        else:
+            ops.activation(self.linear.forward(x, ctx, name + ".up"), act, self.activation)
         return act

@@ -24,6 +24,11 @@ kernel with the gated form; a kernel of its own rotates, scales and lays q, k an
 of more than ``CHUNKED_MIN_TOKENS`` tokens do not walk token by token: a constant decay gives the recurrence over a chunk
 of 64 tokens a closed form (the state in front of the chunk, decayed, plus a causal product inside the chunk), which
 three kernels compute with all chunks side by side, in float32.
+
+Options of ``retention``: ``qkv_activation="silu"`` activates the projections of q, k and v; ``key_scale=1`` leaves the keys
+as they are; ``norm_weight`` multiplies the normed output by a weight (``norm``); ``norm_scope="projection"`` takes the root
+mean square over all heads of a token together (a weight of that size) in the place of one per head;
+``gate_activation="sigmoid"`` gates by ``sigmoid(W_g h)``.  Together they are lightning attention.
 """
 
 from __future__ import annotations
@@ -145,14 +150,26 @@ class Retention(Mixer):
         norm_eps: float,
         position_encoding: PartSpec | None = None,
         key_scale: float | None = None,
+        qkv_activation: str | None = None,
+        norm_scope: str = "head",
+        norm_weight: bool = False,
+        gate_activation: str = "silu",
         names: Mapping[str, str] | None = None,
     ):
         """``decay``: one constant per head, ``0 < a_h <= 1``; ``key_scale``: what rotated keys are multiplied by
-        (default ``head_dim ** -0.5``); ``position_encoding``: a rotate-half rotation that the kernel applies, or none."""
+        (default ``head_dim ** -0.5``); ``position_encoding``: a rotate-half rotation that the kernel applies, or none.  The
+        other options are described at the module's top."""
         if min(num_heads, head_dim, value_dim) < 1:
             raise ValueError("retention: sizes must be positive")
-        if head_dim > 192:
-            raise ValueError(f"retention: the walking kernel keeps a state column of at most 192 key channels in registers, got {head_dim}")
+        if head_dim > ops.RETENTION_MAX_DIM:
+            raise ValueError(f"retention: the walking kernel takes at most {ops.RETENTION_MAX_DIM} key channels per head, got {head_dim}")
+        if qkv_activation not in (None, "silu") or norm_scope not in ("head", "projection") or gate_activation not in ops.FINISH_GATES:
+            raise ValueError("retention: qkv_activation is None or 'silu', norm_scope 'head' or 'projection', gate_activation 'silu' or 'sigmoid'")
+        if qkv_activation is not None and position_encoding is not None:
+            raise ValueError("retention activates its projections or rotates them, not both")
+        self.silu, self.norm_scope, self.gate_kind = qkv_activation == "silu", norm_scope, gate_activation
+        self.norm_len = 0 if not norm_weight else value_dim if norm_scope == "head" else num_heads * value_dim
+        self.norm_weight: torch.Tensor | None = None
         if len(decay) != num_heads or not all(0.0 < float(a) <= 1.0 for a in decay):
             raise ValueError(f"retention: one decay in (0, 1] per head ({num_heads}), got {list(decay)}")
         self.hidden, self.heads, self.dim, self.vdim = hidden_size, num_heads, head_dim, value_dim
@@ -161,7 +178,8 @@ class Retention(Mixer):
         self.position = None
         if position_encoding is not None:
             self.position = build_part("position_encoding", position_encoding, prefix, hidden_size)
-        defaults = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "g": "g_proj.weight", "o": "o_proj.weight"}
+        defaults = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "g": "g_proj.weight", "o": "o_proj.weight",
+                    "norm": "norm.weight"}  # fmt: skip
         self.names = {key: prefix + (names or {}).get(key, value) for key, value in defaults.items()}
         widths = {"q": num_heads * head_dim, "k": num_heads * head_dim, "v": num_heads * value_dim, "g": num_heads * value_dim}
         self.columns, column = {}, 0
@@ -185,10 +203,14 @@ class Retention(Mixer):
             WeightSpec(n["g"], (outer, self.hidden)),
             WeightSpec(n["o"], (self.hidden, outer)),
         ]
+        if self.norm_len:
+            specs.append(WeightSpec(n["norm"], (self.norm_len,), role="vector", init="ones_normal"))
         return specs + (self.position.weight_specs() if self.position is not None else [])
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         n = self.names
+        if self.norm_len:
+            self.norm_weight = tensors[n["norm"]]
         self.proj = Linear(torch.cat([tensors[n[key]] for key in ("q", "k", "v", "g")], dim=0).contiguous())
         self.out = Linear(tensors[n["o"]])
         # a decay enters the recurrence: the float32 nearest to the configuration's number, made from the double
@@ -214,11 +236,11 @@ class Retention(Mixer):
         ops.retention_scan(
             proj=proj, columns=self.columns, cos_sin=table, decay=self.decay, k_scale=self.k_scale, ctx=ctx,
             state=cache.state, out=raw, prepared=prepared, heads=self.heads, dim=self.dim, vdim=self.vdim,
-            chunk_min=chunk_min, chunk_state=chunk_state,
+            chunk_min=chunk_min, chunk_state=chunk_state, silu=self.silu,
         )  # fmt: skip
         gated = ctx.buffer("retention.out", (tokens, self.heads * self.vdim), ctx.dtype)
         ops.gla_finish(
-            o=raw, proj=proj, gate_column=self.columns["g"], weight=None, eps=self.eps, out=gated, heads=self.heads,
-            vdim=self.vdim,
+            o=raw, proj=proj, gate_column=self.columns["g"], weight=self.norm_weight, eps=self.eps, out=gated, heads=self.heads,
+            vdim=self.vdim, gate=self.gate_kind, scope=self.norm_scope,
         )  # fmt: skip
         return self.out.forward(gated, ctx, "retention.o")

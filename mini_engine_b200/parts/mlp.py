@@ -11,7 +11,8 @@ The gate has three constants for models whose gated unit differs: ``y = g * sigm
 ``0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3)))`` in the place of ``g * sigmoid(gate_slope * g)``.
 
 ``mlp`` is the feed-forward without a gate, ``y = act(x Wu^T) Wd^T`` with ``act`` the square of relu (``relu_squared``),
-``relu``, ``silu`` or ``gelu_tanh``: the up product's partial sums meet in the activation kernel, which rounds once.
+``relu``, ``silu``, ``gelu_tanh`` or ``gelu_erf`` (``0.5 z (1 + erf(z / sqrt 2))``): the up product's partial sums meet in the
+activation kernel, which rounds once; a long prompt's product is not split and applies it in its epilogue.
 """
 
 from __future__ import annotations
@@ -22,7 +23,7 @@ import torch
 
 from mini_engine_b200.csrc import ops
 from mini_engine_b200.parts.base import FeedForward, StepContext, register
-from mini_engine_b200.parts.linear import GatedLinear, Linear
+from mini_engine_b200.parts.linear import ActivatedLinear, GatedLinear, Linear
 from mini_engine_b200.weights.loader import WeightSpec
 
 
@@ -90,7 +91,7 @@ class PlainMLP(FeedForward):
         self.hidden, self.inter, self.activation = hidden_size, intermediate_size, activation
         defaults = {"up": "up_proj.weight", "down": "down_proj.weight"}
         self.names = {key: prefix + (names or {}).get(key, value) for key, value in defaults.items()}
-        self.up: Linear | None = None
+        self.up: ActivatedLinear | None = None
         self.down: Linear | None = None
 
     def weight_specs(self) -> list[WeightSpec]:
@@ -100,10 +101,8 @@ class PlainMLP(FeedForward):
         ]
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
-        self.up, self.down = Linear(tensors[self.names["up"]]), Linear(tensors[self.names["down"]])
+        self.up, self.down = ActivatedLinear(tensors[self.names["up"]], self.activation), Linear(tensors[self.names["down"]])
 
     def forward(self, h: torch.Tensor, ctx: StepContext) -> torch.Tensor:
-        sums = self.up.forward(h, ctx, "mlp.up")
-        act = ctx.buffer("mlp.plain_act", (h.shape[0], self.inter), h.dtype)
-        ops.activation(sums, act, self.activation)
+        act = self.up.forward(h, ctx, "mlp.plain")
         return self.down.forward(act, ctx, "mlp.plain_down")

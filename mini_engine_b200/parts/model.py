@@ -28,7 +28,7 @@ from mini_engine_b200.parts.base import (
 from mini_engine_b200.weights.loader import WeightSpec
 
 # Importing the built-in parts registers them.
-from mini_engine_b200.parts import attention, block, ends, latent_attention, linear_attention, mlp, moe, norms, parallel, recurrent, rotary  # noqa: F401,E402
+from mini_engine_b200.parts import attention, block, delta_rule, ends, latent_attention, linear_attention, mlp, moe, norms, parallel, recurrent, rotary  # noqa: F401,E402
 
 
 def build_block(spec: ModelSpec, index: int) -> Block:
@@ -94,6 +94,10 @@ class DecoderModel:
             mixer = self.blocks[entry.layer].mixer
             needs.append((mixer.paged_cache(), mixer.state(), entry.cache_of))
         return needs
+
+    def block_states(self) -> list[StateSpec | None]:
+        """For every entry of the execution order, the per-request state that the layer's block keeps."""
+        return [self.blocks[entry.layer].state() for entry in self.spec.order]
 
     def embedding_state(self) -> StateSpec | None:
         """The per-request state that the embedding part keeps, if any."""

@@ -49,12 +49,14 @@ class RMSNorm(Norm):
     def forward(
         self, state: Residual, ctx: StepContext, out_dtype, rows=None, residual_scale: float = 1.0, keep_normed: bool = False
     ) -> torch.Tensor:
-        if state.pending_bias is not None or state.pending_more is not None:
+        if state.pending_more is not None or (state.pending_bias is not None and state.pending_norm is None):
             raise ValueError("rmsnorm adds one pending output without a bias")
         count = state.x.shape[0] if rows is None else rows.shape[0]
         out = ctx.buffer("norm.out" if rows is None else "norm.rows", (count, self.dim), out_dtype)
         if state.streams is not None:
             return self._forward_streams(state, out, rows, residual_scale, keep_normed)
+        if state.pending_norm is not None:
+            return self._forward_sandwich(state, out, rows, residual_scale, keep_normed)
         ops.add_rmsnorm(
             state.x, state.pending, self.weight, self.eps, out, rows, state.pending_scale, residual_scale, keep_normed
         )
@@ -63,6 +65,19 @@ class RMSNorm(Norm):
             state.rounded = out if keep_normed else None  # with keep_normed, `out` is the new stream, rounded
         return out
 
+    def _forward_sandwich(self, state: Residual, out, rows, residual_scale, keep_normed) -> torch.Tensor:
+        """A pending output that is gated and normed before it is added (see :class:`~mini_engine_b200.parts.base.Residual`)."""
+        if residual_scale != 1.0 or keep_normed or state.pending_scale is not None:
+            raise ValueError("rmsnorm behind a gated and normed output: no factor, no scale, no write-back")
+        weight, eps = state.pending_norm
+        ops.sandwich_norm(
+            x=state.x, pending=state.pending, bias=state.pending_bias, gate=state.pending_gate, gate_bias=state.pending_gate_bias,
+            out_weight=weight, out_eps=eps, weight=self.weight, eps=self.eps, out=out, rows=rows,
+        )  # fmt: skip
+        if rows is None:
+            state.clear()
+            state.rounded = None
+        return out
 
     def _forward_streams(self, state: Residual, out, rows, residual_scale, keep_normed) -> torch.Tensor:
         """Several residual streams: the pending output's update of all streams, their weighted sum and its norm are
@@ -109,7 +124,7 @@ class LayerNorm(Norm):
     def forward(
         self, state: Residual, ctx: StepContext, out_dtype, rows=None, residual_scale: float = 1.0, keep_normed: bool = False
     ) -> torch.Tensor:
-        if residual_scale != 1.0 or keep_normed or state.pending_scale is not None:
+        if residual_scale != 1.0 or keep_normed or state.pending_scale is not None or state.pending_norm is not None:
             raise ValueError("layernorm stands in front of its sublayers: no factor on the stream, no scale, no write-back")
         count = state.x.shape[0] if rows is None else rows.shape[0]
         out = ctx.buffer("norm.out" if rows is None else "norm.rows", (count, self.dim), out_dtype)
