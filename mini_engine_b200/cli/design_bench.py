@@ -1,7 +1,7 @@
-"""Prefill and decode throughput of another design (Pimezen, Molotar, Bevadra, Bizurax) beside Qwen3 dense at equal layer sizes.
+"""Prefill and decode throughput of another design (Pimezen, Molotar, Bevadra, Bizurax, Tobadra) beside Qwen3 dense at equal layer sizes.
 
-    python -m mini_engine_b200.cli.design_bench [--design pimezen|molotar|bevadra|bizurax] [--sizes 1b,8b] [--steps K] [--warmup W]
-    (or: bench.py --design pimezen|molotar|bevadra|bizurax)
+    python -m mini_engine_b200.cli.design_bench [--design pimezen|molotar|bevadra|bizurax|tobadra] [--sizes 1b,8b] [--steps K] [--warmup W]
+    (or: bench.py --design pimezen|molotar|bevadra|bizurax|tobadra)
     python -m mini_engine_b200.cli.design_bench --design bevadra --sizes 8b --capture prompt|decode   (a few eager steps, for a profiler)
 
 For each size both models get the same width, feed-forward width, head counts, head size, layer count
@@ -30,6 +30,15 @@ many heads with the key and value widths of Pimezen's linear attention; its late
 query/key elements, values of 128 and a latent of 512; the attention layers have a squared-relu feed-forward one and a
 half times as wide as Qwen3's (the same weights), the retention layers 8 routed units a quarter as wide of which a token
 uses 2, beside a shared unit half as wide (a token uses as many feed-forward weights as in Qwen3).
+
+Tobadra gets four layers in the order attention, lightning attention, delta rule, attention; its attention has Qwen3's head
+counts and head size, a window of 1,024 tokens and half of each head rotated (the values over their whole width); lightning
+attention and the delta rule have as many heads with the key and value widths of Pimezen's linear attention, the delta
+rule a convolution of four taps and low ranks of 64; the convolution in front of the mixers has four taps; the attention
+layers have a tanh-GELU feed-forward one and a half times as wide as Qwen3's (the same weights), the two others 8 routed
+units three eighths as wide beside 2 units that return their input, in 2 groups of which 1 is kept, of which a token uses
+2, beside a gated shared unit three quarters as wide (a token whose units both have tensors uses as many feed-forward
+weights as in Qwen3).  Every sublayer has a gate of width x width beside these.
 """
 
 from __future__ import annotations
@@ -53,11 +62,13 @@ TIMED = ("biased_attention", "mixed_attention", "gla_scan", "gla_finish", "branc
          "add_rmsnorm", "swiglu", "gemm_tensor_core", "gemm_tensor_core_swiglu", "embedding", "rglru", "route",
          "qk_wide_norm_rope_store", "pair_embedding", "round_rows", "gemm_tensor_core_grouped", "sort_by_unit", "gather_rows",
          "combine_rows", "add_layernorm", "latent_down_finish", "head_product", "logits_finish", "retention_scan", "hyper_step",
-         "activation", "qkv_rope_unit_store")  # fmt: skip
+         "activation", "qkv_rope_unit_store", "sandwich_norm", "input_convolution", "turn_heads_back", "split_halves",
+         "delta_prepare", "delta_scan", "moe_finish", "gemm_tensor_core_activated")  # fmt: skip
 STREAMS, ROUTED_UNITS, ROUTED_USED = 4, 8, 2
 LATENT_RANK, LATENT_ROT = 512, 64
 UNITS, UNITS_USED, UNIT_GROUPS, UNIT_GROUPS_KEPT = 8, 2, 4, 2
 RECURRENCE_BLOCK, RECURRENCE_TAPS = 128, 4
+TAPS, PASSED_UNITS = 4, 2
 
 
 def molotar_config(size: dict):
@@ -111,6 +122,23 @@ def bizurax_config(size: dict):
                                     "residual_mult": 0.5, "streams": STREAMS, "layers": layers})  # fmt: skip
 
 
+def tobadra_config(size: dict):
+    from mini_engine_b200.config import TobadraConfig
+
+    d, h, ff, ld, lv = size["head_dim"], size["heads"], size["ff"], size["lin_dim"], size["lin_vdim"]
+    attention = {"heads": h, "kv_heads": size["kv_heads"], "dim": d, "vdim": d, "scale": d**-0.5, "mask": {"size": WINDOW},
+                 "rot": {"base": 1e5, "dims": d // 2}}  # fmt: skip
+    lightning = {"heads": h, "dim": ld, "vdim": lv, "decay": [1.0 - 2.0 ** (-5 - 6 * i / h) for i in range(h)]}
+    delta = {"heads": h, "kv_heads": h, "dim": ld, "vdim": lv, "conv": TAPS, "decay_rank": size["rank"], "gate_rank": size["rank"]}
+    dense = {"kind": "dense", "ff": 3 * ff // 2}
+    routed = {"kind": "moe", "expert": {"ff": 3 * ff // 8}, "shared": {"ff": 3 * ff // 4},
+              "router": {"experts": ROUTED_UNITS, "identity": PASSED_UNITS, "top": ROUTED_USED, "scale": 2.0, "groups": {"count": 2, "keep": 1}}}  # fmt: skip
+    pattern = [("attention", attention, dense), ("lightning", lightning, routed), ("channel_delta", delta, routed), ("attention", attention, dense)]
+    layers = [{"type": kind, "mixer": mixer, "mlp": mlp} for kind, mixer, mlp in (pattern * size["layers"])[: size["layers"]]]
+    return TobadraConfig.from_dict({"architecture": "Tobadra", "vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-6},
+                                    "canon": {"taps": TAPS}, "logit_scale": 0.25, "layers": layers})  # fmt: skip
+
+
 def configs(size: dict, design: str = "pimezen"):
     from mini_engine_b200.config import PimezenConfig, Qwen3Config
 
@@ -137,6 +165,8 @@ def configs(size: dict, design: str = "pimezen"):
         return {"bevadra": bevadra_config(size), "qwen3": qwen}
     if design == "bizurax":
         return {"bizurax": bizurax_config(size), "qwen3": qwen}
+    if design == "tobadra":
+        return {"tobadra": tobadra_config(size), "qwen3": qwen}
     return {"pimezen": pimezen, "qwen3": qwen}
 
 
@@ -202,7 +232,7 @@ def rooflines(design: str, size: dict, peaks: dict) -> dict:
     def bound(name, nbytes, nflops):
         out[name] = {"bytes": nbytes, "flops": nflops, "roofline_us": max(nbytes / bw, nflops / flops) * 1e6}
 
-    window = WINDOW if design in ("pimezen", "molotar", "bevadra") else None
+    window = WINDOW if design in ("pimezen", "molotar", "bevadra", "tobadra") else None
     keep = KEEP_FIRST if design == "pimezen" else 0
     seen_prompt = visible_sum(0, PROMPT, window, keep)
     seen_decode = BATCH * visible_sum(CONTEXT, CONTEXT + 1, window, keep)
@@ -287,6 +317,39 @@ def rooflines(design: str, size: dict, peaks: dict) -> dict:
                                         "kernels": ("gemm_tensor_core", "gemm_tensor_core_grouped", "gemm_tensor_core_swiglu", "swiglu", "activation")}  # fmt: skip
         # kernel times are averaged over all layers: a quarter have an attention, a quarter a latent attention, half a retention
         share = {"paged_attention": 0.25, "latent_attention": 0.25, "head_product": 0.25, "retention_scan": 0.5}
+        for name in [n for n in out if n.split(".")[1] in share]:
+            factor = share[name.split(".")[1]]
+            nbytes, nflops = out[name]["bytes"] * factor, out[name]["flops"] * factor
+            out[name] = {"bytes": nbytes, "flops": nflops, "roofline_us": max(nbytes / bw, nflops / flops) * 1e6}
+    elif design == "tobadra":
+        ld, lv, rank = size["lin_dim"], size["lin_vdim"], size["rank"]
+        state, row = h * ld * lv * 4, (2 * h * ld + h * lv) * 4  # a request's state; a token's q, k and v sums (32-bit)
+        prepared = h * (3 * ld + lv + 2) * 4  # what the delta rule's walk reads of a token
+        for phase, tokens in (("prompt", PROMPT), ("decode", BATCH)):
+            per_request = 1 if phase == "prompt" else BATCH
+            bound(f"{phase}.retention_scan", tokens * (row + 2 * 3 * h * ld * 4 + h * lv * 4) + per_request * 2 * state, tokens * h * ld * lv * 4)
+            past = 0 if phase == "prompt" else BATCH * 2 * (TAPS - 1) * row
+            bound(f"{phase}.delta_prepare", tokens * (row + h * ld * 4 + prepared) + past, 0)
+            bound(f"{phase}.delta_scan", tokens * (prepared + h * lv * 4) + per_request * 2 * state, tokens * h * ld * lv * 7)
+            # two of each per layer: output and gate in, the stream in and out, the next input out; one convolution
+            bound(f"{phase}.sandwich_norm", 2 * tokens * width * (4 + 4 + 8 + 2), 0)
+            bound(f"{phase}.input_convolution", tokens * width * 4 + (0 if phase == "prompt" else BATCH * 2 * (TAPS - 1) * width * 4), 0)
+            bound(f"{phase}.turn_heads_back", tokens * h * d * 4, 0)
+        linear = width * (2 * h * ld + 2 * h * lv) + h * lv * width
+        delta = width * (2 * h * ld + h * lv + 2 * rank + h) + rank * h * (ld + lv) + h * lv * width
+        attention = width * (h * d + 2 * g * d) + h * d * width
+        mixer = (2 * attention + linear + delta) / 4 + 2 * width * width  # and the two gates
+        unit, shared, dense = 2 * width * (3 * ff // 8), 2 * width * (3 * ff // 4), 2 * width * (3 * ff // 2)
+        chosen = ROUTED_USED * ROUTED_UNITS / (ROUTED_UNITS + PASSED_UNITS)  # units with tensors that a token uses, on average
+        used = 0.5 * dense + 0.5 * (chosen * unit + shared)
+        touched = 0.5 * dense + 0.5 * (ROUTED_UNITS * (1.0 - (1.0 - chosen / ROUTED_UNITS) ** BATCH) * unit + shared)
+        held = 0.5 * dense + 0.5 * (ROUTED_UNITS * unit + shared)
+        for phase, tokens, nbytes in (("prompt", PROMPT, (mixer + held) * 2), ("decode", BATCH, (mixer + touched) * 2)):
+            nflops = 2 * tokens * (mixer + used)
+            out[f"{phase}.products"] = {"bytes": nbytes, "flops": nflops, "roofline_us": max(nbytes / bw, nflops / flops) * 1e6,
+                                        "kernels": ("gemm_tensor_core", "gemm_tensor_core_grouped", "gemm_tensor_core_activated", "activation")}  # fmt: skip
+        # kernel times are averaged over all layers: half have an attention, a quarter lightning attention, a quarter the delta rule
+        share = {"paged_attention": 0.5, "turn_heads_back": 0.5, "retention_scan": 0.25, "delta_prepare": 0.25, "delta_scan": 0.25}
         for name in [n for n in out if n.split(".")[1] in share]:
             factor = share[name.split(".")[1]]
             nbytes, nflops = out[name]["bytes"] * factor, out[name]["flops"] * factor
@@ -468,7 +531,7 @@ def capture_steps(design: str, size_name: str, phase: str) -> None:
 
 def main(argv=None) -> int:
     parser = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
-    parser.add_argument("--design", choices=["pimezen", "molotar", "bevadra", "bizurax"], default="pimezen")
+    parser.add_argument("--design", choices=["pimezen", "molotar", "bevadra", "bizurax", "tobadra"], default="pimezen")
     parser.add_argument("--sizes", default="1b,8b")
     parser.add_argument("--steps", type=int, default=32)
     parser.add_argument("--warmup", type=int, default=5)

@@ -1403,6 +1403,72 @@ __global__ void __launch_bounds__(UNIT_WARPS * 32) qkv_rope_unit_store_kernel(Un
     }
 }
 
+// The same row without a unit norm: a pair of rotated elements stands alone, so a thread takes four pairs of a rotated part (two
+// 16-byte loads, half a rotation apart) or four elements of a part that passes through, of one token (grid: runs of 256
+// such units x tokens).  Every head, rotated part and half of one is a multiple of four elements wide, every pointer
+// 16-byte aligned, at most MAX_UNROLLED_SPLITS sums.
+template <typename OutT, int SPLITS>
+__global__ void __launch_bounds__(256) qkv_rope_vec_store_kernel(UnitQkvArgs a) {
+    const int token = blockIdx.y;
+    int unit = blockIdx.x * 256 + threadIdx.x;
+    pdl_trigger();
+    pdl_wait();
+    const int rotary = a.cos_sin ? a.rotary_dim : 0, value_rotary = a.value_cos_sin ? a.value_dim : 0;
+    const int per_key = rotary / 8 + (a.head_dim - rotary) / 4, per_value = value_rotary / 8 + (a.value_dim - value_rotary) / 4;
+    const int key_units = (a.heads + a.kv_heads) * per_key;
+    if (unit >= key_units + a.kv_heads * per_value) return;
+    const bool is_value = unit >= key_units;
+    if (is_value) unit -= key_units;
+    const int per = is_value ? per_value : per_key, turned = is_value ? value_rotary : rotary, d = is_value ? a.value_dim : a.head_dim;
+    const int which = unit / per, place = unit % per;
+    const bool pair = place < turned / 8;
+    const int e = pair ? 4 * place : turned + 4 * (place - turned / 8), half = turned / 2;
+    const int column = (is_value ? (a.heads + a.kv_heads) * a.head_dim : 0) + which * d + e;
+    const float* src = a.qkv + static_cast<size_t>(token) * a.row_width + column;
+    float4 low[SPLITS], high[SPLITS];
+#pragma unroll
+    for (int s = 0; s < SPLITS; ++s) {
+        if (s >= a.splits) continue;
+        low[s] = *reinterpret_cast<const float4*>(src + s * a.split_stride);
+        if (pair) high[s] = *reinterpret_cast<const float4*>(src + s * a.split_stride + half);
+    }
+    float4 u = make_float4(0.0f, 0.0f, 0.0f, 0.0f), v = u;
+#pragma unroll
+    for (int s = 0; s < SPLITS; ++s) {
+        if (s >= a.splits) continue;
+        add4(u, low[s]);
+        if (pair) add4(v, high[s]);
+    }
+    if (a.bias) {
+        add4(u, *reinterpret_cast<const float4*>(a.bias + column));
+        if (pair) add4(v, *reinterpret_cast<const float4*>(a.bias + column + half));
+    }
+    if (pair) {
+        const float2* angles = (is_value ? a.value_cos_sin : a.cos_sin) + static_cast<size_t>(token) * half + e;
+        const float4 first = *reinterpret_cast<const float4*>(angles), second = *reinterpret_cast<const float4*>(angles + 2);
+        const float4 x = u;
+        u = make_float4(x.x * first.x - v.x * first.y, x.y * first.z - v.y * first.w, x.z * second.x - v.z * second.y, x.w * second.z - v.w * second.w);
+        v = make_float4(v.x * first.x + x.x * first.y, v.y * first.z + x.y * first.w, v.z * second.x + x.z * second.y, v.w * second.z + x.w * second.w);
+    }
+    OutT* dst;
+    const int q_width = a.heads * a.head_dim;
+    if (!is_value && which < a.heads) {
+        dst = static_cast<OutT*>(a.q_out) + static_cast<size_t>(token) * q_width + column;
+    } else {
+        const int head = is_value ? which : which - a.heads;
+        if (a.slot_mapping) {
+            const int slot = a.slot_mapping[token];
+            if (slot < 0) return;
+            const size_t page = slot / a.page_size, offset = slot % a.page_size;
+            dst = static_cast<OutT*>(is_value ? a.v_pages : a.k_pages) + ((page * a.kv_heads + head) * a.page_size + offset) * d + e;
+        } else {
+            dst = static_cast<OutT*>(is_value ? a.v_dense : a.k_dense) + static_cast<size_t>(token) * a.kv_heads * d + head * d + e;
+        }
+    }
+    store4(dst, u);
+    if (pair) store4(dst + half, v);
+}
+
 ME_EXPORT int me_qkv_rope_unit_store(const float* qkv, int splits, long long split_stride, int row_width,
                                      const float* bias, const float* cos_sin, const int* slot_mapping, void* q_out,
                                      void* k_pages, void* v_pages, void* k_dense, void* v_dense, float eps, int out_type,
@@ -1417,6 +1483,21 @@ ME_EXPORT int me_qkv_rope_unit_store(const float* qkv, int splits, long long spl
                   q_out, k_pages, v_pages, k_dense, v_dense, eps, tokens, heads, kv_heads, head_dim, value_dim, page_size,
                   rotary_dim, unit_norm, reinterpret_cast<const float2*>(value_cos_sin)};
     if (value_cos_sin != nullptr && value_dim % 2) return ME_ERR_ARGUMENT;
+    // Which kernel runs follows from the layer and the engine's buffers alone.
+    const bool vec = !unit_norm && head_dim % 4 == 0 && value_dim % 4 == 0 && (cos_sin == nullptr || rotary_dim % 8 == 0) &&
+                     (value_cos_sin == nullptr || value_dim % 8 == 0) && row_width % 4 == 0 && split_stride % 4 == 0 &&
+                     splits <= MAX_UNROLLED_SPLITS && aligned16(qkv) && aligned16(bias) && aligned16(cos_sin) && aligned16(value_cos_sin) &&
+                     aligned16(q_out) && aligned16(k_pages) && aligned16(v_pages) && aligned16(k_dense) && aligned16(v_dense);
+    if (vec) {
+        const int rotary = cos_sin ? rotary_dim : 0, value_rotary = value_cos_sin ? value_dim : 0;
+        const int units = (heads + kv_heads) * (rotary / 8 + (head_dim - rotary) / 4) + kv_heads * (value_rotary / 8 + (value_dim - value_rotary) / 4);
+        const dim3 grid((units + 255) / 256, tokens);
+        if (out_type == ME_BF16)
+            return splits == 1 ? launch_kernel(qkv_rope_vec_store_kernel<__nv_bfloat16, 1>, grid, 256, 0, stream, a)
+                               : launch_kernel(qkv_rope_vec_store_kernel<__nv_bfloat16, MAX_UNROLLED_SPLITS>, grid, 256, 0, stream, a);
+        return splits == 1 ? launch_kernel(qkv_rope_vec_store_kernel<float, 1>, grid, 256, 0, stream, a)
+                           : launch_kernel(qkv_rope_vec_store_kernel<float, MAX_UNROLLED_SPLITS>, grid, 256, 0, stream, a);
+    }
     const long long items = static_cast<long long>(tokens) * (heads + 2 * kv_heads);
     const int blocks = static_cast<int>((items + UNIT_WARPS - 1) / UNIT_WARPS);
     const size_t smem = static_cast<size_t>(UNIT_WARPS) * std::max(head_dim, value_dim) * sizeof(float);

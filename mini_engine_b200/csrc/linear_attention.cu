@@ -702,8 +702,8 @@ __global__ void __launch_bounds__(128) gla_finish_kernel(const float* __restrict
 }
 
 // The same with the root mean square over all `count` columns of a token (every head together) and a weight of that size.
-// One block per token; column i's square goes to the partial sum of thread i % 256 in ascending order.
-template <typename T>
+// One block per token; V columns per thread and step (4: 16-byte loads), whose squares a thread adds in ascending order.
+template <typename T, int V>
 __global__ void __launch_bounds__(256) projection_finish_kernel(const float* __restrict__ o, const float* __restrict__ proj,
                                                                 int splits, size_t split_stride, int width, int g_col,
                                                                 const float* __restrict__ weight, float eps,
@@ -713,8 +713,23 @@ __global__ void __launch_bounds__(256) projection_finish_kernel(const float* __r
     pdl_trigger();
     pdl_wait();
     const float* row = o + token * count;
+    const float* gate_row = proj + token * width + g_col;
+    T* dst = out + token * count;
+    auto load = [](const float* src, float (&v)[V]) {
+        if constexpr (V == 4) {
+            const float4 q = *reinterpret_cast<const float4*>(src);
+            v[0] = q.x, v[1] = q.y, v[2] = q.z, v[3] = q.w;
+        } else {
+            v[0] = src[0];
+        }
+    };
     float sum_sq = 0.0f;
-    for (int i = threadIdx.x; i < count; i += 256) sum_sq = fmaf(row[i], row[i], sum_sq);
+    for (int i = threadIdx.x * V; i < count; i += 256 * V) {
+        float x[V];
+        load(row + i, x);
+#pragma unroll
+        for (int j = 0; j < V; ++j) sum_sq = fmaf(x[j], x[j], sum_sq);
+    }
     sum_sq = warp_sum(sum_sq);
     if ((threadIdx.x & 31) == 0) partial[threadIdx.x >> 5] = sum_sq;
     __syncthreads();
@@ -722,12 +737,29 @@ __global__ void __launch_bounds__(256) projection_finish_kernel(const float* __r
 #pragma unroll
     for (int w = 0; w < 8; ++w) total += partial[w];
     const float inv = rsqrtf(total / static_cast<float>(count) + eps);
-    const float* gate_row = proj + token * width + g_col;
-    T* dst = out + token * count;
-    for (int i = threadIdx.x; i < count; i += 256) {
-        float gate = 0.0f;
-        for (int p = 0; p < splits; ++p) gate += gate_row[p * split_stride + i];
-        dst[i] = from_float<T>((weight ? weight[i] : 1.0f) * (row[i] * inv) * finish_gate(gate, gate_kind));
+    for (int i = threadIdx.x * V; i < count; i += 256 * V) {
+        float x[V], gate[V], part[V], scale[V];
+        load(row + i, x);
+        load(gate_row + i, gate);
+        for (int p = 1; p < splits; ++p) {
+            load(gate_row + p * split_stride + i, part);
+#pragma unroll
+            for (int j = 0; j < V; ++j) gate[j] += part[j];
+        }
+#pragma unroll
+        for (int j = 0; j < V; ++j) scale[j] = 1.0f;
+        if (weight) load(weight + i, scale);
+#pragma unroll
+        for (int j = 0; j < V; ++j) x[j] = scale[j] * (x[j] * inv) * finish_gate(gate[j], gate_kind);
+        if constexpr (V == 4 && sizeof(T) == 2) {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(x[0], x[1]), hi = __floats2bfloat162_rn(x[2], x[3]);
+            uint2 packed;
+            packed.x = *reinterpret_cast<uint32_t*>(&lo), packed.y = *reinterpret_cast<uint32_t*>(&hi);
+            *reinterpret_cast<uint2*>(dst + i) = packed;
+        } else {
+#pragma unroll
+            for (int j = 0; j < V; ++j) dst[i + j] = from_float<T>(x[j]);
+        }
     }
 }
 
@@ -737,11 +769,20 @@ ME_EXPORT int me_gla_finish(const float* o, const float* proj, int splits, long 
     if (tokens <= 0) return 0;
     if (gate_kind != FINISH_SILU && gate_kind != FINISH_SIGMOID) return ME_ERR_ARGUMENT;
     if (whole_projection) {
-        if (type == ME_BF16)
-            return launch_kernel(projection_finish_kernel<__nv_bfloat16>, tokens, 256, 0, stream, o, proj, splits, (size_t)split_stride,
-                                 width, g_col, weight, eps, static_cast<__nv_bfloat16*>(out), heads * vdim, gate_kind);
-        return launch_kernel(projection_finish_kernel<float>, tokens, 256, 0, stream, o, proj, splits, (size_t)split_stride, width,
-                             g_col, weight, eps, static_cast<float*>(out), heads * vdim, gate_kind);
+        const int count = heads * vdim;
+        const auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+        // the choice follows from the sizes and the engine's buffers alone
+        const bool vec = count % 4 == 0 && width % 4 == 0 && g_col % 4 == 0 && split_stride % 4 == 0 && aligned(o) && aligned(proj) &&
+                         aligned(weight) && aligned(out);
+        const size_t stride = static_cast<size_t>(split_stride);
+        if (type == ME_BF16) {
+            auto* dst = static_cast<__nv_bfloat16*>(out);
+            return vec ? launch_kernel(projection_finish_kernel<__nv_bfloat16, 4>, tokens, 256, 0, stream, o, proj, splits, stride, width, g_col, weight, eps, dst, count, gate_kind)
+                       : launch_kernel(projection_finish_kernel<__nv_bfloat16, 1>, tokens, 256, 0, stream, o, proj, splits, stride, width, g_col, weight, eps, dst, count, gate_kind);
+        }
+        auto* dst = static_cast<float*>(out);
+        return vec ? launch_kernel(projection_finish_kernel<float, 4>, tokens, 256, 0, stream, o, proj, splits, stride, width, g_col, weight, eps, dst, count, gate_kind)
+                   : launch_kernel(projection_finish_kernel<float, 1>, tokens, 256, 0, stream, o, proj, splits, stride, width, g_col, weight, eps, dst, count, gate_kind);
     }
     const long long items = static_cast<long long>(tokens) * heads;
     const int blocks = static_cast<int>((items + 3) / 4);

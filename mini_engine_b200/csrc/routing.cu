@@ -11,8 +11,9 @@
 // dense map `weights [T][units with tensors]` (zero for units that were not chosen), and the chosen units and their weights
 // as lists `[T][top]`.  One more row of W_r (`shared_gate`) gives sigmoid(z) in shared_gate [T] and takes no part in the choice.
 //
-// One block per token: warp w forms the scores of units w, w + 8, ...; the first warp then chooses.  The sums
-// run over the columns in a fixed order, so a token's choice never depends on the rest of the batch.
+// A block takes TOKENS tokens (one, or four in a long step, which share what is read of the router): warp w forms the
+// scores of units w, w + 8, ... for all of them; then warp i chooses for token i.  The sums run over the columns in a
+// fixed order, so a token's choice never depends on the rest of the batch.
 #include "common.cuh"
 
 constexpr int ROUTE_WARPS = 8;
@@ -44,52 +45,76 @@ __device__ __forceinline__ void warp_argmax(float& value, int& index) {
     }
 }
 
-template <typename T>
+constexpr int MANY_TOKENS = 4, MANY_MAX_UNITS = 256;  // four tokens to a block, up to that many units
+constexpr int MANY_FROM = 1024;                       // from this many tokens on
+
+template <typename T, int TOKENS, int LIMIT>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_kernel(RouteArgs a) {
     constexpr int NONE = 0x7fffffff;
-    __shared__ float score[MAX_UNITS];   // what the weights are made of
-    __shared__ float choice[MAX_UNITS];  // what the choice is made by
-    __shared__ float worth[MAX_UNITS];   // of a group
-    __shared__ unsigned char eligible[MAX_UNITS];
-    const int token = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    __shared__ float scores[TOKENS][LIMIT];   // what the weights are made of
+    __shared__ float choices[TOKENS][LIMIT];  // what the choice is made by
+    __shared__ float worths[TOKENS][LIMIT];   // of a group
+    __shared__ unsigned char eligibles[TOKENS][LIMIT];
+    const int first_token = blockIdx.x * TOKENS, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     pdl_trigger();
     pdl_wait();
-    const T* h = static_cast<const T*>(a.h) + static_cast<size_t>(token) * a.hidden;
+    const T* rows_of_h[TOKENS];  // a block's last tokens may lie behind the step's: they repeat its last one and choose nothing
+#pragma unroll
+    for (int k = 0; k < TOKENS; ++k)
+        rows_of_h[k] = static_cast<const T*>(a.h) + static_cast<size_t>(min(first_token + k, a.tokens - 1)) * a.hidden;
     const int rows = a.units + (a.shared_gate != nullptr ? 1 : 0), held = a.units - a.tensorless;
     // Lane l adds the products of columns 4 l .. 4 l + 3 (+ 128 j) in ascending order into four sums of its own, which
     // are then added in a fixed order: many loads in flight, and a token's scores are the same bits in every step.
     const bool quads = a.hidden % 4 == 0 && reinterpret_cast<uintptr_t>(a.router) % 16 == 0 && reinterpret_cast<uintptr_t>(a.h) % 8 == 0;
     for (int unit = warp; unit < rows; unit += ROUTE_WARPS) {
         const float* w = a.router + static_cast<size_t>(unit) * a.hidden;
-        float sum = 0.0f;
+        float sums[TOKENS];
         if (quads) {
-            float part[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+            float part[TOKENS][4] = {};
 #pragma unroll 4
             for (int i = lane * 4; i < a.hidden; i += 128) {
                 const float4 weight = *reinterpret_cast<const float4*>(w + i);
-                part[0] = fmaf(to_float(h[i]), weight.x, part[0]);
-                part[1] = fmaf(to_float(h[i + 1]), weight.y, part[1]);
-                part[2] = fmaf(to_float(h[i + 2]), weight.z, part[2]);
-                part[3] = fmaf(to_float(h[i + 3]), weight.w, part[3]);
+#pragma unroll
+                for (int k = 0; k < TOKENS; ++k) {
+                    const T* h = rows_of_h[k] + i;
+                    part[k][0] = fmaf(to_float(h[0]), weight.x, part[k][0]);
+                    part[k][1] = fmaf(to_float(h[1]), weight.y, part[k][1]);
+                    part[k][2] = fmaf(to_float(h[2]), weight.z, part[k][2]);
+                    part[k][3] = fmaf(to_float(h[3]), weight.w, part[k][3]);
+                }
             }
-            sum = (part[0] + part[1]) + (part[2] + part[3]);
+#pragma unroll
+            for (int k = 0; k < TOKENS; ++k) sums[k] = (part[k][0] + part[k][1]) + (part[k][2] + part[k][3]);
         } else {
-            for (int i = lane; i < a.hidden; i += 32) sum = fmaf(to_float(h[i]), w[i], sum);
+#pragma unroll
+            for (int k = 0; k < TOKENS; ++k) {
+                sums[k] = 0.0f;
+                for (int i = lane; i < a.hidden; i += 32) sums[k] = fmaf(to_float(rows_of_h[k][i]), w[i], sums[k]);
+            }
         }
-        sum = warp_sum(sum);
-        if (unit == a.units) {  // the shared unit's gate
-            if (lane == 0) a.shared_gate[token] = 1.0f / (1.0f + expf(-sum));
-            continue;
+#pragma unroll
+        for (int k = 0; k < TOKENS; ++k) {
+            float sum = warp_sum(sums[k]);
+            if (unit == a.units) {  // the shared unit's gate
+                if (lane == 0 && first_token + k < a.tokens) a.shared_gate[first_token + k] = 1.0f / (1.0f + expf(-sum));
+                continue;
+            }
+            if (a.bias) sum += a.bias[unit];
+            if (lane == 0) choices[k][unit] = scores[k][unit] = a.mode == 0 ? 1.0f / (1.0f + expf(-sum)) : sum;
         }
-        if (a.bias) sum += a.bias[unit];
-        if (lane == 0) choice[unit] = score[unit] = a.mode == 0 ? 1.0f / (1.0f + expf(-sum)) : sum;
     }
-    for (int unit = threadIdx.x; unit < a.units; unit += ROUTE_WARPS * 32) {
+    __syncthreads();
+    const int token = first_token + warp;
+    if (warp >= TOKENS || token >= a.tokens) return;
+    float* score = scores[warp];
+    float* choice = choices[warp];
+    float* worth = worths[warp];
+    unsigned char* eligible = eligibles[warp];
+    for (int unit = lane; unit < a.units; unit += 32) {
         eligible[unit] = 0;
         if (unit < held) a.weights[static_cast<size_t>(token) * held + unit] = 0.0f;
     }
-    __syncthreads();
-    if (warp != 0) return;
+    __syncwarp();
     if (a.mode == 2) {
         float largest = -INFINITY, total = 0.0f;
         for (int u = lane; u < a.units; u += 32) largest = fmaxf(largest, score[u]);
@@ -170,8 +195,13 @@ ME_EXPORT int me_route(const void* h, int h_type, const float* router, const flo
     if (correction != nullptr && mode != 2) return ME_ERR_ARGUMENT;
     RouteArgs a{h, router, bias, mode, weights, chosen, chosen_weight, tokens, hidden, units, top, group_count, group_keep, weight_scale,
                 correction, tensorless, identity_weight, shared_gate};
-    if (h_type == ME_BF16) return launch_kernel(route_kernel<__nv_bfloat16>, tokens, ROUTE_WARPS * 32, 0, stream, a);
-    return launch_kernel(route_kernel<float>, tokens, ROUTE_WARPS * 32, 0, stream, a);
+    if (tokens >= MANY_FROM && units <= MANY_MAX_UNITS) {
+        const int blocks = (tokens + MANY_TOKENS - 1) / MANY_TOKENS;
+        if (h_type == ME_BF16) return launch_kernel(route_kernel<__nv_bfloat16, MANY_TOKENS, MANY_MAX_UNITS>, blocks, ROUTE_WARPS * 32, 0, stream, a);
+        return launch_kernel(route_kernel<float, MANY_TOKENS, MANY_MAX_UNITS>, blocks, ROUTE_WARPS * 32, 0, stream, a);
+    }
+    if (h_type == ME_BF16) return launch_kernel(route_kernel<__nv_bfloat16, 1, MAX_UNITS>, tokens, ROUTE_WARPS * 32, 0, stream, a);
+    return launch_kernel(route_kernel<float, 1, MAX_UNITS>, tokens, ROUTE_WARPS * 32, 0, stream, a);
 }
 
 // ------------------------------------------------------------- rows sorted by unit, for grouped products

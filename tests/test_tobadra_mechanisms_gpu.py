@@ -113,6 +113,32 @@ def test_input_convolution_in_portions_of_unequal_requests(taps, width):
             close(torch.cat(got[r]), want[r], tolerance)
 
 
+@pytest.mark.parametrize("taps", [1, 2, 3, 4, 6])
+def test_input_convolution_of_a_long_step(taps):
+    """Enough tokens that a thread takes a run of them: entries that start and end inside a run, entries shorter than the
+    taps, entries that go on from their past beside fresh ones."""
+    from mini_engine_b200.csrc import ops
+
+    g = torch.Generator().manual_seed(taps)
+    width, cut = 40, [300, 1, 2, 5, 8, 260, 3]
+    w, requests = randn(g, width, taps), [randn(g, 20 + n, width).float().double() for n in cut]
+    state = torch.full((8, taps - 1, width), 9.0, dtype=torch.float32, device="cuda") if taps > 1 else None
+    for starts in ([20] * 7, [20, 0, 20, 0, 20, 0, 0]):
+        for r, first in zip(requests, starts):  # what came before, request by request
+            if first:
+                slot = next(i for i, x in enumerate(requests) if x is r)
+                ops.input_convolution(h=f32(r[:first]), taps=f32(w.T), ctx=Context([first], [0], [slot]), state=state, out=f32(r[:first]))
+        h = torch.cat([r[s : s + n] for r, s, n in zip(requests, starts, cut)])
+        out = torch.empty(h.shape, dtype=torch.float32, device="cuda")
+        ops.input_convolution(h=f32(h), taps=f32(w.T), ctx=Context(cut, starts, list(range(7))), state=state, out=out)
+        want = torch.cat([(r + plain.causal_conv(r, w))[s : s + n] for r, s, n in zip(requests, starts, cut)])
+        close(out, want, 3e-6)
+        if taps > 1:
+            for slot, (r, s, n) in enumerate(zip(requests, starts, cut)):
+                held = torch.cat((torch.zeros(taps - 1, width, dtype=torch.float64), r))[s + n : s + n + taps - 1]
+                assert torch.equal(state[slot].cpu(), held.float())
+
+
 # ------------------------------------------------------------------- attention with rotated values
 
 
@@ -390,6 +416,30 @@ def test_delta_rule_whole_in_portions_and_token_by_token(heads, qk_heads, dim, v
         assert torch.equal(torch.cat(got[r]), whole[r])
 
 
+@pytest.mark.parametrize("taps", [1, 2, 3, 4, 6])
+@pytest.mark.parametrize("heads,qk_heads,dim,vdim", [(2, 1, 16, 40), (1, 1, 130, 9), (2, 2, 100, 128)])
+def test_delta_rule_over_a_long_step(taps, heads, qk_heads, dim, vdim):
+    """Enough tokens that a warp takes a run of them: entries that start and end inside a run, entries shorter than the
+    taps, entries that go on from their past: the very bits of the same tokens in short steps."""
+    g = torch.Generator().manual_seed(taps)
+    run = DeltaRun(heads, qk_heads, dim, vdim, taps, slots=12)
+    cut = [300, 1, 2, 5, 8, 260]
+    starts = [20, 20, 0, 20, 0, 20]
+    data = [(randn(g, 20 + n, run.width), randn(g, 20 + n, heads * dim)) for n in cut]
+    rest = (randn(g, run.channels, taps), torch.linspace(-6.0, 0.5, heads, dtype=torch.float64), randn(g, heads * dim))
+    wants = []
+    for slot, ((p, s), first, n) in enumerate(zip(data, starts, cut)):
+        if first:
+            for where in (slot, slot + 6):
+                run.step(p[:first], s[:first], *rest, [first], [0], [where])
+        short = [run.step(p[a:b], s[a:b], *rest, [b - a], [a], [slot + 6]) for a, b in zip(range(first, first + n, 100), [*range(first + 100, first + n, 100), first + n])]
+        wants.append(torch.cat(short))
+    take = lambda which: torch.cat([d[which][f : f + n] for d, f, n in zip(data, starts, cut)])  # noqa: E731
+    out = run.step(take(0), take(1), *rest, cut, starts, list(range(6)))
+    assert torch.equal(out, torch.cat(wants)) and torch.equal(run.state[:6], run.state[6:])
+    close(out[: cut[0]], run.plain(*data[0], *rest)[0][20:], 3e-5)
+
+
 @pytest.mark.parametrize("dim,vdim", [(16, 8), (64, 64), (128, 96)])
 def test_delta_rule_remembers_and_replaces(dim, vdim):
     """Straight into the recurrence: hardly any decay, beta near 1.  A value written under one key is read back 400 tokens
@@ -478,6 +528,17 @@ def test_router_with_a_correction_groups_and_units_without_tensors(experts, iden
     close(gate, plain.sigmoid(h.double() @ shared.T)[:, 0], 1e-5)
     if units > 2 and units > top:
         assert not torch.equal(run_route(h, router, torch.zeros(units), spec)[0], want)  # the correction decides
+
+
+def test_a_long_step_routes_every_token_as_a_short_one():
+    g = torch.Generator().manual_seed(9)
+    spec = {"experts": 10, "identity": 2, "top": 3, "scale": 1.5, "groups": {"count": 4, "keep": 2}}
+    h, router, correction, shared = randn(g, 1101, 72).float(), randn(g, 12, 72), 0.3 * randn(g, 12), randn(g, 1, 72)
+    whole = run_route(h, router, correction, spec, shared)
+    pieces = [run_route(h[a : a + 300], router, correction, spec, shared) for a in range(0, 1101, 300)]
+    for i in range(5):
+        assert torch.equal(whole[i], torch.cat([p[i] for p in pieces]))
+    assert torch.equal(whole[0], plain.route(h.double(), {"router": router, "correction": correction}, "", spec)[0])
 
 
 def test_units_of_other_groups_count_as_minus_infinity_and_not_zero():
