@@ -80,7 +80,10 @@ struct DeltaPrepArgs {
     float* scalars;  // [tokens][heads][2]: beta, q . k
     float q_scale, unit_eps;
     int tokens, heads, qk_heads, dim, vdim, K, channels, run;
+    int whole_runs_elsewhere;  // 1: whole runs of tokens are another launch's
 };
+
+__device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.0f + expf(-z)); }  // the division is within two ulp
 
 struct ConvWindow {
     const DeltaPrepArgs& a;
@@ -103,7 +106,7 @@ struct ConvWindow {
             else continue;
             sum = fmaf(a.conv[static_cast<size_t>(j) * a.channels + channel], x, sum);
         }
-        return sum / (1.0f + expf(-sum));
+        return silu(sum);
     }
 };
 
@@ -118,7 +121,36 @@ __device__ __forceinline__ void keep_history(const DeltaPrepArgs& a, const ConvW
     }
 }
 
-// A q/k head of one token: unit q (times its scale), unit k and their dot product.  Lane l holds channels l + 32 i.
+template <int PER>
+__device__ __forceinline__ void load_neighbours(const float* src, float (&x)[PER]) {
+    if constexpr (PER == 4) {
+        const float4 q = *reinterpret_cast<const float4*>(src);
+        x[0] = q.x, x[1] = q.y, x[2] = q.z, x[3] = q.w;
+    } else if constexpr (PER == 2) {
+        const float2 q = *reinterpret_cast<const float2*>(src);
+        x[0] = q.x, x[1] = q.y;
+    } else {
+#pragma unroll
+        for (int i = 0; i < PER; ++i) x[i] = src[i];
+    }
+}
+template <int PER>
+__device__ __forceinline__ void store_neighbours(float* dst, const float (&x)[PER]) {
+    if constexpr (PER == 4) {
+        *reinterpret_cast<float4*>(dst) = make_float4(x[0], x[1], x[2], x[3]);
+    } else if constexpr (PER == 2) {
+        *reinterpret_cast<float2*>(dst) = make_float2(x[0], x[1]);
+    } else {
+#pragma unroll
+        for (int i = 0; i < PER; ++i) dst[i] = x[i];
+    }
+}
+
+// The i-th channel of a lane: neighbours where a warp's lanes hold a head exactly, so that they may be fetched together.
+template <int PER>
+__device__ __forceinline__ int channel_of(int lane, int i, int extent) { return extent == 32 * PER ? lane * PER + i : lane + 32 * i; }
+
+// A q/k head of one token: unit q (times its scale), unit k and their dot product.
 template <int PER>
 __device__ __forceinline__ void store_unit_pair(const DeltaPrepArgs& a, size_t token, int item, int lane, float (&q)[PER], float (&k)[PER]) {
     float q_sq = 0.0f, k_sq = 0.0f;
@@ -129,14 +161,27 @@ __device__ __forceinline__ void store_unit_pair(const DeltaPrepArgs& a, size_t t
     float* dst = a.qk + (token * a.qk_heads + item) * 2 * a.dim;
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
-        const int d = lane + 32 * i;
         q[i] = q[i] * q_inv * a.q_scale, k[i] = k[i] * k_inv;
         dot = fmaf(q[i], k[i], dot);
-        if (d < a.dim) dst[d] = q[i], dst[a.dim + d] = k[i];
+    }
+    if ((PER == 2 || PER == 4) && a.dim == 32 * PER && reinterpret_cast<uintptr_t>(a.qk) % 16 == 0) {
+        store_neighbours<PER>(dst + lane * PER, q);
+        store_neighbours<PER>(dst + a.dim + lane * PER, k);
+    } else {
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int d = channel_of<PER>(lane, i, a.dim);
+            if (d < a.dim) dst[d] = q[i], dst[a.dim + d] = k[i];
+        }
     }
     dot = warp_sum(dot);
     const int per = a.heads / a.qk_heads;
     for (int h = lane; h < per; h += 32) a.scalars[(token * a.heads + item * per + h) * 2 + 1] = dot;
+}
+
+__device__ __forceinline__ float decay_of(float z, float rate) {
+    const float softplus = fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z)));
+    return 1.0f + expm1f(rate * softplus);  // the float nearest to the decay where it is near 1
 }
 
 // The decays and beta of one head and token.
@@ -146,140 +191,155 @@ __device__ __forceinline__ void store_decays(const DeltaPrepArgs& a, const ConvW
     for (int d = lane; d < a.dim; d += 32) {
         float z = a.dt_bias[head * a.dim + d];
         for (int s = 0; s < a.second_splits; ++s) z += logits[s * a.second_stride + d];
-        const float softplus = fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z)));
-        dst[d] = 1.0f + expm1f(rate * softplus);  // the float nearest to the decay where it is near 1
+        dst[d] = decay_of(z, rate);
     }
     if (lane == 0) a.scalars[(token * a.heads + head) * 2] = 1.0f / (1.0f + expf(-window.input(static_cast<int>(token), a.beta_col + head)));
 }
 
 // One warp per (a.run tokens, item): items [0, qk_heads) form q, k and q . k of a q/k head, items behind them v, the
-// decays and beta of a head; a lane holds channels lane, lane + 32, ... (PER of them at most).  Tokens that have K - 1
-// tokens of their entry in front of them slide a window of inputs in registers (KC = K; KC = 0: more taps than that, read
-// again for every token).  The first K - 1 tokens of an entry reach into the request's past; the warp that holds the
-// entry's first token computes all of them and then leaves the entry's last inputs of its channels in the slot, so that
-// nothing is read after it was replaced.  Both forms add a channel's products in the same order.
+// decays and beta of a head; a lane holds at most PER channels at a time.  The first K - 1 tokens of an entry reach into the
+// request's past; the warp that holds the entry's first token computes all of them and then leaves the entry's last
+// inputs of its channels in the slot, so that nothing is read after it was replaced.
 constexpr int PREP_RUN = 8;           // tokens of a warp in a long step
 constexpr int PREP_RUN_TOKENS = 512;  // from this many tokens on; a shorter step gives every token warps of its own
 
+// Whether the PREP_RUN tokens from `run_begin` on lie in one entry with K - 1 of its tokens in front of them.
+__device__ __forceinline__ bool whole_run(const DeltaPrepArgs& a, int run_begin) {
+    if (run_begin + PREP_RUN > a.tokens) return false;
+    const int entry = a.entry_of_token[run_begin];
+    return a.entry_of_token[run_begin + PREP_RUN - 1] == entry && run_begin - a.cu_tokens[entry] >= a.K - 1;
+}
+
+// The whole runs of a long step, whose projections are not split: every input of the run is fetched before any is used.
+// dim is 32 PER, vdim a multiple of it, every row and segment starts on 16 bytes.  The same bits as the kernel below.
 template <int PER, int KC>
+__global__ void __launch_bounds__(PREP_WARPS * 32, 2) delta_prepare_runs_kernel(DeltaPrepArgs a) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, item = blockIdx.y;
+    const int run_begin = (blockIdx.x * PREP_WARPS + warp) * PREP_RUN;
+    pdl_trigger();
+    pdl_wait();
+    if (run_begin >= a.tokens || !whole_run(a, run_begin)) return;
+    constexpr int ROWS = PREP_RUN + KC - 1;
+    auto fetch = [&](int column, float (&x)[ROWS][PER]) {
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r)
+            load_neighbours<PER>(a.proj + static_cast<size_t>(run_begin - (KC - 1) + r) * a.width + column + lane * PER, x[r]);
+    };
+    auto convolve = [&](int column, const float (&x)[ROWS][PER], float (&y)[PREP_RUN][PER]) {
+        float taps[KC][PER];
+#pragma unroll
+        for (int j = 0; j < KC; ++j) load_neighbours<PER>(a.conv + static_cast<size_t>(j) * a.channels + column + lane * PER, taps[j]);
+#pragma unroll
+        for (int t = 0; t < PREP_RUN; ++t)
+#pragma unroll
+            for (int i = 0; i < PER; ++i) {
+                float sum = 0.0f;
+#pragma unroll
+                for (int j = 0; j < KC; ++j) sum = fmaf(taps[j][i], x[t + j][i], sum);
+                y[t][i] = silu(sum);
+            }
+    };
+    if (item < a.qk_heads) {
+        const int q_column = a.q_col + item * a.dim, k_column = a.k_col + item * a.dim;
+        float x[ROWS][PER], q[PREP_RUN][PER], k[PREP_RUN][PER];
+        fetch(q_column, x);
+        convolve(q_column, x, q);
+        fetch(k_column, x);
+        convolve(k_column, x, k);
+#pragma unroll
+        for (int t = 0; t < PREP_RUN; ++t) store_unit_pair<PER>(a, run_begin + t, item, lane, q[t], k[t]);
+        return;
+    }
+    const int head = item - a.qk_heads;
+    const float rate = -expf(a.a_log[head]);
+    const size_t step = static_cast<size_t>(a.heads) * (a.dim + a.vdim);
+    float* dst = a.gv + (static_cast<size_t>(run_begin) * a.heads + head) * (a.dim + a.vdim) + lane * PER;
+    float logits[PREP_RUN][PER], bias[PER];
+#pragma unroll
+    for (int t = 0; t < PREP_RUN; ++t)
+        load_neighbours<PER>(a.second + static_cast<size_t>(run_begin + t) * a.second_width + head * a.dim + lane * PER, logits[t]);
+    load_neighbours<PER>(a.dt_bias + head * a.dim + lane * PER, bias);
+    if (lane < PREP_RUN) {
+        const float z = a.proj[static_cast<size_t>(run_begin + lane) * a.width + a.beta_col + head];
+        a.scalars[(static_cast<size_t>(run_begin + lane) * a.heads + head) * 2] = 1.0f / (1.0f + expf(-z));
+    }
+    for (int offset = 0; offset < a.vdim; offset += 32 * PER) {
+        const int column = a.v_col + head * a.vdim + offset;
+        float x[ROWS][PER], v[PREP_RUN][PER];
+        fetch(column, x);
+        convolve(column, x, v);
+#pragma unroll
+        for (int t = 0; t < PREP_RUN; ++t) store_neighbours<PER>(dst + t * step + a.dim + offset, v[t]);
+    }
+#pragma unroll
+    for (int t = 0; t < PREP_RUN; ++t) {
+#pragma unroll
+        for (int i = 0; i < PER; ++i) logits[t][i] = decay_of(bias[i] + logits[t][i], rate);
+        store_neighbours<PER>(dst + t * step, logits[t]);
+    }
+}
+
+template <int PER>
 __global__ void __launch_bounds__(PREP_WARPS * 32) delta_prepare_kernel(DeltaPrepArgs a) {
-    constexpr int WINDOW = KC > 1 ? KC - 1 : 1;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, item = blockIdx.y;
     const int run_begin = (blockIdx.x * PREP_WARPS + warp) * a.run, run_end = min(run_begin + a.run, a.tokens);
     pdl_trigger();
     pdl_wait();
+    if (run_begin >= a.tokens || (a.whole_runs_elsewhere && whole_run(a, run_begin))) return;
     const bool is_qk = item < a.qk_heads;
     const int head = item - a.qk_heads;
     const float rate = is_qk ? 0.0f : -expf(a.a_log[head]);
-    const int q_column = a.q_col + item * a.dim, k_column = a.k_col + item * a.dim;
-    // channels of this lane: of q and k, or of v in the place of q
-    const int column = is_qk ? q_column : a.v_col + head * a.vdim, extent = is_qk ? a.dim : a.vdim;
-    const int blocks_of_v = is_qk ? 1 : (a.vdim + 32 * PER - 1) / (32 * PER);
-    for (int block = 0; block < blocks_of_v; ++block) {  // a value head wider than 32 PER channels takes several rounds
-        const int offset = block * 32 * PER;
-        float held[2][WINDOW][PER], taps[2][KC > 0 ? KC : 1][PER];
-        if constexpr (KC > 0) {
-#pragma unroll
-            for (int j = 0; j < KC; ++j)
-#pragma unroll
-                for (int i = 0; i < PER; ++i) {
-                    const int d = offset + lane + 32 * i;
-                    taps[0][j][i] = d < extent ? a.conv[static_cast<size_t>(j) * a.channels + column + d] : 0.0f;
-                    taps[1][j][i] = is_qk && d < extent ? a.conv[static_cast<size_t>(j) * a.channels + k_column + d] : 0.0f;
-                }
-        }
-        int filled = -1;  // the token in front of which the window stands
-        for (int t = run_begin; t < run_end; ++t) {
-            const int entry = a.entry_of_token[t], first = a.cu_tokens[entry], n0 = t - first;
-            if (n0 > 0 && n0 < a.K - 1) continue;  // done by the warp of the entry's first token
-            float* slot = a.state + static_cast<size_t>(a.state_slots[entry]) * a.slot_floats + a.matrix;
-            const bool past = a.K > 1 && a.fresh[entry] == 0;
-            const ConvWindow window{a, first, past ? slot : nullptr};
-            float x[2][PER];
-            if (KC > 0 && n0 >= a.K - 1) {
-                if (filled != t) {
-#pragma unroll
-                    for (int w = 0; w < KC - 1; ++w)
-#pragma unroll
-                        for (int i = 0; i < PER; ++i) {
-                            const int d = offset + lane + 32 * i;
-                            held[0][w][i] = d < extent ? window.input(t - (KC - 1) + w, column + d) : 0.0f;
-                            held[1][w][i] = is_qk && d < extent ? window.input(t - (KC - 1) + w, k_column + d) : 0.0f;
-                        }
-                }
-#pragma unroll
-                for (int which = 0; which < 2; ++which)
-#pragma unroll
-                    for (int i = 0; i < PER; ++i) {
-                        const int d = offset + lane + 32 * i;
-                        x[which][i] = 0.0f;
-                        if (which == 1 && !is_qk) continue;
-                        const float now = d < extent ? window.input(t, (which ? k_column : column) + d) : 0.0f;
-                        float sum = 0.0f;
-#pragma unroll
-                        for (int w = 0; w < KC - 1; ++w) sum = fmaf(taps[which][w][i], held[which][w][i], sum);
-                        sum = fmaf(taps[which][KC > 0 ? KC - 1 : 0][i], now, sum);
-                        x[which][i] = sum / (1.0f + expf(-sum));
-#pragma unroll
-                        for (int w = 0; w + 1 < KC - 1; ++w) held[which][w][i] = held[which][w + 1][i];
-                        if (KC > 1) held[which][WINDOW - 1][i] = now;
-                    }
-                filled = t + 1;
-                if (is_qk) {
-                    store_unit_pair<PER>(a, t, item, lane, x[0], x[1]);
-                } else {
-                    float* dst = a.gv + (static_cast<size_t>(t) * a.heads + head) * (a.dim + a.vdim) + a.dim;
-#pragma unroll
-                    for (int i = 0; i < PER; ++i)
-                        if (offset + lane + 32 * i < extent) dst[offset + lane + 32 * i] = x[0][i];
-                    if (block == 0) store_decays(a, window, t, head, rate, lane);
-                }
-                continue;
-            }
-            // the entry's first tokens, or more taps than the window holds
-            const int count = a.cu_tokens[entry + 1] - first;
-            const int run = n0 == 0 ? min(count, max(a.K - 1, 1)) : 1;
-            for (int n = n0; n < n0 + run; ++n) {
-                const size_t token = static_cast<size_t>(first + n);
+    const int q_column = a.q_col + item * a.dim, k_column = a.k_col + item * a.dim, v_column = a.v_col + head * a.vdim;
+    for (int t = run_begin; t < run_end; ++t) {
+        const int entry = a.entry_of_token[t], first = a.cu_tokens[entry], n0 = t - first;
+        if (n0 > 0 && n0 < a.K - 1) continue;  // done by the warp of the entry's first token
+        float* slot = a.state + static_cast<size_t>(a.state_slots[entry]) * a.slot_floats + a.matrix;
+        const bool past = a.K > 1 && a.fresh[entry] == 0;
+        const ConvWindow window{a, first, past ? slot : nullptr};
+        const int count = a.cu_tokens[entry + 1] - first;
+        const int run = n0 == 0 ? min(count, max(a.K - 1, 1)) : 1;
+        for (int n = n0; n < n0 + run; ++n) {
+            const size_t token = static_cast<size_t>(first + n);
+            if (is_qk) {
+                float q[PER], k[PER];
 #pragma unroll
                 for (int i = 0; i < PER; ++i) {
-                    const int d = offset + lane + 32 * i;
-                    x[0][i] = d < extent ? window(n, column + d) : 0.0f;
-                    x[1][i] = is_qk && d < extent ? window(n, k_column + d) : 0.0f;
+                    const int d = channel_of<PER>(lane, i, a.dim);
+                    q[i] = d < a.dim ? window(n, q_column + d) : 0.0f;
+                    k[i] = d < a.dim ? window(n, k_column + d) : 0.0f;
                 }
-                if (is_qk) {
-                    store_unit_pair<PER>(a, token, item, lane, x[0], x[1]);
-                    continue;
-                }
+                store_unit_pair<PER>(a, token, item, lane, q, k);
+            } else {
                 float* dst = a.gv + (token * a.heads + head) * (a.dim + a.vdim) + a.dim;
-#pragma unroll
-                for (int i = 0; i < PER; ++i)
-                    if (offset + lane + 32 * i < extent) dst[offset + lane + 32 * i] = x[0][i];
-                if (block == 0) store_decays(a, window, token, head, rate, lane);
+                for (int e = lane; e < a.vdim; e += 32) dst[e] = window(n, v_column + e);
+                store_decays(a, window, token, head, rate, lane);
             }
-            if (n0 != 0) continue;
-#pragma unroll
-            for (int i = 0; i < PER; ++i) {
-                const int d = offset + lane + 32 * i;
-                if (d >= extent) continue;
-                keep_history(a, window, slot, past, count, column + d);
-                if (is_qk) keep_history(a, window, slot, past, count, k_column + d);
-            }
+        }
+        if (n0 != 0) continue;
+        const int extent = is_qk ? a.dim : a.vdim;
+        for (int d = lane; d < extent; d += 32) {
+            keep_history(a, window, slot, past, count, (is_qk ? q_column : v_column) + d);
+            if (is_qk) keep_history(a, window, slot, past, count, k_column + d);
         }
     }
 }
 
 template <int PER>
-static int launch_delta_prepare(const DeltaPrepArgs& a, cudaStream_t stream) {
+static int launch_delta_prepare(DeltaPrepArgs a, cudaStream_t stream) {
     const dim3 grid((a.tokens + PREP_WARPS * a.run - 1) / (PREP_WARPS * a.run), a.qk_heads + a.heads);
-    constexpr int THREADS = PREP_WARPS * 32;
-    if (PER <= 4) {  // the window of a wider head does not fit the registers
-        if (a.K == 1) return launch_kernel(delta_prepare_kernel<PER, PER <= 4 ? 1 : 0>, grid, THREADS, 0, stream, a);
-        if (a.K == 2) return launch_kernel(delta_prepare_kernel<PER, PER <= 4 ? 2 : 0>, grid, THREADS, 0, stream, a);
-        if (a.K == 3) return launch_kernel(delta_prepare_kernel<PER, PER <= 4 ? 3 : 0>, grid, THREADS, 0, stream, a);
-        if (a.K == 4) return launch_kernel(delta_prepare_kernel<PER, PER <= 4 ? 4 : 0>, grid, THREADS, 0, stream, a);
+    if constexpr (PER <= 4) {
+        const auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+        if (a.run == PREP_RUN && a.K >= 2 && a.K <= 4 && a.splits == 1 && a.second_splits == 1 && a.dim == 32 * PER &&
+            a.vdim % (32 * PER) == 0 && a.width % 4 == 0 && a.second_width % 4 == 0 && aligned(a.proj) && aligned(a.second) &&
+            aligned(a.conv) && aligned(a.dt_bias) && aligned(a.qk) && aligned(a.gv)) {
+            const int code = a.K == 2   ? launch_kernel(delta_prepare_runs_kernel<PER, 2>, grid, PREP_WARPS * 32, 0, stream, a)
+                             : a.K == 3 ? launch_kernel(delta_prepare_runs_kernel<PER, 3>, grid, PREP_WARPS * 32, 0, stream, a)
+                                        : launch_kernel(delta_prepare_runs_kernel<PER, 4>, grid, PREP_WARPS * 32, 0, stream, a);
+            if (code) return code;
+            a.whole_runs_elsewhere = 1;
+        }
     }
-    return launch_kernel(delta_prepare_kernel<PER, 0>, grid, THREADS, 0, stream, a);
+    return launch_kernel(delta_prepare_kernel<PER>, grid, PREP_WARPS * 32, 0, stream, a);
 }
 
 ME_EXPORT int me_delta_prepare(const float* proj, int splits, long long split_stride, int width, int q_col, int k_col, int v_col,
@@ -297,7 +357,7 @@ ME_EXPORT int me_delta_prepare(const float* proj, int splits, long long split_st
     DeltaPrepArgs a{proj, splits, (size_t)split_stride, width, q_col, k_col, v_col, beta_col, second, second_splits,
                     (size_t)second_stride, second_width, conv, a_log, dt_bias, entry_of_token, cu_tokens, state_slots, fresh,
                     state, (size_t)slot_floats, (size_t)matrix, qk, gv, scalars, q_scale, unit_eps, tokens, heads, qk_heads,
-                    dim, vdim, taps_count, channels, tokens >= PREP_RUN_TOKENS ? PREP_RUN : 1};
+                    dim, vdim, taps_count, channels, tokens >= PREP_RUN_TOKENS ? PREP_RUN : 1, 0};
     if (dim <= 32) return launch_delta_prepare<1>(a, stream);
     if (dim <= 64) return launch_delta_prepare<2>(a, stream);
     if (dim <= 128) return launch_delta_prepare<4>(a, stream);
@@ -312,10 +372,10 @@ ME_EXPORT int me_delta_prepare(const float* proj, int splits, long long split_st
 // * C columns, so that a head needs several warps.  The walk's time is the latency of one token's step; the next token's q,
 // k and decays are read while it runs.  Per token the two dots S^T k and S^T q of the decayed state run together and meet
 // in one butterfly over the L lanes; o = S^T q + (q . k) u needs no second one after the correction.
-// A block of WARPS warps shares the tokens' q, k, decays, values and scalars, fetched SC tokens ahead by asynchronous
-// copies.  Columns are independent and a token's output depends on the tokens before it through the state alone: the
+// The walking warps of a block share the tokens' q, k, decays, values and scalars; one more warp fetches them, SC tokens
+// ahead, by asynchronous copies, and stores the outputs of the SC tokens before.  Columns are independent and a token's output depends on the tokens before it through the state alone: the
 // bits are the same for a whole prompt, its portions and single decoded tokens.
-constexpr int SCAN_WARPS = 4;  // most warps of a block
+constexpr int SCAN_WARPS = 4;  // most walking warps of a block
 
 struct DeltaScanArgs {
     const float* qk;       // [tokens][qk_heads][2][dim]
@@ -347,12 +407,12 @@ template <int R>
 struct TokenRow {
     float2 k[R / 2], q[R / 2], g[R / 2];
     template <int L>
-    __device__ __forceinline__ void load(const float* q_s, const float* k_s, const float* g_s, int at) {
+    __device__ __forceinline__ void load(const float* at) {
 #pragma unroll
         for (int i = 0; i < R / 4; ++i) {
-            const float4 k4 = *reinterpret_cast<const float4*>(k_s + at + 4 * i * L);
-            const float4 q4 = *reinterpret_cast<const float4*>(q_s + at + 4 * i * L);
-            const float4 g4 = *reinterpret_cast<const float4*>(g_s + at + 4 * i * L);
+            const float4 q4 = *reinterpret_cast<const float4*>(at + 4 * i * L);
+            const float4 k4 = *reinterpret_cast<const float4*>(at + L * R + 4 * i * L);
+            const float4 g4 = *reinterpret_cast<const float4*>(at + 2 * L * R + 4 * i * L);
             k[2 * i] = make_float2(k4.x, k4.y), k[2 * i + 1] = make_float2(k4.z, k4.w);
             q[2 * i] = make_float2(q4.x, q4.y), q[2 * i + 1] = make_float2(q4.z, q4.w);
             g[2 * i] = make_float2(g4.x, g4.y), g[2 * i + 1] = make_float2(g4.z, g4.w);
@@ -361,18 +421,19 @@ struct TokenRow {
 };
 
 template <int L, int R, int C, int SC>
-__global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(DeltaScanArgs a) {
+__global__ void __launch_bounds__((SCAN_WARPS + 1) * 32) delta_scan_kernel(DeltaScanArgs a) {
     constexpr int DP = L * R;  // the key channels a column has room for
     constexpr int GROUPS = 32 / L, COLUMNS = GROUPS * C;  // of a warp
-    constexpr bool PREFETCH = R <= 16;  // registers for a second token's row
     extern __shared__ __align__(16) float staged[];
-    const int threads = blockDim.x, columns = (threads >> 5) * COLUMNS;
+    const int threads = blockDim.x, warp = threadIdx.x >> 5, warps = (threads >> 5) - 1, columns = warps * COLUMNS;
     const int stage_floats = SC * (3 * DP + columns + 2);
-    // one stage: q [SC][DP], k [SC][DP], g [SC][DP], v [SC][columns], scalars [SC][2]
+    float* results = staged + 2 * stage_floats;  // [2][SC][columns]
+    const bool fetches = warp == warps;  // the last warp
+    // one stage: q, k and the decays of every token [SC][3][DP], v [SC][columns], scalars [SC][2]
     const int entry = blockIdx.x, head = blockIdx.y, qk_head = head / (a.heads / a.qk_heads);
     const int first_column = blockIdx.z * columns;
     const int lane = threadIdx.x & 31, part = lane % L;
-    const int local_column = (threadIdx.x >> 5) * COLUMNS + lane / L;  // and GROUPS, 2 GROUPS, ... behind it
+    const int local_column = warp * COLUMNS + lane / L;  // and GROUPS, 2 GROUPS, ... behind it
     const int dim = a.dim;
     for (int i = threadIdx.x; i < 2 * SC * 3 * (DP - dim); i += threads) {  // channels dim .. DP are zero for good
         const int stage = i / (SC * 3 * (DP - dim)), j = i % (SC * 3 * (DP - dim));
@@ -386,7 +447,7 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(DeltaScanAr
     bool live[C];
 #pragma unroll
     for (int c = 0; c < C; ++c) {
-        live[c] = first_column + local_column + c * GROUPS < a.vdim;
+        live[c] = !fetches && first_column + local_column + c * GROUPS < a.vdim;
         const bool load = live[c] && a.fresh[entry] == 0;
         const float* src = state + static_cast<size_t>(c) * GROUPS * dim;
 #pragma unroll
@@ -405,66 +466,80 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(DeltaScanAr
         }
     }
 
+    const int live_columns = min(columns, a.vdim - first_column);
+    // The fetching warp's lane holds 16-byte pieces lane, lane + 32, ... of a token's q, k and decays (piece j belongs at
+    // float 4 j of the token's row); their sources move on by one token at a time.
+    constexpr int PIECES = (3 * DP / 4 + 31) / 32;
+    const float* source[PIECES];
+    bool wanted[PIECES];
+    const size_t qk_step = static_cast<size_t>(a.qk_heads) * 2 * dim, gv_step = static_cast<size_t>(a.heads) * (dim + a.vdim);
+    const float* qk_begin = a.qk + (static_cast<size_t>(begin) * a.qk_heads + qk_head) * 2 * dim;
+    const float* gv_begin = a.gv + (static_cast<size_t>(begin) * a.heads + head) * (dim + a.vdim);
+#pragma unroll
+    for (int i = 0; i < PIECES; ++i) {
+        const int j = lane + 32 * i, which = j / (DP / 4), d = j % (DP / 4) * 4;
+        wanted[i] = which < 3 && d < dim;
+        source[i] = which < 2 ? qk_begin + which * dim + d : gv_begin + d;
+    }
+    const float* value_source = gv_begin + dim + first_column;
+    const float* scalar_source = a.scalars + (static_cast<size_t>(begin) * a.heads + head) * 2;
     auto stage_tokens = [&](int chunk, float* stage) {
         const int count = min(SC, end - chunk);
-        float* q_s = stage;
         float* v_s = stage + SC * 3 * DP;
-        float* scalars_s = v_s + SC * columns;
-        if (a.vector) {
-            const int quads = dim / 4;
-            for (int i = threadIdx.x; i < count * 3 * quads; i += threads) {
-                const int t = i / (3 * quads), j = i % (3 * quads), which = j / quads, d = (j % quads) * 4;
-                const size_t token = static_cast<size_t>(chunk + t);
-                const float* src = which < 2 ? a.qk + ((token * a.qk_heads + qk_head) * 2 + which) * dim + d
-                                             : a.gv + (token * a.heads + head) * (dim + a.vdim) + d;
-                copy_async_16(q_s + (which * SC + t) * DP + d, src);
+        for (int t = 0; t < count; ++t) {
+            if (a.vector) {
+#pragma unroll
+                for (int i = 0; i < PIECES; ++i) {
+                    if (wanted[i]) copy_async_16(stage + t * 3 * DP + 4 * (lane + 32 * i), source[i]);
+                    source[i] += (lane + 32 * i) / (DP / 4) < 2 ? qk_step : gv_step;
+                }
+            } else {
+                const float* qk = qk_begin + (chunk - begin + t) * qk_step;
+                const float* gv = gv_begin + (chunk - begin + t) * gv_step;
+                for (int j = lane; j < 2 * dim; j += 32) copy_async_4(stage + t * 3 * DP + j + (j < dim ? 0 : DP - dim), qk + j);
+                for (int j = lane; j < dim; j += 32) copy_async_4(stage + (t * 3 + 2) * DP + j, gv + j);
             }
-        } else {
-            for (int i = threadIdx.x; i < count * 3 * dim; i += threads) {
-                const int t = i / (3 * dim), j = i % (3 * dim), which = j / dim, d = j % dim;
-                const size_t token = static_cast<size_t>(chunk + t);
-                const float* src = which < 2 ? a.qk + ((token * a.qk_heads + qk_head) * 2 + which) * dim + d
-                                             : a.gv + (token * a.heads + head) * (dim + a.vdim) + d;
-                copy_async_4(q_s + (which * SC + t) * DP + d, src);
-            }
+            for (int j = lane; j < live_columns; j += 32) copy_async_4(v_s + t * columns + j, value_source + j);
+            if (lane < 2) copy_async_4(v_s + SC * columns + 2 * t + lane, scalar_source + lane);
+            value_source += gv_step;
+            scalar_source += a.heads * 2;
         }
-        for (int i = threadIdx.x; i < count * columns; i += threads) {
-            const int t = i / columns, c = i % columns;
-            if (first_column + c < a.vdim)
-                copy_async_4(v_s + t * columns + c, a.gv + (static_cast<size_t>(chunk + t) * a.heads + head) * (dim + a.vdim) + dim + first_column + c);
-        }
-        for (int i = threadIdx.x; i < count * 2; i += threads)
-            copy_async_4(scalars_s + i, a.scalars + (static_cast<size_t>(chunk + i / 2) * a.heads + head) * 2 + i % 2);
         copy_async_commit();
     };
 
-    if (begin < end) stage_tokens(begin, staged);
+    auto store_results = [&](int chunk, const float* tile) {
+        const int count = min(SC, end - chunk);
+        float* out = a.out + (static_cast<size_t>(chunk) * a.heads + head) * a.vdim + first_column;
+        for (int t = 0; t < count; ++t)
+            for (int j = lane; j < live_columns; j += 32) out[static_cast<size_t>(t) * a.heads * a.vdim + j] = tile[t * columns + j];
+    };
+
+    __syncthreads();  // the zeros of the unused channels
+    if (fetches && begin < end) {
+        stage_tokens(begin, staged);
+        copy_async_wait<0>();
+    }
+    __syncthreads();
     int buffer = 0;
     for (int chunk = begin; chunk < end; chunk += SC, buffer ^= 1) {
         const int count = min(SC, end - chunk);
-        if (chunk + SC < end) {
-            stage_tokens(chunk + SC, staged + (buffer ^ 1) * stage_floats);
-            copy_async_wait<1>();
-        } else {
+        if (fetches) {
+            if (chunk + SC < end) stage_tokens(chunk + SC, staged + (buffer ^ 1) * stage_floats);
+            if (chunk > begin) store_results(chunk - SC, results + (buffer ^ 1) * SC * columns);
             copy_async_wait<0>();
+            __syncthreads();
+            continue;
         }
-        __syncthreads();
-        const float* q_s = staged + buffer * stage_floats;
-        const float* k_s = q_s + SC * DP;
-        const float* g_s = k_s + SC * DP;
-        const float* v_s = g_s + SC * DP;
+        const float* rows_s = staged + buffer * stage_floats + 4 * part;
+        const float* v_s = staged + buffer * stage_floats + SC * 3 * DP;
         const float* scalars_s = v_s + SC * columns;
-        TokenRow<R> row;
-        row.template load<L>(q_s, k_s, g_s, 4 * part);
-#pragma unroll 1
-        for (int t = 0; t < count; ++t) {
-            TokenRow<R> next;
-            if constexpr (PREFETCH) next.template load<L>(q_s, k_s, g_s, min(t + 1, count - 1) * DP + 4 * part);
-            const float beta = scalars_s[2 * t], dot = scalars_s[2 * t + 1];
+        // One token: its row is in registers already.
+        auto walk = [&](const TokenRow<R>& row, int t) {
+            const float2 scalars = *reinterpret_cast<const float2*>(scalars_s + 2 * t);  // beta, q . k
             float dot_k[C], dot_q[C], v[C];
 #pragma unroll
             for (int c = 0; c < C; ++c) {
-                v[c] = live[c] ? v_s[t * columns + local_column + c * GROUPS] : 0.0f;
+                v[c] = v_s[t * columns + local_column + c * GROUPS];  // a column behind the last one reads what is there and is never stored
                 float2 on_k[2] = {make_float2(0.0f, 0.0f), make_float2(0.0f, 0.0f)};
                 float2 on_q[2] = {make_float2(0.0f, 0.0f), make_float2(0.0f, 0.0f)};
 #pragma unroll
@@ -484,20 +559,31 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(DeltaScanAr
                     dot_q[c] += __shfl_xor_sync(0xffffffffu, dot_q[c], offset);
                 }
             }
-            float* out = a.out + (static_cast<size_t>(chunk + t) * a.heads + head) * a.vdim + first_column + local_column;
+            float mine = 0.0f;  // lane number c of a group stores column c
 #pragma unroll
             for (int c = 0; c < C; ++c) {
-                const float u = beta * (v[c] - dot_k[c]);
+                const float u = scalars.x * (v[c] - dot_k[c]);
                 const float2 uu = make_float2(u, u);
 #pragma unroll
                 for (int i = 0; i < R / 2; ++i) s[c][i] = __ffma2_rn(row.k[i], uu, s[c][i]);
-                if (live[c] && part == 0) out[c * GROUPS] = fmaf(dot, u, dot_q[c]);
+                const float o = fmaf(scalars.y, u, dot_q[c]);
+                if (c == 0 || part == c) mine = o;
             }
-            if constexpr (PREFETCH) row = next;
-            else row.template load<L>(q_s, k_s, g_s, min(t + 1, count - 1) * DP + 4 * part);
+            if (part < C) results[(buffer * SC + t) * columns + local_column + part * GROUPS] = mine;
+        };
+        TokenRow<R> even, odd;
+        even.template load<L>(rows_s);
+#pragma unroll 1
+        for (int t = 0; t < count; t += 2) {
+            if (t + 1 < count) odd.template load<L>(rows_s + (t + 1) * 3 * DP);
+            walk(even, t);
+            if (t + 1 >= count) break;
+            if (t + 2 < count) even.template load<L>(rows_s + (t + 2) * 3 * DP);
+            walk(odd, t + 1);
         }
         __syncthreads();
     }
+    if (fetches && begin < end) store_results(begin + (end - begin - 1) / SC * SC, results + (buffer ^ 1) * SC * columns);
 #pragma unroll
     for (int c = 0; c < C; ++c) {
         if (!live[c]) continue;
@@ -528,11 +614,11 @@ static int launch_delta_scan(const DeltaScanArgs& a, int entries, cudaStream_t s
                          (warps / 2) * COLUMNS >= a.vdim))
         warps /= 2;
     const int columns = warps * COLUMNS;
-    const size_t smem = static_cast<size_t>(2) * SC * (3 * L * R + columns + 2) * sizeof(float);
+    const size_t smem = static_cast<size_t>(2) * SC * (3 * L * R + 2 * columns + 2) * sizeof(float);
     if (smem > 48 * 1024)
         if (const int e = opt_in(delta_scan_kernel<L, R, C, SC>, 200 * 1024)) return e;
     const dim3 grid(entries, a.heads, (a.vdim + columns - 1) / columns);
-    return launch_kernel_in_order(delta_scan_kernel<L, R, C, SC>, grid, warps * 32, smem, stream, a);
+    return launch_kernel_in_order(delta_scan_kernel<L, R, C, SC>, grid, (warps + 1) * 32, smem, stream, a);
 }
 
 ME_EXPORT int me_delta_scan(const float* qk, const float* gv, const float* scalars, const int* cu_tokens, const int* state_slots,
@@ -544,8 +630,8 @@ ME_EXPORT int me_delta_scan(const float* qk, const float* gv, const float* scala
     const auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
     const int vector = dim % 4 == 0 && vdim % 4 == 0 && slot_floats % 4 == 0 && aligned(qk) && aligned(gv) && aligned(state);
     DeltaScanArgs a{qk, gv, scalars, cu_tokens, state_slots, fresh, state, (size_t)slot_floats, out, heads, qk_heads, dim, vdim, vector};
-    if (dim <= 32) return launch_delta_scan<8, 4, 2, 16>(a, entries, stream);
-    if (dim <= 64) return launch_delta_scan<8, 8, 2, 16>(a, entries, stream);
+    if (dim <= 32) return launch_delta_scan<8, 4, 1, 16>(a, entries, stream);
+    if (dim <= 64) return launch_delta_scan<8, 8, 1, 16>(a, entries, stream);
     if (dim <= 128) return launch_delta_scan<8, 16, 2, 16>(a, entries, stream);
     if (dim <= 256) return launch_delta_scan<16, 16, 2, 8>(a, entries, stream);
     if (dim <= MAX_DIM) return launch_delta_scan<16, 32, 1, 8>(a, entries, stream);

@@ -331,12 +331,12 @@ def test_finish_with_a_norm_per_head_and_a_sigmoid_gate(dtype):
 
 
 class DeltaRun:
-    """A delta-rule mixer's two kernels on given sums (two partial sums that meet in the kernels)."""
+    """A delta-rule mixer's two kernels on given sums (with ``halves``: two partial sums that meet in the kernels)."""
 
-    def __init__(self, heads, qk_heads, dim, vdim, taps, slots=4):
-        self.__dict__.update(heads=heads, qk_heads=qk_heads, dim=dim, vdim=vdim, taps=taps)
+    def __init__(self, heads, qk_heads, dim, vdim, taps, slots=4, halves=True):
+        self.__dict__.update(heads=heads, qk_heads=qk_heads, dim=dim, vdim=vdim, taps=taps, halves=halves)
         self.channels = 2 * qk_heads * dim + heads * vdim
-        self.width = self.channels + heads
+        self.width = -(-(self.channels + heads) // 4) * 4
         self.columns = {"q": 0, "k": qk_heads * dim, "v": 2 * qk_heads * dim, "beta": self.channels}
         self.matrix = heads * dim * vdim
         self.state = torch.full((slots, self.matrix + (taps - 1) * self.channels), 5.0, dtype=torch.float32, device="cuda")
@@ -348,7 +348,7 @@ class DeltaRun:
         ctx = Context(counts, starts, slots)
         new = lambda *shape: torch.full(shape, float("nan"), dtype=torch.float32, device="cuda")  # noqa: E731
         qk, gv, scalars = new(tokens, self.qk_heads * 2 * self.dim), new(tokens, self.heads * (self.dim + self.vdim)), new(tokens, self.heads * 2)
-        halves = lambda t: f32(torch.stack((0.25 * t, 0.75 * t)))  # noqa: E731
+        halves = lambda t: f32(torch.stack((0.25 * t, 0.75 * t)) if self.halves else t.unsqueeze(0))  # noqa: E731
         ops.delta_prepare(proj=halves(proj), columns=self.columns, second=halves(second), conv=f32(conv.T), a_log=f32(a_log),
                           dt_bias=f32(dt_bias), ctx=ctx, state=self.state, matrix=self.matrix, qk=qk, gv=gv, scalars=scalars,
                           q_scale=self.dim**-0.5, unit_eps=1e-6, **sizes)  # fmt: skip
@@ -365,7 +365,7 @@ class DeltaRun:
         w = {"a1": torch.eye(second.shape[1], dtype=torch.float64), "a2": torch.eye(second.shape[1], dtype=torch.float64),
              "A_log": a_log, "dt_bias": dt_bias}  # fmt: skip
         eye = torch.eye(self.width + second.shape[1], dtype=torch.float64)
-        spans = {"q": (0, c["k"]), "k": (c["k"], c["v"]), "v": (c["v"], c["beta"]), "b": (c["beta"], self.width)}
+        spans = {"q": (0, c["k"]), "k": (c["k"], c["v"]), "v": (c["v"], c["beta"]), "b": (c["beta"], c["beta"] + self.heads)}
         for name, (a, b) in spans.items():
             w[name] = eye[a:b]
             if name != "b":
@@ -417,12 +417,13 @@ def test_delta_rule_whole_in_portions_and_token_by_token(heads, qk_heads, dim, v
 
 
 @pytest.mark.parametrize("taps", [1, 2, 3, 4, 6])
-@pytest.mark.parametrize("heads,qk_heads,dim,vdim", [(2, 1, 16, 40), (1, 1, 130, 9), (2, 2, 100, 128)])
-def test_delta_rule_over_a_long_step(taps, heads, qk_heads, dim, vdim):
+@pytest.mark.parametrize("heads,qk_heads,dim,vdim,halves", [(2, 1, 16, 40, True), (1, 1, 130, 9, False), (2, 2, 100, 128, True),
+                                                            (2, 1, 64, 192, False), (3, 1, 128, 128, False)])  # fmt: skip
+def test_delta_rule_over_a_long_step(taps, heads, qk_heads, dim, vdim, halves):
     """Enough tokens that a warp takes a run of them: entries that start and end inside a run, entries shorter than the
     taps, entries that go on from their past: the very bits of the same tokens in short steps."""
     g = torch.Generator().manual_seed(taps)
-    run = DeltaRun(heads, qk_heads, dim, vdim, taps, slots=12)
+    run = DeltaRun(heads, qk_heads, dim, vdim, taps, slots=12, halves=halves)
     cut = [300, 1, 2, 5, 8, 260]
     starts = [20, 20, 0, 20, 0, 20]
     data = [(randn(g, 20 + n, run.width), randn(g, 20 + n, heads * dim)) for n in cut]
