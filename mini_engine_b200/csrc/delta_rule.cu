@@ -92,21 +92,37 @@ struct ConvWindow {
     __device__ __forceinline__ float input(int token, int channel) const {
         const float* src = a.proj + static_cast<size_t>(token) * a.width + channel;
         float x = 0.0f;
+#pragma unroll 4
         for (int s = 0; s < a.splits; ++s) x += src[s * a.split_stride];
         return x;
     }
-    // silu of the convolution at the entry's token number n (columns q | k | v of the projection are the channels)
-    __device__ __forceinline__ float operator()(int n, int channel) const {
-        float sum = 0.0f;
+    // silu of the convolution at the entry's token number n for COUNT channels of a lane (columns q | k | v of the
+    // projection are the channels; the ones behind `extent` are zero): channel i is first_channel + channel(i).
+    template <int COUNT, typename Channel>
+    __device__ __forceinline__ void convolve(int n, int first_channel, int extent, Channel channel, float (&y)[COUNT]) const {
+#pragma unroll
+        for (int i = 0; i < COUNT; ++i) y[i] = 0.0f;
+#pragma unroll 1
         for (int j = 0; j < a.K; ++j) {
             const int from = n - (a.K - 1) + j;
-            float x;
-            if (from >= 0) x = input(first + from, channel);
-            else if (history) x = history[static_cast<size_t>(from + a.K - 1) * a.channels + channel];
-            else continue;
-            sum = fmaf(a.conv[static_cast<size_t>(j) * a.channels + channel], x, sum);
+            if (from < 0 && !history) continue;
+            // a past input is one row of the history, an input of this step the sum of its partial sums
+            const float* src = from >= 0 ? a.proj + static_cast<size_t>(first + from) * a.width : history + static_cast<size_t>(from + a.K - 1) * a.channels;
+            const int splits = from >= 0 ? a.splits : 1;
+            float x[COUNT];
+#pragma unroll
+            for (int i = 0; i < COUNT; ++i) x[i] = 0.0f;
+#pragma unroll 2
+            for (int s = 0; s < splits; ++s)
+#pragma unroll
+                for (int i = 0; i < COUNT; ++i)
+                    if (channel(i) < extent) x[i] += src[s * a.split_stride + first_channel + channel(i)];
+#pragma unroll
+            for (int i = 0; i < COUNT; ++i)
+                if (channel(i) < extent) y[i] = fmaf(a.conv[static_cast<size_t>(j) * a.channels + first_channel + channel(i)], x[i], y[i]);
         }
-        return silu(sum);
+#pragma unroll
+        for (int i = 0; i < COUNT; ++i) y[i] = channel(i) < extent ? silu(y[i]) : 0.0f;
     }
 };
 
@@ -190,6 +206,7 @@ __device__ __forceinline__ void store_decays(const DeltaPrepArgs& a, const ConvW
     const float* logits = a.second + token * a.second_width + head * a.dim;
     for (int d = lane; d < a.dim; d += 32) {
         float z = a.dt_bias[head * a.dim + d];
+#pragma unroll 4
         for (int s = 0; s < a.second_splits; ++s) z += logits[s * a.second_stride + d];
         dst[d] = decay_of(z, rate);
     }
@@ -282,10 +299,10 @@ __global__ void __launch_bounds__(PREP_WARPS * 32, 2) delta_prepare_runs_kernel(
 template <int PER>
 __global__ void __launch_bounds__(PREP_WARPS * 32) delta_prepare_kernel(DeltaPrepArgs a) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, item = blockIdx.y;
-    const int run_begin = (blockIdx.x * PREP_WARPS + warp) * a.run, run_end = min(run_begin + a.run, a.tokens);
+    const int run_begin = (blockIdx.x * PREP_WARPS + warp) * a.run, run_end = min(run_begin + a.run, a.tokens);  // (with whole runs elsewhere: one token)
     pdl_trigger();
     pdl_wait();
-    if (run_begin >= a.tokens || (a.whole_runs_elsewhere && whole_run(a, run_begin))) return;
+    if (run_begin >= a.tokens || (a.whole_runs_elsewhere && whole_run(a, run_begin / PREP_RUN * PREP_RUN))) return;
     const bool is_qk = item < a.qk_heads;
     const int head = item - a.qk_heads;
     const float rate = is_qk ? 0.0f : -expf(a.a_log[head]);
@@ -302,16 +319,20 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) delta_prepare_kernel(DeltaPre
             const size_t token = static_cast<size_t>(first + n);
             if (is_qk) {
                 float q[PER], k[PER];
-#pragma unroll
-                for (int i = 0; i < PER; ++i) {
-                    const int d = channel_of<PER>(lane, i, a.dim);
-                    q[i] = d < a.dim ? window(n, q_column + d) : 0.0f;
-                    k[i] = d < a.dim ? window(n, k_column + d) : 0.0f;
-                }
+                const auto channel = [&](int i) { return channel_of<PER>(lane, i, a.dim); };
+                window.template convolve<PER>(n, q_column, a.dim, channel, q);
+                window.template convolve<PER>(n, k_column, a.dim, channel, k);
                 store_unit_pair<PER>(a, token, item, lane, q, k);
             } else {
                 float* dst = a.gv + (token * a.heads + head) * (a.dim + a.vdim) + a.dim;
-                for (int e = lane; e < a.vdim; e += 32) dst[e] = window(n, v_column + e);
+                for (int e = 0; e < a.vdim; e += 128) {
+                    float v[4];
+                    const auto channel = [&](int i) { return e + lane + 32 * i; };
+                    window.template convolve<4>(n, v_column, a.vdim, channel, v);
+#pragma unroll
+                    for (int i = 0; i < 4; ++i)
+                        if (channel(i) < a.vdim) dst[channel(i)] = v[i];
+                }
                 store_decays(a, window, token, head, rate, lane);
             }
         }
@@ -326,7 +347,7 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) delta_prepare_kernel(DeltaPre
 
 template <int PER>
 static int launch_delta_prepare(DeltaPrepArgs a, cudaStream_t stream) {
-    const dim3 grid((a.tokens + PREP_WARPS * a.run - 1) / (PREP_WARPS * a.run), a.qk_heads + a.heads);
+    dim3 grid((a.tokens + PREP_WARPS * a.run - 1) / (PREP_WARPS * a.run), a.qk_heads + a.heads);
     if constexpr (PER <= 4) {
         const auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
         if (a.run == PREP_RUN && a.K >= 2 && a.K <= 4 && a.splits == 1 && a.second_splits == 1 && a.dim == 32 * PER &&
@@ -336,9 +357,11 @@ static int launch_delta_prepare(DeltaPrepArgs a, cudaStream_t stream) {
                              : a.K == 3 ? launch_kernel(delta_prepare_runs_kernel<PER, 3>, grid, PREP_WARPS * 32, 0, stream, a)
                                         : launch_kernel(delta_prepare_runs_kernel<PER, 4>, grid, PREP_WARPS * 32, 0, stream, a);
             if (code) return code;
-            a.whole_runs_elsewhere = 1;
+            a.whole_runs_elsewhere = 1;  // what is left are the entries' ends: every token has warps of its own again
+            a.run = 1;
         }
     }
+    grid.x = (a.tokens + PREP_WARPS * a.run - 1) / (PREP_WARPS * a.run);
     return launch_kernel(delta_prepare_kernel<PER>, grid, PREP_WARPS * 32, 0, stream, a);
 }
 
