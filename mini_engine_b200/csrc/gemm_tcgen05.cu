@@ -97,13 +97,15 @@ __device__ __forceinline__ float plain_activation(float z, int act) {
     return act == PLAIN_RELU_SQUARED ? r * r : r;
 }
 
-// One sum of a product without a gate at element `at` of the output.
+// One sum of a product without a gate at element `at` of the output (ACT: activated, bfloat16; a form of its own of every
+// kernel, so that the plain products' epilogues carry nothing of it).
+template <bool ACT>
 __device__ __forceinline__ void store_sum(const GemmParams& p, size_t at, float v) {
-    if (p.plain_act >= 0) static_cast<__nv_bfloat16*>(p.out)[at] = __float2bfloat16_rn(plain_activation(v, p.plain_act));
+    if constexpr (ACT) static_cast<__nv_bfloat16*>(p.out)[at] = __float2bfloat16_rn(plain_activation(v, p.plain_act));
     else static_cast<float*>(p.out)[at] = v;
 }
 
-template <int BLOCK_T, bool DUAL>
+template <int BLOCK_T, bool DUAL, bool ACT>
 __global__ void __launch_bounds__(GEMM_THREADS)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, GemmParams p) {
     using C = Config<BLOCK_T, DUAL>;
@@ -227,7 +229,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
 #pragma unroll
                         for (int c = 0; c < 16; ++c) {
                             const int t = t0 + c0 + c;
-                            if (t < p.tokens) store_sum(p, base + static_cast<size_t>(t) * p.outs + n, v[c]);
+                            if (t < p.tokens) store_sum<ACT>(p, base + static_cast<size_t>(t) * p.outs + n, v[c]);
                         }
                     }
                 }
@@ -480,7 +482,7 @@ struct PairConfig {
 };
 constexpr int PAIR_T = 256;
 
-template <bool DUAL>
+template <bool DUAL, bool ACT>
 __global__ void __launch_bounds__(GEMM_THREADS)
 gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, GemmParams p) {
     using C = PairConfig<DUAL>;
@@ -596,7 +598,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid
                         const size_t base = static_cast<size_t>(split) * p.tokens * p.outs;
 #pragma unroll
                         for (int c = 0; c < 16; ++c)
-                            if (t0 + c0 + c < p.tokens) store_sum(p, base + static_cast<size_t>(t0 + c0 + c) * p.outs + n, v[c]);
+                            if (t0 + c0 + c < p.tokens) store_sum<ACT>(p, base + static_cast<size_t>(t0 + c0 + c) * p.outs + n, v[c]);
                     }
                 } else {
                     float gate[16], up[16];
@@ -676,7 +678,7 @@ __device__ __forceinline__ void pair_item(const GemmParams& p, int item, int& t0
     feature_tile = rest / wide;
 }
 
-template <bool DUAL>
+template <bool DUAL, bool ACT>
 __global__ void __launch_bounds__(PersistentConfig<DUAL>::THREADS)
 gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, GemmParams p) {
     using C = PersistentConfig<DUAL>;
@@ -805,7 +807,7 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const 
                     if (n < p.outs) {
 #pragma unroll
                         for (int c = 0; c < 16; ++c)
-                            if (t0 + c0 + c < p.tokens) store_sum(p, static_cast<size_t>(t0 + c0 + c) * p.outs + n, v[c]);
+                            if (t0 + c0 + c < p.tokens) store_sum<ACT>(p, static_cast<size_t>(t0 + c0 + c) * p.outs + n, v[c]);
                     }
                 } else {
                     float gate[16], up[16];
@@ -871,10 +873,10 @@ ME_EXPORT int me_make_tensor_map(void* out, const void* base, unsigned long long
     return 0;
 }
 
-template <int BLOCK_T, bool DUAL>
+template <int BLOCK_T, bool DUAL, bool ACT = false>
 static int launch(const CUtensorMap& map_w, const CUtensorMap& map_x, const GemmParams& p, int splits, cudaStream_t stream) {
     using C = Config<BLOCK_T, DUAL>;
-    auto kernel = gemm_tcgen05_kernel<BLOCK_T, DUAL>;
+    auto kernel = gemm_tcgen05_kernel<BLOCK_T, DUAL, ACT>;
     static SharedMemoryOptIn opt_in;
     if (const int e = opt_in(kernel, C::SMEM_BYTES)) return e;
     dim3 grid((p.tokens + BLOCK_T - 1) / BLOCK_T, (p.outs + BLOCK_N - 1) / BLOCK_N, splits);
@@ -923,13 +925,14 @@ ME_EXPORT int me_gemm_tcgen05_grouped(const void* map_w, const void* map_x, void
     p.group_rows = group_rows;
     p.act_slope = slope, p.act_limit = limit, p.act_offset = offset;
     p.plain_act = plain_act;
-    return dual_row_offset > 0 ? launch<128, true>(w, x, p, 1, stream) : launch<128, false>(w, x, p, 1, stream);
+    if (dual_row_offset > 0) return launch<128, true>(w, x, p, 1, stream);
+    return plain_act >= 0 ? launch<128, false, true>(w, x, p, 1, stream) : launch<128, false>(w, x, p, 1, stream);
 }
 
-template <bool DUAL>
+template <bool DUAL, bool ACT = false>
 static int launch_pair(const CUtensorMap& map_w, const CUtensorMap& map_x, const GemmParams& p, cudaStream_t stream, int splits = 1) {
     using C = PairConfig<DUAL>;
-    auto kernel = gemm_tcgen05_pair_kernel<DUAL>;
+    auto kernel = gemm_tcgen05_pair_kernel<DUAL, ACT>;
     static SharedMemoryOptIn opt_in;
     if (const int e = opt_in(kernel, C::SMEM_BYTES)) return e;
     int device = 0, sms = 0;
@@ -981,10 +984,10 @@ ME_EXPORT int me_gemm_tcgen05_pair_split(const void* map_w, const void* map_x, f
     return launch_pair<false>(w, x, p, stream, splits);
 }
 
-template <bool DUAL>
+template <bool DUAL, bool ACT = false>
 static int launch_persistent(const CUtensorMap& map_w, const CUtensorMap& map_x, const GemmParams& p, int group, cudaStream_t stream) {
     using C = PersistentConfig<DUAL>;
-    auto kernel = gemm_tcgen05_persistent_kernel<DUAL>;
+    auto kernel = gemm_tcgen05_persistent_kernel<DUAL, ACT>;
     static SharedMemoryOptIn opt_in;
     if (const int e = opt_in(kernel, C::SMEM_BYTES)) return e;
     int device = 0, sms = 0;
@@ -1001,7 +1004,7 @@ static int launch_persistent(const CUtensorMap& map_w, const CUtensorMap& map_x,
     q.full_tiles = tiles / pairs * pairs;
     q.tail_parts = 1;
     while (q.tail_parts < 4 && (tiles - q.full_tiles) * q.tail_parts * 2 <= pairs) q.tail_parts *= 2;
-    if (tiles <= pairs) return launch_pair<DUAL>(map_w, map_x, p, stream);  // one tile per pair: nothing to overlap
+    if (tiles <= pairs) return launch_pair<DUAL, ACT>(map_w, map_x, p, stream);  // one tile per pair: nothing to overlap
     q.items = q.full_tiles + (tiles - q.full_tiles) * q.tail_parts;
     const int clusters = q.items < pairs ? q.items : pairs;
     cudaLaunchConfig_t config = {};
@@ -1032,7 +1035,7 @@ ME_EXPORT int me_gemm_tcgen05_persistent(const void* map_w, const void* map_x, v
     memcpy(&x, map_x, sizeof(x));
     GemmParams p{out, tokens, outs, (inner + BLOCK_K - 1) / BLOCK_K, 0, 0, 0, 0, 1, 0, 0, 0};
     p.plain_act = plain_act;
-    return launch_persistent<false>(w, x, p, group, stream);
+    return plain_act >= 0 ? launch_persistent<false, true>(w, x, p, group, stream) : launch_persistent<false>(w, x, p, group, stream);
 }
 
 // act[t][n] (bfloat16) = silu(x . w[n]) * (x . w[dual_row_offset + n]) by persistent CTA pairs.
