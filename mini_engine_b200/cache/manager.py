@@ -52,6 +52,7 @@ class GroupSpec:
     num_blocks: int | None = None
     shareable: bool = True
     keep_first: int = 0  # with a window: the first tokens of a sequence stay readable, their pages are never given back
+    chunk: int | None = None  # with a window of that size: only keys of the next query's own chunk of positions are read
 
 
 @dataclass(frozen=True)
@@ -207,6 +208,8 @@ class CacheManager:
         it too and are needed all the same: see :meth:`_kept_pages`.)"""
         if group.window is None:
             return 0
+        if group.chunk is not None:  # the next query's chunk starts at or behind its window
+            return num_computed // group.chunk * group.chunk // self.block_size
         return max(0, num_computed - group.window + 1) // self.block_size
 
     def _kept_pages(self, group: GroupSpec) -> int:

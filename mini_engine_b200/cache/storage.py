@@ -91,8 +91,8 @@ def group_names(specs: list[PagedCacheSpec], pages: list[int]) -> list[GroupSpec
     return [
         GroupSpec(
             f"kv{i}:{s.kv_heads}x{s.head_dim}" + (f"+{s.v_dim}" if s.v_dim not in (0, s.head_dim) else "") + ("=v" if s.v_dim == 0 else "")
-            + (f":w{s.window}" if s.window else "") + (f":first{s.keep_first}" if s.window and s.keep_first else ""),
-            s.window, count, keep_first=s.keep_first if s.window else 0,
+            + (f":w{s.window}" if s.window else "") + (f":first{s.keep_first}" if s.window and s.keep_first else "") + (":chunk" if s.chunk else ""),
+            s.window, count, keep_first=s.keep_first if s.window else 0, chunk=s.chunk,
         )
         for i, (s, count) in enumerate(zip(specs, pages))
     ]  # fmt: skip

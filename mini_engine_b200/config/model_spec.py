@@ -68,11 +68,15 @@ class OrderEntry:
     ``layer`` indexes :attr:`ModelSpec.layers`; the same index may appear in several
     entries (the weights are then shared, each entry keeps a cache of its own).
     ``cache_of`` is ``None`` when the entry owns its cache, else the index of an *earlier
-    entry* whose cache this entry's mixer reads without writing to it.
+    entry* whose cache this entry's mixer reads without writing to it.  ``junction`` indexes
+    :attr:`ModelSpec.junctions`: what happens to the residual stream in front of this entry, as the junction's turn
+    number ``turn`` (the pass of a loop over layers, say).
     """
 
     layer: int
     cache_of: int | None = None
+    junction: int | None = None
+    turn: int = 0
 
 
 @dataclass(frozen=True)
@@ -84,11 +88,14 @@ class ModelSpec:
     order: tuple[OrderEntry, ...]
     final_norm: PartSpec
     head: PartSpec
+    junctions: tuple[PartSpec, ...] = ()
 
     def __post_init__(self) -> None:
         for position, entry in enumerate(self.order):
             if not 0 <= entry.layer < len(self.layers):
                 raise ValueError(f"order[{position}] names layer {entry.layer}, which does not exist")
+            if entry.junction is not None and not 0 <= entry.junction < len(self.junctions):
+                raise ValueError(f"order[{position}] names junction {entry.junction}, which does not exist")
             if entry.cache_of is not None:
                 if not 0 <= entry.cache_of < position:
                     raise ValueError(

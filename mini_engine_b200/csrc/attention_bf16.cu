@@ -54,7 +54,19 @@ struct AttnParams {
     const float* slopes = nullptr;       // [heads] slope_h of a distance bias slope_h * (p - j) taken off the scaled scores, or null
     const float* sink_values = nullptr;  // [heads] with sink: the silent participant's score (zero when null)
     float cap_log2 = 0.0f;  // > 0: a scaled score s (log2 domain) becomes cap * tanh(s / cap); cap * log2(e) here
+    int chunk = 0;          // > 0: a query sees keys of its own chunk of positions only, from floor(p / chunk) * chunk on
+    const float* sigmoid_bias = nullptr;  // [heads] a key's weight is sigmoid(score + bias), not normalised, in the place of a softmax; or null
 };
+
+// The first key that the query at `position` sees.
+__device__ __forceinline__ int lowest_key(const AttnParams& p, int position) {
+    const int behind = p.window > 0 ? max(position - p.window + 1, 0) : 0;
+    return p.chunk > 0 ? max(behind, position / p.chunk * p.chunk) : behind;
+}
+// Weights without a softmax keep 0 as the reference of their (unscaled) sums: partial results then merge as plain sums.
+__device__ __forceinline__ float first_max(const AttnParams& p) { return p.sigmoid_bias ? 0.0f : -INFINITY; }
+__device__ __forceinline__ float weight_bias_of(const AttnParams& p, int head) { return p.sigmoid_bias ? p.sigmoid_bias[head] * LOG2E : 0.0f; }
+__device__ __forceinline__ float sigmoid_log2(float x_log2) { return __fdividef(1.0f, 1.0f + exp2f(-x_log2)); }
 
 // The cap on a scaled score, both in the log2 domain (their quotient is the natural one).  The hardware's tanh is good
 // to about 2^-11 of its value, which on scores of a few units is below what bfloat16 probabilities resolve.
@@ -68,6 +80,10 @@ __device__ __forceinline__ float capped_score(float s_log2, float cap_log2) {
 // What the silent participant adds to a denominator that is relative to `max_log2` (scores in the log2 domain).
 __device__ __forceinline__ float sink_term(const AttnParams& p, float max_log2, int head) {
     return p.sink ? exp2f((p.sink_values ? p.sink_values[head] * LOG2E : 0.0f) - max_log2) : 0.0f;
+}
+// What a head's weighted sum is multiplied by at the end.
+__device__ __forceinline__ float inverse_of(const AttnParams& p, float denom, float max_log2, int head) {
+    return p.sigmoid_bias ? 1.0f : 1.0f / (denom + sink_term(p, max_log2, head));
 }
 // The multiplier of element `col` of one (token, head)'s output.
 __device__ __forceinline__ float gate_of(const AttnParams& p, size_t token, int head, int col) {
@@ -144,13 +160,13 @@ __device__ __forceinline__ void accumulate_pv(float (&acc)[D / 8][4], const floa
 // Masks the scores of one tile, updates the running maximum and sum of the thread's two rows
 // (row `g` and row `g + 8` of the warp's 16) and turns the scores into probabilities.
 // `row_pos[i]` is the absolute position of row i's query; keys are visible in
-// [row_pos - window + 1, row_pos] (window <= 0: from 0).  `row_slope[i]` (log2 domain) times the distance to the
-// key is taken off row i's scaled scores.
+// [row_lowest, row_pos].  `row_slope[i]` (log2 domain) times the distance to the
+// key is taken off row i's scaled scores.  With `sigmoid` the weights are sigmoid(score + row_bias) and nothing is rescaled.
 template <int D, int KEYS>
 __device__ __forceinline__ void softmax_step(float (&s)[KEYS / 8][4], float (&acc)[D / 8][4], float (&row_max)[2],
                                              float (&row_sum)[2], const int (&row_pos)[2], int first_key,
-                                             int window, float scale_log2, int lane, const float (&row_slope)[2],
-                                             float cap_log2 = 0.0f) {
+                                             const int (&row_lowest)[2], float scale_log2, int lane, const float (&row_slope)[2],
+                                             float cap_log2, bool sigmoid, const float (&row_bias)[2]) {
     const int col0 = first_key + 2 * (lane & 3);
     float tile_max[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -159,10 +175,17 @@ __device__ __forceinline__ void softmax_step(float (&s)[KEYS / 8][4], float (&ac
         for (int i = 0; i < 4; ++i) {
             const int key = col0 + n * 8 + (i & 1);
             const int r = i >> 1;
-            const bool visible = key <= row_pos[r] && (window <= 0 || key > row_pos[r] - window);
+            const bool visible = key <= row_pos[r] && key >= row_lowest[r];
             s[n][i] = visible ? capped_score(s[n][i] * scale_log2, cap_log2) - row_slope[r] * static_cast<float>(row_pos[r] - key) : -INFINITY;
             tile_max[r] = fmaxf(tile_max[r], s[n][i]);
         }
+    if (sigmoid) {  // uniform for the launch
+#pragma unroll
+        for (int n = 0; n < KEYS / 8; ++n)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) s[n][i] = s[n][i] == -INFINITY ? 0.0f : sigmoid_log2(s[n][i] + row_bias[i >> 1]);
+        return;
+    }
     float rescale[2], base[2];
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
@@ -211,7 +234,7 @@ __global__ void __launch_bounds__(ATTN_THREADS) attention_portions_kernel(AttnPa
     const int rows_valid = min(BLOCK_M, new_tokens - q_block * BLOCK_M);
     const int pos0 = p.context_lens[entry] - new_tokens + q_block * BLOCK_M;  // position of row 0
     const int last_key = pos0 + rows_valid - 1;
-    const int lowest = p.window > 0 ? max(pos0 - p.window + 1, 0) : 0;
+    const int lowest = lowest_key(p, pos0);
     const int kv_head = head / (p.heads / p.kv_heads);
     const int* table = p.block_table + static_cast<size_t>(entry) * p.table_width;
     const int my_chunk = threadIdx.x % CHUNKS, my_row = threadIdx.x / CHUNKS;
@@ -250,9 +273,10 @@ __global__ void __launch_bounds__(ATTN_THREADS) attention_portions_kernel(AttnPa
     for (int n = 0; n < D / 8; ++n)
 #pragma unroll
         for (int i = 0; i < 4; ++i) acc[n][i] = 0.0f;
-    float row_max[2] = {-INFINITY, -INFINITY}, row_sum[2] = {0.0f, 0.0f};
+    float row_max[2] = {first_max(p), first_max(p)}, row_sum[2] = {0.0f, 0.0f};
     const int row_pos[2] = {pos0 + warp * 16 + (lane >> 2), pos0 + warp * 16 + (lane >> 2) + 8};
-    const float row_slope[2] = {slope_of(p, head), slope_of(p, head)};
+    const float row_slope[2] = {slope_of(p, head), slope_of(p, head)}, row_bias[2] = {weight_bias_of(p, head), weight_bias_of(p, head)};
+    const int row_lowest[2] = {lowest_key(p, row_pos[0]), lowest_key(p, row_pos[1])};
 
     for (int tile = first_tile; tile <= last_tile; ++tile) {
         const int s = (tile - first_tile) & 1;
@@ -274,7 +298,7 @@ __global__ void __launch_bounds__(ATTN_THREADS) attention_portions_kernel(AttnPa
         const __nv_bfloat16* k_tile = kv_tiles + s * 2 * BLOCK_KEYS * D;
         float scores[BLOCK_KEYS / 8][4];
         scores_tile<D, BLOCK_KEYS>(scores, q_frag, k_tile, lane);
-        softmax_step<D, BLOCK_KEYS>(scores, acc, row_max, row_sum, row_pos, tile * BLOCK_KEYS, p.window, p.scale_log2, lane, row_slope, p.cap_log2);
+        softmax_step<D, BLOCK_KEYS>(scores, acc, row_max, row_sum, row_pos, tile * BLOCK_KEYS, row_lowest, p.scale_log2, lane, row_slope, p.cap_log2, p.sigmoid_bias != nullptr, row_bias);
         accumulate_pv<D, BLOCK_KEYS>(acc, scores, k_tile + BLOCK_KEYS * D, lane);
         __syncthreads();  // the next iteration's prefetch overwrites the other stage's reader
     }
@@ -288,7 +312,7 @@ __global__ void __launch_bounds__(ATTN_THREADS) attention_portions_kernel(AttnPa
     for (int r = 0; r < 2; ++r) {
         const int row = warp * 16 + (lane >> 2) + r * 8;
         if (row >= rows_valid) continue;
-        const float inv = 1.0f / (row_sum[r] + sink_term(p, row_max[r], head));
+        const float inv = inverse_of(p, row_sum[r], row_max[r], head);
         const size_t token = static_cast<size_t>(token0 + q_block * BLOCK_M + row);
         __nv_bfloat16* dst = p.out + (token * p.heads + head) * D;
         const float whole = p.gate_width == 1 ? inv * gate_of(p, token, head, 0) : inv;
@@ -345,7 +369,7 @@ __global__ void __launch_bounds__(ATTN_THREADS, 3) attention_decode_kernel(AttnP
     pdl_wait();
     const int entry = p.entry_ids ? p.entry_ids[blockIdx.z] : blockIdx.z;
     const int position = p.context_lens[entry] - 1;  // the query's position; it sees keys <= position
-    const int lowest = p.window > 0 ? max(position - p.window + 1, 0) : 0;
+    const int lowest = lowest_key(p, position);
     const int span = p.tiles_per_cta * DECODE_CHUNK;
     const int cta_start = split * span;
     if (cta_start > position || cta_start + span <= lowest) return;
@@ -389,11 +413,13 @@ __global__ void __launch_bounds__(ATTN_THREADS, 3) attention_decode_kernel(AttnP
     for (int n = 0; n < D / 8; ++n)
 #pragma unroll
         for (int i = 0; i < 4; ++i) acc[n][i] = 0.0f;
-    float row_max[2] = {-INFINITY, -INFINITY}, row_sum[2] = {0.0f, 0.0f};
+    float row_max[2] = {first_max(p), first_max(p)}, row_sum[2] = {0.0f, 0.0f};
     uint32_t q_frag[D / 16][4];
     const int row_pos[2] = {position, position};
     const int row_head[2] = {kv_head * group + min(lane >> 2, group - 1), kv_head * group + min((lane >> 2) + 8, group - 1)};
     const float row_slope[2] = {slope_of(p, row_head[0]), slope_of(p, row_head[1])};
+    const float row_bias[2] = {weight_bias_of(p, row_head[0]), weight_bias_of(p, row_head[1])};
+    const int row_lowest[2] = {lowest, lowest};
 
 #pragma unroll 1
     for (int t = 0; t < tiles; ++t) {
@@ -413,7 +439,7 @@ __global__ void __launch_bounds__(ATTN_THREADS, 3) attention_decode_kernel(AttnP
         const int first_key = cta_start + t * DECODE_CHUNK + warp * KEYS;
         float scores[KEYS / 8][4];
         scores_tile<D, KEYS>(scores, q_frag, k_tile, lane);
-        softmax_step<D, KEYS>(scores, acc, row_max, row_sum, row_pos, first_key, p.window, p.scale_log2, lane, row_slope, p.cap_log2);
+        softmax_step<D, KEYS>(scores, acc, row_max, row_sum, row_pos, first_key, row_lowest, p.scale_log2, lane, row_slope, p.cap_log2, p.sigmoid_bias != nullptr, row_bias);
         __syncwarp();  // every lane has read the keys: the next tile's keys may overwrite them
         if (more) issue(k_tile, p.k_pages, offset_next);
         cp_async_commit();
@@ -545,7 +571,7 @@ __device__ __forceinline__ void merge_head(const AttnParams& p, int entry, int h
     }
     const int token = p.cu_tokens[entry];
     __nv_bfloat16* dst = p.out + (static_cast<size_t>(token) * p.heads + head) * D + lane * PER_LANE;
-    float inv = 1.0f / (denom + sink_term(p, total_max, head));
+    float inv = inverse_of(p, denom, total_max, head);
     if (p.gate_width == 1) inv *= gate_of(p, token, head, 0);
 #pragma unroll
     for (int i = 0; i < PER_LANE; i += 2) {
@@ -565,7 +591,7 @@ __global__ void __launch_bounds__(128) attention_decode_merge_kernel(AttnParams 
     const int listed = item / p.heads, head = item % p.heads;
     const int entry = p.entry_ids ? p.entry_ids[listed] : listed;
     const int position = p.context_lens[entry] - 1;
-    const int lowest = p.window > 0 ? max(position - p.window + 1, 0) : 0;
+    const int lowest = lowest_key(p, position);
     const int span = p.tiles_per_cta * DECODE_CHUNK;
     int first_slot, last_slot;
     decode_slot_range(p, position, lowest, span, first_slot, last_slot);
@@ -637,7 +663,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __g
     const int* table = p.block_table + static_cast<size_t>(entry) * p.table_width;
     const int position = p.context_lens[entry] - 1;  // the query's position; it sees keys <= position
     const int token = p.cu_tokens[entry];
-    const int lowest = p.window > 0 ? max(position - p.window + 1, 0) : 0;
+    const int lowest = lowest_key(p, position);
     const int group = p.heads / p.kv_heads;
     // This CTA's tiles [tile, tile_end) among the request's visible ones.
     const int lowest_tile = lowest / TILE_KEYS, tile_count = position / TILE_KEYS - lowest_tile + 1;
@@ -725,9 +751,11 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __g
     for (int i = 0; i < D / 16; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) acc[i][j] = 0.0f;
-    float row_max[2] = {-INFINITY, -INFINITY}, row_sum[2] = {0.0f, 0.0f};  // of heads 2 (lane % 4) and + 1
+    float row_max[2] = {first_max(p), first_max(p)}, row_sum[2] = {0.0f, 0.0f};  // of heads 2 (lane % 4) and + 1
     const float head_slope[2] = {slope_of(p, kv_head * group + min(2 * (lane & 3), group - 1)),
                                  slope_of(p, kv_head * group + min(2 * (lane & 3) + 1, group - 1))};
+    const float head_bias[2] = {weight_bias_of(p, kv_head * group + min(2 * (lane & 3), group - 1)),
+                                weight_bias_of(p, kv_head * group + min(2 * (lane & 3) + 1, group - 1))};
     uint32_t phase = 0;
     bool failed = false;
 
@@ -765,6 +793,11 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __g
             for (int j = 0; j < 2; ++j) {
                 const float a = seen0 ? capped_score(s[j] * p.scale_log2, p.cap_log2) - head_slope[j] * static_cast<float>(position - key0) : -INFINITY;
                 const float b = seen1 ? capped_score(s[j + 2] * p.scale_log2, p.cap_log2) - head_slope[j] * static_cast<float>(position - key0 - 8) : -INFINITY;
+                if (p.sigmoid_bias) {  // uniform for the launch
+                    prob[j] = seen0 ? sigmoid_log2(a + head_bias[j]) : 0.0f, prob[j + 2] = seen1 ? sigmoid_log2(b + head_bias[j]) : 0.0f;
+                    rescale[j] = 1.0f;
+                    continue;
+                }
                 float tile_max = fmaxf(a, b);
                 tile_max = fmaxf(tile_max, __shfl_xor_sync(0xffffffffu, tile_max, 4));
                 tile_max = fmaxf(tile_max, __shfl_xor_sync(0xffffffffu, tile_max, 8));
@@ -865,7 +898,8 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __g
         if (!direct)
             p.partials[((static_cast<size_t>(entry) * p.heads + head) * p.max_splits + split) * STRIDE + col] = value;
         else if (col < D) {
-            const float result = value / (denom + sink_term(p, total_max, head)) * gate_of(p, token, head, col);
+            const float whole = p.sigmoid_bias ? value : value / (denom + sink_term(p, total_max, head));
+            const float result = whole * gate_of(p, token, head, col);
             p.out[(static_cast<size_t>(token) * p.heads + head) * D + col] = __float2bfloat16(result);
         }
     }
@@ -897,7 +931,7 @@ __global__ void __launch_bounds__(128) attention_decode_tma_merge_kernel(AttnPar
     const int listed = item / p.heads, head = item % p.heads;
     const int entry = p.entry_ids ? p.entry_ids[listed] : listed;
     const int position = p.context_lens[entry] - 1;
-    const int lowest = p.window > 0 ? max(position - p.window + 1, 0) : 0;
+    const int lowest = lowest_key(p, position);
     const int tile_count = position / TILE_KEYS - lowest / TILE_KEYS + 1;
     const int per_cta = max((tile_count + p.max_splits - 1) / p.max_splits, TMA_MIN_TILES);
     merge_head<D>(p, entry, head, 0, (tile_count + per_cta - 1) / per_cta - 1, lane);
@@ -960,14 +994,14 @@ ME_EXPORT int me_attention_portions_bf16(const void* q, const void* k_pages, con
                                          int entries, int max_new_tokens, int heads, int kv_heads, int head_dim,
                                          int page_size, int table_width, int window, const int* entry_ids,
                                          int sink, const float* gate, int gate_width, const float* slopes,
-                                         const float* sink_values, float softcap, cudaStream_t stream) {
+                                         const float* sink_values, float softcap, int chunk, const float* sigmoid_bias, cudaStream_t stream) {
     if (entries <= 0) return 0;
     if (!sizes_ok(head_dim, heads, kv_heads)) return ME_ERR_UNSUPPORTED;
     AttnParams p{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_pages),
                  static_cast<const __nv_bfloat16*>(v_pages), block_table, cu_tokens, context_lens,
                  static_cast<__nv_bfloat16*>(out), nullptr, nullptr, entry_ids, scale * LOG2E, heads, kv_heads,
                  page_size, table_width, window, 0, shift_of(page_size), 1, sink, gate, gate_width, slopes, sink_values,
-                 softcap * LOG2E};
+                 softcap * LOG2E, chunk, sigmoid_bias};
     return head_dim == 128 ? launch_portions<128>(p, entries, max_new_tokens, stream)
                            : launch_portions<64>(p, entries, max_new_tokens, stream);
 }
@@ -984,7 +1018,7 @@ ME_EXPORT int me_attention_decode_bf16_tiled(const void* q, const void* k_pages,
                                              int tiles_per_cta, int heads, int kv_heads, int head_dim, int page_size,
                                              int table_width, int window, const int* entry_ids, int sink,
                                              const float* gate, int gate_width, const float* slopes,
-                                             const float* sink_values, float softcap, cudaStream_t stream) {
+                                             const float* sink_values, float softcap, int chunk, const float* sigmoid_bias, cudaStream_t stream) {
     if (entries <= 0) return 0;
     if (!sizes_ok(head_dim, heads, kv_heads) || heads / kv_heads > 16 || max_splits < 1) return ME_ERR_UNSUPPORTED;
     if (tiles_per_cta < 1 || tiles_per_cta > MAX_DECODE_TILES) return ME_ERR_ARGUMENT;
@@ -992,7 +1026,7 @@ ME_EXPORT int me_attention_decode_bf16_tiled(const void* q, const void* k_pages,
                  static_cast<const __nv_bfloat16*>(v_pages), block_table, cu_tokens, context_lens,
                  static_cast<__nv_bfloat16*>(out), partials, counters, entry_ids, scale * LOG2E, heads, kv_heads,
                  page_size, table_width, window, max_splits, shift_of(page_size), tiles_per_cta, sink, gate, gate_width,
-                 slopes, sink_values, softcap * LOG2E};
+                 slopes, sink_values, softcap * LOG2E, chunk, sigmoid_bias};
     return head_dim == 128 ? launch_decode<128>(p, entries, stream) : launch_decode<64>(p, entries, stream);
 }
 
@@ -1008,8 +1042,8 @@ ME_EXPORT int me_attention_decode_bf16_tma(const void* k_map, const void* v_map,
                                            int* counters, float scale, int entries, int splits, int warps, int heads,
                                            int kv_heads, int head_dim, int page_size, int table_width, int window,
                                            const int* entry_ids, int sink, const float* gate, int gate_width,
-                                           const float* slopes, const float* sink_values, float softcap,
-                                           cudaStream_t stream) {
+                                           const float* slopes, const float* sink_values, float softcap, int chunk,
+                                           const float* sigmoid_bias, cudaStream_t stream) {
     if (entries <= 0) return 0;
     if (!sizes_ok(head_dim, heads, kv_heads) || heads / kv_heads > 8) return ME_ERR_UNSUPPORTED;
     if (shift_of(page_size) < 3) return ME_ERR_UNSUPPORTED;
@@ -1018,7 +1052,7 @@ ME_EXPORT int me_attention_decode_bf16_tma(const void* k_map, const void* v_map,
     AttnParams p{static_cast<const __nv_bfloat16*>(q), nullptr, nullptr, block_table, cu_tokens, context_lens,
                  static_cast<__nv_bfloat16*>(out), partials, counters, entry_ids, scale * LOG2E, heads, kv_heads,
                  page_size, table_width, window, splits, shift_of(page_size), 0, sink, gate, gate_width, slopes, sink_values,
-                 softcap * LOG2E};
+                 softcap * LOG2E, chunk, sigmoid_bias};
     CUtensorMap maps[2];
     memcpy(&maps[0], k_map, sizeof(CUtensorMap));
     memcpy(&maps[1], v_map, sizeof(CUtensorMap));
@@ -1046,7 +1080,7 @@ ME_EXPORT int me_attention_decode_bf16(const void* q, const void* k_pages, const
                                        int page_size, int table_width, int window, cudaStream_t stream) {
     return me_attention_decode_bf16_tiled(q, k_pages, v_pages, block_table, cu_tokens, context_lens, out, partials,
                                           nullptr, scale, entries, max_splits, 1, heads, kv_heads, head_dim, page_size,
-                                          table_width, window, nullptr, 0, nullptr, 1, nullptr, nullptr, 0.0f, stream);
+                                          table_width, window, nullptr, 0, nullptr, 1, nullptr, nullptr, 0.0f, 0, nullptr, stream);
 }
 
 // ------------------------------------------------- decode attention without allocation

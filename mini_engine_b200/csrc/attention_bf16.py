@@ -6,8 +6,8 @@
   the one that gathers keys row by row;
 * otherwise, head size 128, pages of 8 to 128 tokens and a portion of at least 32 tokens in the
   batch: the tcgen05 kernel (both products on the tensor cores with accumulators in tensor memory,
-  keys and values fetched by TMA page by page; with a window, a distance bias, a silent participant
-  or a gate, its form of one query head per CTA that knows them);
+  keys and values fetched by TMA page by page; with a window, chunks, a distance bias, a silent participant
+  or a gate, its form of one query head per CTA that knows them; with sigmoid weights, a third form);
 * otherwise: the mma.sync portions kernel, for any mix of portion lengths.
 
 Head sizes 64 and 128 are taken; other sizes use the generic kernel.
@@ -41,7 +41,7 @@ def _tc_library():
         import ctypes
 
         lib = load_library("attention_tcgen05")
-        lib.me_attention_tcgen05.argtypes = [c_void_p] * 7 + [c_float] + [c_int] * 7 + [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p]
+        lib.me_attention_tcgen05.argtypes = [c_void_p] * 7 + [c_float] + [c_int] * 7 + [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p]
         lib.me_attention_tcgen05.restype = c_int
         lib.me_attention_take_error.argtypes = [ctypes.POINTER(c_int)]
         lib.me_attention_take_error.restype = c_int
@@ -113,11 +113,11 @@ def _library():
         import ctypes
 
         lib = load_library("attention_bf16")
-        lib.me_attention_portions_bf16.argtypes = [c_void_p] * 7 + [c_float] + [c_int] * 8 + [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p]
+        lib.me_attention_portions_bf16.argtypes = [c_void_p] * 7 + [c_float] + [c_int] * 8 + [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p]
         lib.me_attention_portions_bf16.restype = c_int
-        lib.me_attention_decode_bf16_tiled.argtypes = [c_void_p] * 9 + [c_float] + [c_int] * 9 + [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p]
+        lib.me_attention_decode_bf16_tiled.argtypes = [c_void_p] * 9 + [c_float] + [c_int] * 9 + [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p]
         lib.me_attention_decode_bf16_tiled.restype = c_int
-        lib.me_attention_decode_bf16_tma.argtypes = [c_void_p] * 9 + [c_float] + [c_int] * 9 + [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p]
+        lib.me_attention_decode_bf16_tma.argtypes = [c_void_p] * 9 + [c_float] + [c_int] * 9 + [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p]
         lib.me_attention_decode_bf16_tma.restype = c_int
         lib.me_attention_bf16_take_error.argtypes = [ctypes.POINTER(c_int)]
         lib.me_attention_bf16_take_error.restype = c_int
@@ -189,7 +189,8 @@ def decode_splits(max_context_len: int, tiles_per_cta: int = 1) -> int:
 def paged_attention(q, k_pages, v_pages, block_table, ctx, out, heads, kv_heads, head_dim, scale, window,
                     decode_warps: int | None = None, decode_splits_per_pair: int | None = None, sink: bool = False,
                     gate: torch.Tensor | None = None, slopes: torch.Tensor | None = None,
-                    sink_values: torch.Tensor | None = None, softcap: float = 0.0) -> None:
+                    sink_values: torch.Tensor | None = None, softcap: float = 0.0, chunk: int = 0,
+                    sigmoid_bias: torch.Tensor | None = None) -> None:
     """Attention of the batch's new tokens.  Entries that bring one token take the split decode
     kernel, the others a portions kernel; a step that holds both kinds is two launches, each over
     its own list of entries.  ``decode_warps`` (6 or 8) and ``decode_splits_per_pair`` pin the form
@@ -199,7 +200,10 @@ def paged_attention(q, k_pages, v_pages, block_table, ctx, out, heads, kv_heads,
     ``sink_values[h]`` (float32 ``[heads]``); ``gate`` (float32 ``[T, heads]`` or ``[T, heads * head_dim]``): a
     multiplier on every head's output, or on every element; ``slopes`` (float32 ``[heads]``): ``slopes[h] * (p - j)``
     is taken off the scaled score of query ``p`` and key ``j``; ``softcap`` > 0: a scaled score ``s`` becomes ``softcap *
-    tanh(s / softcap)`` (before the distance bias).  Every kernel knows all of them."""
+    tanh(s / softcap)`` (before the distance bias); ``chunk`` > 0: a query at ``p`` sees keys from ``p // chunk * chunk`` on;
+    ``sigmoid_bias`` (float32 ``[heads]``): a key's weight is ``sigmoid(s + bias_h)``, not normalised, in the place of a
+    softmax (without a sink).  Every kernel knows all of them, but the tcgen05 one takes sigmoid weights only without a gate,
+    a distance bias and a cap."""
     for name, t in (("q", q), ("out", out), ("k_pages", k_pages), ("v_pages", v_pages)):
         if t.dtype != torch.bfloat16 or not t.is_contiguous():
             raise ops.KernelError(f"{name} must be contiguous bfloat16")
@@ -210,12 +214,15 @@ def paged_attention(q, k_pages, v_pages, block_table, ctx, out, heads, kv_heads,
         if gate.dtype != torch.float32 or not gate.is_contiguous() or gate.shape not in ((q.shape[0], heads), (q.shape[0], heads * head_dim)):
             raise ops.KernelError("gate must be contiguous float32 [tokens, heads] or [tokens, heads * head_dim]")
         gate_width = gate.shape[1] // heads
-    for name, vector in (("slopes", slopes), ("sink_values", sink_values)):
+    if sigmoid_bias is not None and (sink or sink_values is not None):
+        raise ops.KernelError("weights without a softmax have no silent participant")
+    for name, vector in (("slopes", slopes), ("sink_values", sink_values), ("sigmoid_bias", sigmoid_bias)):
         if vector is not None and (vector.dtype != torch.float32 or not vector.is_contiguous() or vector.shape != (heads,)):
             raise ops.KernelError(f"{name} must be contiguous float32 [heads]")
     sink_flag, gate_ptr = (1 if (sink or sink_values is not None) else 0), (None if gate is None else gate.data_ptr())
     options = (sink_flag, gate_ptr, gate_width, None if slopes is None else slopes.data_ptr(),
-               None if sink_values is None else sink_values.data_ptr(), float(softcap or 0.0))  # fmt: skip
+               None if sink_values is None else sink_values.data_ptr(), float(softcap or 0.0), int(chunk),
+               None if sigmoid_bias is None else sigmoid_bias.data_ptr())  # fmt: skip
     stream = _ops_stream()
     page_size, width = k_pages.shape[2], block_table.shape[1]
     common = (q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(), ctx.cu_tokens.data_ptr(),
@@ -257,7 +264,9 @@ def paged_attention(q, k_pages, v_pages, block_table, ctx, out, heads, kv_heads,
                 head_dim, page_size, width, window, ids_ptr, *options, stream,
             )  # fmt: skip
             ops._check(code, "attention_decode_bf16")
-        elif tensor_memory_kernel_takes(head_dim, page_size, window, longest):
+        elif tensor_memory_kernel_takes(head_dim, page_size, window, longest) and not (
+            sigmoid_bias is not None and (gate is not None or slopes is not None or softcap)
+        ):
             code = _tc_library().me_attention_tcgen05(
                 _query_map(q), _page_map(k_pages), _page_map(v_pages), *common[3:], scale, entries, longest, heads,
                 kv_heads, head_dim, page_size, width, ids_ptr, window, *options, stream,

@@ -11,7 +11,9 @@
 // on the output (`gate`, float32 [tokens][heads][gate_width] with gate_width 1, one per head, or value_dim, one per
 // element); a distance bias that is linear in the distance (`slopes`, one per head: s -= slope_h * (p - j), after
 // the scale); a cap on the scaled scores (`softcap`: s becomes softcap * tanh(s / softcap)); and values that are the first value_dim elements of the key rows (`value_stride`: elements between
-// two value rows; pass the key pages as value pages and head_dim as the stride).
+// two value rows; pass the key pages as value pages and head_dim as the stride); chunks (`chunk`: the query at position p sees
+// keys from floor(p / chunk) * chunk on); and weights without a softmax (`sigmoid_bias`, one per head: the weight of a visible
+// key is sigmoid(s + bias_h), not normalised over the keys).
 //
 // Keys are visited in tiles of 32 whose boundaries are multiples of 32 in *absolute position*
 // and are combined in ascending order, so the arithmetic of a query depends only on its own
@@ -35,6 +37,8 @@ struct AttnArgs {
     const float* slopes;       // [heads] or null
     const float* sink_values;  // [heads] or null (with sink: the silent participant's score, zero when null)
     float softcap;             // > 0: the scaled score s becomes softcap * tanh(s / softcap)
+    int chunk;                  // > 0: keys of the query's own chunk of positions only
+    const float* sigmoid_bias;  // [heads] weights sigmoid(s + bias) in the place of a softmax, or null
 };
 
 constexpr int ATTN_WARPS = 4;
@@ -64,7 +68,10 @@ __global__ void __launch_bounds__(ATTN_WARPS * 32) paged_attention_generic_kerne
 
     const float slope = a.slopes ? a.slopes[head] : 0.0f;
     const size_t v_stride = static_cast<size_t>(a.value_stride);
-    const int lowest = a.window > 0 ? max(position - a.window + 1, 0) : 0;
+    int lowest = a.window > 0 ? max(position - a.window + 1, 0) : 0;
+    if (a.chunk > 0) lowest = max(lowest, position / a.chunk * a.chunk);
+    const bool sigmoid = a.sigmoid_bias != nullptr;
+    const float weight_bias = sigmoid ? a.sigmoid_bias[head] : 0.0f;
     float running_max = -INFINITY, denom = 0.0f;
     float acc[MAX_DIM_PER_LANE];
 #pragma unroll
@@ -88,14 +95,19 @@ __global__ void __launch_bounds__(ATTN_WARPS * 32) paged_attention_generic_kerne
             if (a.softcap > 0.0f) score = a.softcap * tanhf(score / a.softcap);
             if (a.slopes) score -= slope * static_cast<float>(position - key);
         }
-        const float new_max = fmaxf(running_max, warp_max(score));
-        if (new_max == -INFINITY) continue;  // nothing visible yet (uniform across the warp)
-        const float p = base >= 0 ? expf(score - new_max) : 0.0f;
-        const float rescale = expf(running_max - new_max);  // 0 on the first tile (exp(-inf))
-        denom = denom * rescale + warp_sum(p);
-        running_max = new_max;
+        float p;
+        if (sigmoid) {
+            p = base >= 0 ? 1.0f / (1.0f + expf(-(score + weight_bias))) : 0.0f;
+        } else {
+            const float new_max = fmaxf(running_max, warp_max(score));
+            if (new_max == -INFINITY) continue;  // nothing visible yet (uniform across the warp)
+            p = base >= 0 ? expf(score - new_max) : 0.0f;
+            const float rescale = expf(running_max - new_max);  // 0 on the first tile (exp(-inf))
+            denom = denom * rescale + warp_sum(p);
+            running_max = new_max;
 #pragma unroll
-        for (int i = 0; i < MAX_DIM_PER_LANE; ++i) acc[i] *= rescale;
+            for (int i = 0; i < MAX_DIM_PER_LANE; ++i) acc[i] *= rescale;
+        }
         for (int j = 0; j < 32; ++j) {
             const float pj = __shfl_sync(0xffffffffu, p, j);
             const long long bj = __shfl_sync(0xffffffffu, base, j);
@@ -110,7 +122,7 @@ __global__ void __launch_bounds__(ATTN_WARPS * 32) paged_attention_generic_kerne
     }
     T* out = static_cast<T*>(a.out) + (static_cast<size_t>(token) * a.heads + head) * dv;
     if (a.sink) denom += expf((a.sink_values ? a.sink_values[head] : 0.0f) - running_max);  // the silent participant
-    float inv = 1.0f / denom;
+    float inv = sigmoid ? 1.0f : 1.0f / denom;
     const float* gate = a.gate ? a.gate + (static_cast<size_t>(token) * a.heads + head) * a.gate_width : nullptr;
     if (gate && a.gate_width == 1) inv *= gate[0];
 #pragma unroll
@@ -130,15 +142,15 @@ ME_EXPORT int me_paged_attention_generic(const void* q, const void* k_pages, con
                                          int heads, int kv_heads, int head_dim, int page_size, int table_width,
                                          int window, int value_dim, int sink, const float* gate, int gate_width,
                                          int value_stride, const float* slopes, const float* sink_values,
-                                         float softcap, cudaStream_t stream) {
+                                         float softcap, int chunk, const float* sigmoid_bias, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (gate && gate_width != 1 && gate_width != value_dim) return ME_ERR_ARGUMENT;
-    if (value_stride < value_dim) return ME_ERR_ARGUMENT;
+    if (value_stride < value_dim || chunk < 0 || (sigmoid_bias && sink)) return ME_ERR_ARGUMENT;
     if (head_dim > MAX_KEY_DIM || value_dim < 1 || value_dim > 32 * MAX_DIM_PER_LANE || heads % kv_heads)
         return ME_ERR_UNSUPPORTED;
     AttnArgs a{q, k_pages, v_pages, block_table, entry_of_token, positions, out, scale,
                tokens, heads, kv_heads, head_dim, page_size, table_width, window, value_dim, sink, gate,
-               gate_width, value_stride, slopes, sink_values, softcap};
+               gate_width, value_stride, slopes, sink_values, softcap, chunk, sigmoid_bias};
     const long long items = static_cast<long long>(tokens) * heads;
     const int blocks = static_cast<int>((items + ATTN_WARPS - 1) / ATTN_WARPS);
     const size_t smem = static_cast<size_t>(ATTN_WARPS) * head_dim * sizeof(float);

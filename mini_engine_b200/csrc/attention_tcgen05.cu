@@ -31,8 +31,9 @@
 // Formula and conventions as in attention_bf16.cu (YuvGev00/mini-engine:
 // src/mini_engine/attention.py:84-86,160-175; probabilities rounded to the value dtype before the
 // second product, :173).  head_dim is 128; pages of 8 to 128 tokens.  The form of one query head per CTA also
-// takes a sliding window, a linear distance bias, a silent participant of the softmax and a gate on the output
-// (attention_tcgen05_kernel<true>); the form of two heads per CTA takes none of them.
+// takes a sliding window, chunks of positions, a linear distance bias, a silent participant of the softmax and a gate on the
+// output (attention_tcgen05_kernel<OPTIONS>), or weights sigmoid(score + bias_h) in the place of a softmax, with a window or
+// chunks (attention_tcgen05_kernel<SIGMOID>); the form of two heads per CTA takes none of them.
 #include "tcgen05.cuh"
 
 constexpr int TC_ROWS = 128;   // query rows per CTA
@@ -54,7 +55,7 @@ struct TcAttnParams {
     __nv_bfloat16* out;       // [tokens][heads][128]
     float scale_log2;
     int heads, kv_heads, page_size, table_width;
-    // The options of attention_tcgen05_kernel<true>:
+    // The options of attention_tcgen05_kernel<OPTIONS>:
     int window;                // query p sees keys (p - window, p]; 0: all keys up to p
     int sink;                  // the softmax has one more participant without a value
     int gate_width;            // 1: a gate per (token, head); 128: a gate per output element
@@ -62,7 +63,15 @@ struct TcAttnParams {
     const float* sink_values;  // [heads] the silent participant's score (null with `sink`: zero)
     const float* gate;         // [tokens][heads * gate_width] multiplier of the output, or null
     float cap_log2;            // > 0: a scaled score s (log2 domain) becomes cap * tanh(s / cap); cap * log2(e) here
+    int chunk;                 // > 0: query p sees keys from floor(p / chunk) * chunk on
+    const float* sigmoid_bias; // SIGMOID: [heads] weights sigmoid(score + bias), not normalised
 };
+
+// The first key that the query at `position` sees.
+__device__ __forceinline__ int lowest_key(const TcAttnParams& p, int position) {
+    const int behind = p.window > 0 ? max(position - p.window + 1, 0) : 0;
+    return p.chunk > 0 ? max(behind, position / p.chunk * p.chunk) : behind;
+}
 
 // 2^x by the special-function unit alone (about 2 ulp; the result is rounded to bfloat16 anyway).
 __device__ __forceinline__ float fast_exp2(float x) {
@@ -132,11 +141,29 @@ __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
     return packed;
 }
 
-// OPT: the kernel also knows a sliding window (tiles wholly behind the window of the block's first row are never
+// 1 / (1 + 2^y) for four values with one reciprocal: r = 1 / (a b c d) and products of r with the other three.  y is held
+// below 30, so that the product of four stays finite; a weight is then at least 2^-30.
+__device__ __forceinline__ void inverse_one_plus_exp2(float (&y)[4]) {
+    float2 first = make_float2(1.0f + fast_exp2(fminf(y[0], 30.0f)), 1.0f + fast_exp2(fminf(y[1], 30.0f)));   // a, b
+    float2 second = make_float2(1.0f + fast_exp2(fminf(y[2], 30.0f)), 1.0f + fast_exp2(fminf(y[3], 30.0f)));  // c, d
+    const float2 pairs = __fmul2_rn(make_float2(first.x, second.x), make_float2(first.y, second.y));          // ab, cd
+    float r;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(pairs.x * pairs.y));
+    const float2 inverse = __fmul2_rn(make_float2(r, r), make_float2(pairs.y, pairs.x));  // 1 / ab, 1 / cd
+    first = __fmul2_rn(make_float2(inverse.x, inverse.x), make_float2(first.y, first.x));
+    second = __fmul2_rn(make_float2(inverse.y, inverse.y), make_float2(second.y, second.x));
+    y[0] = first.x, y[1] = first.y, y[2] = second.x, y[3] = second.y;
+}
+
+enum : int { PLAIN = 0, OPTIONS = 1, SIGMOID = 2 };
+
+// OPTIONS: the kernel also knows a sliding window (tiles wholly behind the window of the block's first row are never
 // fetched; the edge tiles are masked element by element), a linear distance bias, a silent participant in the
 // softmax's denominator and a multiplier on the output.  Scaled, biased scores and the mask are formed before the
 // row's maximum is taken, so the maximum is that of the values whose exponentials are summed.
-template <bool OPT>
+// SIGMOID: weights sigmoid(score * scale + bias_h) in the place of a softmax.  There is no maximum, no sum and nothing to rescale:
+// the two threads of a row never meet, and each writes its weights over its own score columns.
+template <int FORM>
 __global__ void __launch_bounds__(TC_THREADS, 2)
 attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                          const __grid_constant__ CUtensorMap map_v, TcAttnParams p) {
@@ -185,7 +212,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const int context = p.context_lens[entry];
     const int rows_valid = min(TC_ROWS, new_tokens - q_block * TC_ROWS);
     const int pos0 = context - new_tokens + q_block * TC_ROWS;  // position of row 0
-    const int lowest = (OPT && p.window > 0) ? max(pos0 - p.window + 1, 0) : 0;  // the first key that row 0 sees
+    constexpr bool OPT = FORM == OPTIONS;
+    const int lowest = FORM != PLAIN ? lowest_key(p, pos0) : 0;  // the first key that row 0 sees
     const int first_tile = lowest / TC_KEYS;
     const int tiles_count = has_work ? (pos0 + rows_valid - 1) / TC_KEYS + 1 - first_tile : 0;
 
@@ -262,7 +290,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 for (int kk = 0; kk < TC_KEYS / 16; ++kk) {
                     // 16 keys = 16 rows of 128 bytes; the second 64 dimensions are one half further
                     const uint64_t v_desc = smem_desc_sw128_mn(smem_u32(v_tile) + kk * 16 * 128, TC_HALF_BYTES);
-                    tcgen05_mma_bf16_ts(tmem_o, tmem_s + kk * 8, v_desc, idesc_o, (j > 0 || kk > 0) ? 1u : 0u);
+                    const uint32_t weights = FORM == SIGMOID ? (kk / 4) * 64 + (kk % 4) * 8 : kk * 8;  // columns
+                    tcgen05_mma_bf16_ts(tmem_o, tmem_s + weights, v_desc, idesc_o, (j > 0 || kk > 0) ? 1u : 0u);
                 }
                 tcgen05_commit(o_full + (j & 1));
                 tcgen05_commit(v_empty);
@@ -281,7 +310,49 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         // A wait that ran out must not leave other threads at a named barrier: a thread that saw
         // one keeps walking to the next barrier, where all 256 learn of it and leave together.
         bool ok = true;
+        const int lowest_seen = FORM != PLAIN ? lowest_key(p, row_pos) : 0;
+        const int last_lowest = FORM != PLAIN ? lowest_key(p, pos0 + TC_ROWS - 1) : 0;  // the last row's first key
         int j = 0;
+        if constexpr (FORM == SIGMOID) {
+            const float minus_bias = -p.sigmoid_bias[head] * TC_LOG2E;
+            const float2 minus_scale2 = make_float2(-p.scale_log2, -p.scale_log2), minus_bias2 = make_float2(minus_bias, minus_bias);
+            for (; j < tiles_count; ++j) {
+                ok = __all_sync(0xffffffffu, mbar_wait(s_full, j & 1));
+                if (!ok) break;
+                tcgen05_fence_after();
+                const int tile = first_tile + j, first_key = tile * TC_KEYS + col0;
+                const bool masked_tile = tile * TC_KEYS + TC_KEYS - 1 > pos0 || tile * TC_KEYS < last_lowest;
+#pragma unroll
+                for (int c = 0; c < 2; ++c) {
+                    uint32_t raw[32], packed[16];
+                    tcgen05_ld32_nowait(tmem_s + lane_base + col0 + c * 32, raw);
+                    tcgen05_wait_ld();
+                    tcgen05_pin32(raw);
+#pragma unroll
+                    for (int i = 0; i < 32; i += 4) {
+                        const float2 a = __ffma2_rn(make_float2(__uint_as_float(raw[i]), __uint_as_float(raw[i + 1])), minus_scale2, minus_bias2);
+                        const float2 b = __ffma2_rn(make_float2(__uint_as_float(raw[i + 2]), __uint_as_float(raw[i + 3])), minus_scale2, minus_bias2);
+                        float weight[4] = {a.x, a.y, b.x, b.y};
+                        inverse_one_plus_exp2(weight);
+                        if (masked_tile) {
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) {
+                                const int key = first_key + c * 32 + i + e;
+                                if (key > row_pos || key < lowest_seen) weight[e] = 0.0f;
+                            }
+                        }
+                        packed[i / 2] = pack_bf16x2(weight[0], weight[1]);
+                        packed[i / 2 + 1] = pack_bf16x2(weight[2], weight[3]);
+                    }
+                    // weights of keys [64 half + 32 c, +32) over the first columns of this thread's own half of the scores;
+                    // the scores that are still to be read lie behind them
+                    tcgen05_st16(tmem_s + lane_base + col0 + c * 16, packed);
+                }
+                tcgen05_wait_st();
+                tcgen05_fence_before();
+                mbar_arrive(p_full);
+            }
+        } else
         for (; j < tiles_count; ++j) {
             const uint32_t parity = j & 1;
             ok = ok && mbar_wait(s_full, parity);
@@ -290,8 +361,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             const int first_key = tile * TC_KEYS + col0;
             // Only the last tile or two of a block hold keys that some row must not see (and, with a window, the
             // first one or two); every other tile takes the path without per-element position tests.
-            const bool masked_tile = tile * TC_KEYS + TC_KEYS - 1 > pos0 ||
-                                     (OPT && p.window > 0 && tile * TC_KEYS < pos0 + TC_ROWS - p.window);
+            const bool masked_tile = tile * TC_KEYS + TC_KEYS - 1 > pos0 || (OPT && tile * TC_KEYS < last_lowest);
             uint32_t raw[64];
             tcgen05_ld32_nowait(tmem_s + lane_base + col0, raw);
             tcgen05_ld32_nowait(tmem_s + lane_base + col0 + 32, raw + 32);
@@ -305,7 +375,6 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 const float cap_scale = p.cap_log2 > 0.0f ? p.scale_log2 / p.cap_log2 : 0.0f;  // score -> tanh's argument
                 const float2 cap2 = make_float2(p.cap_log2, p.cap_log2), cap_scale2 = make_float2(cap_scale, cap_scale);
                 float2 distance = make_float2(static_cast<float>(first_key - row_pos), static_cast<float>(first_key + 1 - row_pos));
-                const int lowest_seen = p.window > 0 ? row_pos - p.window + 1 : 0;
 #pragma unroll
                 for (int i = 0; i < 64; i += 2) {
                     float2 x;
@@ -424,7 +493,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             row_sum += exp2f((p.sink_values ? p.sink_values[head] * TC_LOG2E : 0.0f) - (row_max == -INFINITY ? 0.0f : row_max));
         if (ok) {
             tcgen05_fence_after();
-            float inv = 1.0f / row_sum;
+            float inv = FORM == SIGMOID ? 1.0f : 1.0f / row_sum;
             const size_t pair_index = static_cast<size_t>(token0 + q_block * TC_ROWS + row) * p.heads + head;
             const bool element_gates = OPT && p.gate != nullptr && p.gate_width > 1;
             if (OPT && p.gate != nullptr && p.gate_width == 1 && row < rows_valid) inv *= p.gate[pair_index];
@@ -808,10 +877,10 @@ ME_EXPORT int me_attention_tcgen05(const void* map_q, const void* map_k, const v
                                    const int* cu_tokens, const int* context_lens, void* out, float scale, int entries,
                                    int max_new_tokens, int heads, int kv_heads, int head_dim, int page_size,
                                    int table_width, const int* entry_ids, int window, int sink, const float* gate,
-                                   int gate_width, const float* slopes, const float* sink_values, float softcap,
-                                   cudaStream_t stream) {
+                                   int gate_width, const float* slopes, const float* sink_values, float softcap, int chunk,
+                                   const float* sigmoid_bias, cudaStream_t stream) {
     if (entries <= 0) return 0;
-    if (window < 0 || (gate != nullptr && gate_width != 1 && gate_width != TC_DIM)) return ME_ERR_ARGUMENT;
+    if (window < 0 || chunk < 0 || (gate != nullptr && gate_width != 1 && gate_width != TC_DIM)) return ME_ERR_ARGUMENT;
     if (head_dim != TC_DIM || kv_heads < 1 || heads % kv_heads) return ME_ERR_UNSUPPORTED;
     if (page_size < 8 || page_size > TC_KEYS || TC_KEYS % page_size) return ME_ERR_UNSUPPORTED;
     alignas(64) CUtensorMap q, k, v;
@@ -820,13 +889,19 @@ ME_EXPORT int me_attention_tcgen05(const void* map_q, const void* map_k, const v
     memcpy(&v, map_v, sizeof(v));
     TcAttnParams p{block_table, cu_tokens, context_lens, entry_ids, static_cast<__nv_bfloat16*>(out), scale * TC_LOG2E,
                    heads, kv_heads, page_size, table_width, window, (sink || sink_values) ? 1 : 0, gate_width, slopes, sink_values, gate,
-                   softcap > 0.0f ? softcap * TC_LOG2E : 0.0f};
+                   softcap > 0.0f ? softcap * TC_LOG2E : 0.0f, chunk, sigmoid_bias};
     const int blocks = (max_new_tokens + TC_ROWS - 1) / TC_ROWS;
     constexpr int SMEM = 6 * TC_HALF_BYTES + 1024 + 256 + 2 * 2 * 128 * 4;
-    if (window > 0 || p.sink || gate != nullptr || slopes != nullptr || p.cap_log2 > 0.0f) {
+    if (sigmoid_bias != nullptr) {
+        if (p.sink || gate != nullptr || slopes != nullptr || p.cap_log2 > 0.0f) return ME_ERR_UNSUPPORTED;
+        static SharedMemoryOptIn with_sigmoid;
+        if (const int e = with_sigmoid(attention_tcgen05_kernel<SIGMOID>, SMEM)) return e;
+        return launch_kernel(attention_tcgen05_kernel<SIGMOID>, dim3(heads, blocks, entries), TC_THREADS, SMEM, stream, q, k, v, p);
+    }
+    if (window > 0 || chunk > 0 || p.sink || gate != nullptr || slopes != nullptr || p.cap_log2 > 0.0f) {
         static SharedMemoryOptIn with_options;
-        if (const int e = with_options(attention_tcgen05_kernel<true>, SMEM)) return e;
-        return launch_kernel(attention_tcgen05_kernel<true>, dim3(heads, blocks, entries), TC_THREADS, SMEM, stream, q, k, v, p);
+        if (const int e = with_options(attention_tcgen05_kernel<OPTIONS>, SMEM)) return e;
+        return launch_kernel(attention_tcgen05_kernel<OPTIONS>, dim3(heads, blocks, entries), TC_THREADS, SMEM, stream, q, k, v, p);
     }
     if ((heads / kv_heads) % 2 == 0) {  // two query heads of a KV group per CTA
         static SharedMemoryOptIn duo_opt_in;
@@ -835,8 +910,8 @@ ME_EXPORT int me_attention_tcgen05(const void* map_q, const void* map_k, const v
                              stream, q, k, v, p);
     }
     static SharedMemoryOptIn opt_in;
-    if (const int e = opt_in(attention_tcgen05_kernel<false>, SMEM)) return e;
-    return launch_kernel(attention_tcgen05_kernel<false>, dim3(heads, blocks, entries), TC_THREADS, SMEM, stream, q, k, v, p);
+    if (const int e = opt_in(attention_tcgen05_kernel<PLAIN>, SMEM)) return e;
+    return launch_kernel(attention_tcgen05_kernel<PLAIN>, dim3(heads, blocks, entries), TC_THREADS, SMEM, stream, q, k, v, p);
 }
 
 ME_EXPORT int me_attention_take_error(int* code) {

@@ -40,6 +40,7 @@ LIBRARIES = {
     "hyper_connections": "hyper_connections.cu",
     "sandwich": "sandwich.cu",
     "delta_rule": "delta_rule.cu",
+    "mixing": "mixing.cu",
     "recurrent": "recurrent.cu",
     "routing": "routing.cu",
     "gemm_tcgen05": "gemm_tcgen05.cu",

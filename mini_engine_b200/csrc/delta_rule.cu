@@ -3,7 +3,18 @@
 //
 //   S <- diag(g_t) S,   u_t = beta_t (v_t - S^T k_t),   S <- S + k_t u_t^T,   o_t = S^T q_t.
 //
-// `split_halves` hands the low-rank sums of the layer's input projection to the product with the second factors.
+// Two relatives walk through the same kernel.  The generalized delta rule removes with a rate a per key channel what the unit
+// key u = k / sqrt(k . k + eps) reads, both terms from the old state, and adds the key as it is:
+//
+//   S <- diag(g_t) S - (a_t * u_t) (u_t^T S) + k_t v_t^T,   o_t = S^T q_t.
+//
+// The recurrence with a bonus reads before it writes, the current token through a weight per key channel of its own:
+//
+//   o_t = (S + diag(b) k_t v_t^T)^T q_t,   S <- diag(g_t) S + k_t v_t^T.
+//
+// `state_prepare` makes what these two take.
+//
+// `split_halves` hands the low-rank sums of the layer's input projection (or their tanh) to the product with the second factors.
 // `delta_prepare` forms everything that enters the recurrence for all tokens at once: the short causal convolution of q,
 // k and v with silu, unit q and k, beta and the decays.  `delta_scan` walks the tokens of every entry.
 //
@@ -15,10 +26,11 @@
 
 // ------------------------------------------------------------------------- low-rank sums, halved
 
-// out[t] = (sums rounded to bfloat16 | what the rounding left, rounded to bfloat16); in float32 the sums themselves.
+// out[t] = (sums rounded to bfloat16 | what the rounding left, rounded to bfloat16); in float32 the sums themselves.  With
+// `activate` the tanh of the sums in their place.
 template <typename T>
 __global__ void __launch_bounds__(256) split_halves_kernel(const float* __restrict__ proj, int splits, size_t split_stride, int width,
-                                                           int column, int count, T* __restrict__ out, int tokens) {
+                                                           int column, int count, T* __restrict__ out, int tokens, int activate) {
     pdl_trigger();
     pdl_wait();
     const size_t total = static_cast<size_t>(tokens) * count;
@@ -28,6 +40,7 @@ __global__ void __launch_bounds__(256) split_halves_kernel(const float* __restri
         const float* src = proj + t * width + column + i;
         float sum = 0.0f;
         for (int s = 0; s < splits; ++s) sum += src[s * split_stride];
+        if (activate) sum = tanhf(sum);
         if constexpr (sizeof(T) == 2) {
             const T high = from_float<T>(sum);
             out[t * 2 * count + i] = high;
@@ -39,15 +52,15 @@ __global__ void __launch_bounds__(256) split_halves_kernel(const float* __restri
 }
 
 ME_EXPORT int me_split_halves(const float* proj, int splits, long long split_stride, int width, int column, int count, void* out,
-                              int out_type, int tokens, cudaStream_t stream) {
+                              int out_type, int tokens, int activate, cudaStream_t stream) {
     if (tokens <= 0 || count <= 0) return 0;
     const size_t total = static_cast<size_t>(tokens) * count;
     const int blocks = static_cast<int>(std::min<size_t>((total + 255) / 256, 148 * 8));
     if (out_type == ME_BF16)
         return launch_kernel(split_halves_kernel<__nv_bfloat16>, blocks, 256, 0, stream, proj, splits, (size_t)split_stride, width,
-                             column, count, static_cast<__nv_bfloat16*>(out), tokens);
+                             column, count, static_cast<__nv_bfloat16*>(out), tokens, activate);
     return launch_kernel(split_halves_kernel<float>, blocks, 256, 0, stream, proj, splits, (size_t)split_stride, width, column,
-                         count, static_cast<float*>(out), tokens);
+                         count, static_cast<float*>(out), tokens, activate);
 }
 
 // -------------------------------------------------------------------------------------- prepare
@@ -388,6 +401,127 @@ ME_EXPORT int me_delta_prepare(const float* proj, int splits, long long split_st
     return launch_delta_prepare<16>(a, stream);
 }
 
+// --------------------------------------------------------- prepare: the generalized rule and the bonus
+
+enum : int { RULE_DELTA = 0, RULE_REMOVAL = 1, RULE_BONUS = 2 };
+
+template <int RULE>
+struct Rule;
+// VECTORS: what the walk reads per token and head beside the values ([VECTORS][dim]); SCALARS: numbers per token and head.
+template <>
+struct Rule<RULE_DELTA> { static constexpr int VECTORS = 3, SCALARS = 2; };    // q, k, g; beta, q . k
+template <>
+struct Rule<RULE_REMOVAL> { static constexpr int VECTORS = 4, SCALARS = 4; };  // q g, k, g, a k; 1 / (k . k + eps), that times sum q a k, q . k
+template <>
+struct Rule<RULE_BONUS> { static constexpr int VECTORS = 3, SCALARS = 2; };    // q, k, g; sum q b k
+
+// Columns of a product's partial sums.
+struct Columns {
+    const float* sums;  // [splits][tokens][width], moved to the first column
+    int splits;
+    size_t stride;
+    int width;
+    __device__ __forceinline__ float at(size_t token, int column) const {
+        const float* src = sums + token * width + column;
+        float x = 0.0f;
+#pragma unroll 4
+        for (int s = 0; s < splits; ++s) x += src[s * stride];
+        return x;
+    }
+};
+
+struct StatePrepArgs {
+    Columns q, k, v, logits, rate;  // [heads * dim] each (v: [heads * vdim]); rate for the removal only
+    const float* decay_bias;  // [heads * dim]: added to the decay's logits
+    const float* channel;     // [heads * dim]: the removal's rate bias, or the bonus
+    float* rows;              // [tokens][heads][VECTORS * dim + vdim]
+    float* scalars;           // [tokens][heads][SCALARS]
+    float decay_scale, unit_eps;
+    int tokens, heads, dim, vdim;
+};
+
+// One warp per (token, head), a lane's channels 32 apart.  The decay is exp(-decay_scale * sigmoid(z)) (removal) or
+// exp(-exp(z)) (bonus), as 1 + expm1: the float nearest to it where it is near 1.
+template <int RULE, int PER>
+__global__ void __launch_bounds__(PREP_WARPS * 32) state_prepare_kernel(StatePrepArgs a) {
+    const long long item = static_cast<long long>(blockIdx.x) * PREP_WARPS + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31;
+    pdl_trigger();
+    pdl_wait();
+    if (item >= static_cast<long long>(a.tokens) * a.heads) return;
+    const size_t token = static_cast<size_t>(item / a.heads);
+    const int head = static_cast<int>(item % a.heads), first = head * a.dim;
+    constexpr int VECTORS = Rule<RULE>::VECTORS;
+    float q[PER], k[PER], z[PER], rate[PER];
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int d = lane + 32 * i;
+        const bool live = d < a.dim;
+        q[i] = live ? a.q.at(token, first + d) : 0.0f;
+        k[i] = live ? a.k.at(token, first + d) : 0.0f;
+        z[i] = live ? a.logits.at(token, first + d) + a.decay_bias[first + d] : 0.0f;
+        if (RULE == RULE_REMOVAL) rate[i] = live ? a.rate.at(token, first + d) + a.channel[first + d] : 0.0f;
+        else rate[i] = live ? a.channel[first + d] : 0.0f;
+    }
+    float* row = a.rows + static_cast<size_t>(item) * (VECTORS * a.dim + a.vdim);
+    float squares = 0.0f, dot = 0.0f, weighted = 0.0f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int d = lane + 32 * i;
+        if (d >= a.dim) continue;
+        float decay;
+        if constexpr (RULE == RULE_REMOVAL) {
+            decay = 1.0f + expm1f(-a.decay_scale / (1.0f + expf(-z[i])));
+            const float removed = k[i] / (1.0f + expf(-rate[i]));  // a k
+            row[d] = q[i] * decay;
+            row[3 * a.dim + d] = removed;
+            squares = fmaf(k[i], k[i], squares);
+            dot = fmaf(q[i], k[i], dot);
+            weighted = fmaf(q[i], removed, weighted);
+        } else {
+            decay = 1.0f + expm1f(-expf(z[i]));
+            row[d] = q[i];
+            weighted = fmaf(q[i] * rate[i], k[i], weighted);
+        }
+        row[a.dim + d] = k[i];
+        row[2 * a.dim + d] = decay;
+    }
+    for (int e = lane; e < a.vdim; e += 32) row[VECTORS * a.dim + e] = a.v.at(token, head * a.vdim + e);
+    weighted = warp_sum(weighted);
+    float* scalars = a.scalars + static_cast<size_t>(item) * Rule<RULE>::SCALARS;
+    if constexpr (RULE == RULE_REMOVAL) {
+        squares = warp_sum(squares), dot = warp_sum(dot);
+        const float inverse = 1.0f / (squares + a.unit_eps);
+        if (lane == 0) scalars[0] = inverse, scalars[1] = inverse * weighted, scalars[2] = dot, scalars[3] = 0.0f;
+    } else if (lane == 0) {
+        scalars[0] = weighted, scalars[1] = 0.0f;
+    }
+}
+
+template <int RULE>
+static int launch_state_prepare(const StatePrepArgs& a, cudaStream_t stream) {
+    const long long items = static_cast<long long>(a.tokens) * a.heads;
+    const int blocks = static_cast<int>((items + PREP_WARPS - 1) / PREP_WARPS);
+    if (a.dim <= 32) return launch_kernel(state_prepare_kernel<RULE, 1>, blocks, PREP_WARPS * 32, 0, stream, a);
+    if (a.dim <= 64) return launch_kernel(state_prepare_kernel<RULE, 2>, blocks, PREP_WARPS * 32, 0, stream, a);
+    if (a.dim <= 128) return launch_kernel(state_prepare_kernel<RULE, 4>, blocks, PREP_WARPS * 32, 0, stream, a);
+    return launch_kernel(state_prepare_kernel<RULE, 16>, blocks, PREP_WARPS * 32, 0, stream, a);
+}
+
+// The five column ranges are given as pointer, splits, stride and width each: q, k, v, the decay's logits, the removal's rate.
+ME_EXPORT int me_state_prepare(const float* const* sums, const int* splits, const long long* strides, const int* widths, int rule,
+                               const float* decay_bias, const float* channel, float* rows, float* scalars, float decay_scale,
+                               float unit_eps, int tokens, int heads, int dim, int vdim, cudaStream_t stream) {
+    if (tokens <= 0) return 0;
+    if (dim < 1 || vdim < 1 || heads < 1 || (rule != RULE_REMOVAL && rule != RULE_BONUS)) return ME_ERR_ARGUMENT;
+    if (dim > MAX_DIM) return ME_ERR_UNSUPPORTED;
+    Columns ranges[5];
+    for (int i = 0; i < 5; ++i) ranges[i] = Columns{sums[i], splits[i], (size_t)strides[i], widths[i]};
+    StatePrepArgs a{ranges[0], ranges[1], ranges[2], ranges[3], ranges[4], decay_bias, channel, rows, scalars, decay_scale,
+                    unit_eps, tokens, heads, dim, vdim};
+    return rule == RULE_REMOVAL ? launch_state_prepare<RULE_REMOVAL>(a, stream) : launch_state_prepare<RULE_BONUS>(a, stream);
+}
+
 // ----------------------------------------------------------------------------------------- scan
 
 // A value column's state [dim] is held by L neighbouring lanes, R channels each (float4 number i of lane l holds channels
@@ -398,12 +532,14 @@ ME_EXPORT int me_delta_prepare(const float* proj, int splits, long long split_st
 // The walking warps of a block share the tokens' q, k, decays, values and scalars; one more warp fetches them, SC tokens
 // ahead, by asynchronous copies, and stores the outputs of the SC tokens before.  Columns are independent and a token's output depends on the tokens before it through the state alone: the
 // bits are the same for a whole prompt, its portions and single decoded tokens.
+// The generalized rule reads S^T k and S^T (q g) of the old state in the same butterfly: with c = 1 / (k . k + eps) the removal is
+// (a k) c (S^T k) and o = S^T (q g) - c (sum q a k) (S^T k) + (q . k) v.  With the bonus o = S^T q + (sum q b k) v.
 constexpr int SCAN_WARPS = 4;  // most walking warps of a block
 
 struct DeltaScanArgs {
-    const float* qk;       // [tokens][qk_heads][2][dim]
-    const float* gv;       // [tokens][heads][dim + vdim]
-    const float* scalars;  // [tokens][heads][2]
+    const float* qk;       // [tokens][qk_heads][2][dim] (the delta rule; else unused)
+    const float* gv;       // [tokens][heads][dim + vdim]; the other rules: all vectors, [tokens][heads][VECTORS * dim + vdim]
+    const float* scalars;  // [tokens][heads][SCALARS]
     const int* cu_tokens;
     const int* state_slots;
     const int* fresh;
@@ -425,10 +561,10 @@ __device__ __forceinline__ void copy_async_commit() { asm volatile("cp.async.com
 template <int LEFT>
 __device__ __forceinline__ void copy_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(LEFT) : "memory"); }
 
-// What a lane reads of one token: its R channels of k, q and the decays.
-template <int R>
+// What a lane reads of one token: its R channels of k, q and the decays (and of what the generalized rule removes).
+template <int R, int VECTORS>
 struct TokenRow {
-    float2 k[R / 2], q[R / 2], g[R / 2];
+    float2 k[R / 2], q[R / 2], g[R / 2], removed[VECTORS > 3 ? R / 2 : 1];
     template <int L>
     __device__ __forceinline__ void load(const float* at) {
 #pragma unroll
@@ -439,27 +575,32 @@ struct TokenRow {
             k[2 * i] = make_float2(k4.x, k4.y), k[2 * i + 1] = make_float2(k4.z, k4.w);
             q[2 * i] = make_float2(q4.x, q4.y), q[2 * i + 1] = make_float2(q4.z, q4.w);
             g[2 * i] = make_float2(g4.x, g4.y), g[2 * i + 1] = make_float2(g4.z, g4.w);
+            if constexpr (VECTORS > 3) {
+                const float4 a4 = *reinterpret_cast<const float4*>(at + 3 * L * R + 4 * i * L);
+                removed[2 * i] = make_float2(a4.x, a4.y), removed[2 * i + 1] = make_float2(a4.z, a4.w);
+            }
         }
     }
 };
 
-template <int L, int R, int C, int SC>
+template <int RULE, int L, int R, int C, int SC>
 __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32) delta_scan_kernel(DeltaScanArgs a) {
+    constexpr int VECTORS = Rule<RULE>::VECTORS, SCALARS = Rule<RULE>::SCALARS;
     constexpr int DP = L * R;  // the key channels a column has room for
     constexpr int GROUPS = 32 / L, COLUMNS = GROUPS * C;  // of a warp
     extern __shared__ __align__(16) float staged[];
     const int threads = blockDim.x, warp = threadIdx.x >> 5, warps = (threads >> 5) - 1, columns = warps * COLUMNS;
-    const int stage_floats = SC * (3 * DP + columns + 2);
+    const int stage_floats = SC * (VECTORS * DP + columns + SCALARS);
     float* results = staged + 2 * stage_floats;  // [2][SC][columns]
     const bool fetches = warp == warps;  // the last warp
-    // one stage: q, k and the decays of every token [SC][3][DP], v [SC][columns], scalars [SC][2]
+    // one stage: q, k, the decays (and the rest) of every token [SC][VECTORS][DP], v [SC][columns], scalars [SC][SCALARS]
     const int entry = blockIdx.x, head = blockIdx.y, qk_head = head / (a.heads / a.qk_heads);
     const int first_column = blockIdx.z * columns;
     const int lane = threadIdx.x & 31, part = lane % L;
     const int local_column = warp * COLUMNS + lane / L;  // and GROUPS, 2 GROUPS, ... behind it
     const int dim = a.dim;
-    for (int i = threadIdx.x; i < 2 * SC * 3 * (DP - dim); i += threads) {  // channels dim .. DP are zero for good
-        const int stage = i / (SC * 3 * (DP - dim)), j = i % (SC * 3 * (DP - dim));
+    for (int i = threadIdx.x; i < 2 * SC * VECTORS * (DP - dim); i += threads) {  // channels dim .. DP are zero for good
+        const int stage = i / (SC * VECTORS * (DP - dim)), j = i % (SC * VECTORS * (DP - dim));
         staged[stage * stage_floats + (j / (DP - dim)) * DP + dim + j % (DP - dim)] = 0.0f;
     }
     const int begin = a.cu_tokens[entry], end = a.cu_tokens[entry + 1];
@@ -492,30 +633,34 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32) delta_scan_kernel(Delta
     const int live_columns = min(columns, a.vdim - first_column);
     // The fetching warp's lane holds 16-byte pieces lane, lane + 32, ... of a token's q, k and decays (piece j belongs at
     // float 4 j of the token's row); their sources move on by one token at a time.
-    constexpr int PIECES = (3 * DP / 4 + 31) / 32;
+    constexpr int PIECES = (VECTORS * DP / 4 + 31) / 32;
+    constexpr bool ONE_ROW = RULE != RULE_DELTA;  // all vectors of a token and head lie side by side
     const float* source[PIECES];
     bool wanted[PIECES];
-    const size_t qk_step = static_cast<size_t>(a.qk_heads) * 2 * dim, gv_step = static_cast<size_t>(a.heads) * (dim + a.vdim);
+    const size_t qk_step = static_cast<size_t>(a.qk_heads) * 2 * dim, gv_step = static_cast<size_t>(a.heads) * ((ONE_ROW ? VECTORS : 1) * dim + a.vdim);
     const float* qk_begin = a.qk + (static_cast<size_t>(begin) * a.qk_heads + qk_head) * 2 * dim;
-    const float* gv_begin = a.gv + (static_cast<size_t>(begin) * a.heads + head) * (dim + a.vdim);
+    const float* gv_begin = a.gv + (static_cast<size_t>(begin) * a.heads + head) * ((ONE_ROW ? VECTORS : 1) * dim + a.vdim);
 #pragma unroll
     for (int i = 0; i < PIECES; ++i) {
         const int j = lane + 32 * i, which = j / (DP / 4), d = j % (DP / 4) * 4;
-        wanted[i] = which < 3 && d < dim;
-        source[i] = which < 2 ? qk_begin + which * dim + d : gv_begin + d;
+        wanted[i] = which < VECTORS && d < dim;
+        source[i] = ONE_ROW ? gv_begin + which * dim + d : which < 2 ? qk_begin + which * dim + d : gv_begin + d;
     }
-    const float* value_source = gv_begin + dim + first_column;
-    const float* scalar_source = a.scalars + (static_cast<size_t>(begin) * a.heads + head) * 2;
+    const float* value_source = gv_begin + (ONE_ROW ? VECTORS : 1) * dim + first_column;
+    const float* scalar_source = a.scalars + (static_cast<size_t>(begin) * a.heads + head) * SCALARS;
     auto stage_tokens = [&](int chunk, float* stage) {
         const int count = min(SC, end - chunk);
-        float* v_s = stage + SC * 3 * DP;
+        float* v_s = stage + SC * VECTORS * DP;
         for (int t = 0; t < count; ++t) {
             if (a.vector) {
 #pragma unroll
                 for (int i = 0; i < PIECES; ++i) {
-                    if (wanted[i]) copy_async_16(stage + t * 3 * DP + 4 * (lane + 32 * i), source[i]);
-                    source[i] += (lane + 32 * i) / (DP / 4) < 2 ? qk_step : gv_step;
+                    if (wanted[i]) copy_async_16(stage + t * VECTORS * DP + 4 * (lane + 32 * i), source[i]);
+                    source[i] += !ONE_ROW && (lane + 32 * i) / (DP / 4) < 2 ? qk_step : gv_step;
                 }
+            } else if constexpr (ONE_ROW) {
+                const float* row = gv_begin + (chunk - begin + t) * gv_step;
+                for (int j = lane; j < VECTORS * dim; j += 32) copy_async_4(stage + (t * VECTORS + j / dim) * DP + j % dim, row + j);
             } else {
                 const float* qk = qk_begin + (chunk - begin + t) * qk_step;
                 const float* gv = gv_begin + (chunk - begin + t) * gv_step;
@@ -523,9 +668,9 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32) delta_scan_kernel(Delta
                 for (int j = lane; j < dim; j += 32) copy_async_4(stage + (t * 3 + 2) * DP + j, gv + j);
             }
             for (int j = lane; j < live_columns; j += 32) copy_async_4(v_s + t * columns + j, value_source + j);
-            if (lane < 2) copy_async_4(v_s + SC * columns + 2 * t + lane, scalar_source + lane);
+            if (lane < SCALARS) copy_async_4(v_s + SC * columns + SCALARS * t + lane, scalar_source + lane);
             value_source += gv_step;
-            scalar_source += a.heads * 2;
+            scalar_source += a.heads * SCALARS;
         }
         copy_async_commit();
     };
@@ -554,11 +699,12 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32) delta_scan_kernel(Delta
             continue;
         }
         const float* rows_s = staged + buffer * stage_floats + 4 * part;
-        const float* v_s = staged + buffer * stage_floats + SC * 3 * DP;
+        const float* v_s = staged + buffer * stage_floats + SC * VECTORS * DP;
         const float* scalars_s = v_s + SC * columns;
         // One token: its row is in registers already.
-        auto walk = [&](const TokenRow<R>& row, int t) {
-            const float2 scalars = *reinterpret_cast<const float2*>(scalars_s + 2 * t);  // beta, q . k
+        auto walk = [&](const TokenRow<R, VECTORS>& row, int t) {
+            const float2 scalars = *reinterpret_cast<const float2*>(scalars_s + SCALARS * t);  // the delta rule: beta, q . k
+            const float q_dot_k = SCALARS > 2 ? scalars_s[SCALARS * t + (SCALARS > 2 ? 2 : 0)] : 0.0f;
             float dot_k[C], dot_q[C], v[C];
 #pragma unroll
             for (int c = 0; c < C; ++c) {
@@ -567,8 +713,8 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32) delta_scan_kernel(Delta
                 float2 on_q[2] = {make_float2(0.0f, 0.0f), make_float2(0.0f, 0.0f)};
 #pragma unroll
                 for (int i = 0; i < R / 2; ++i) {
-                    s[c][i] = __fmul2_rn(row.g[i], s[c][i]);
-                    on_k[i & 1] = __ffma2_rn(row.k[i], s[c][i], on_k[i & 1]);
+                    if (RULE == RULE_DELTA) s[c][i] = __fmul2_rn(row.g[i], s[c][i]);
+                    if (RULE != RULE_BONUS) on_k[i & 1] = __ffma2_rn(row.k[i], s[c][i], on_k[i & 1]);
                     on_q[i & 1] = __ffma2_rn(row.q[i], s[c][i], on_q[i & 1]);
                 }
                 dot_k[c] = (on_k[0].x + on_k[0].y) + (on_k[1].x + on_k[1].y);
@@ -578,30 +724,45 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32) delta_scan_kernel(Delta
             for (int offset = L / 2; offset > 0; offset >>= 1) {
 #pragma unroll
                 for (int c = 0; c < C; ++c) {
-                    dot_k[c] += __shfl_xor_sync(0xffffffffu, dot_k[c], offset);
+                    if (RULE != RULE_BONUS) dot_k[c] += __shfl_xor_sync(0xffffffffu, dot_k[c], offset);
                     dot_q[c] += __shfl_xor_sync(0xffffffffu, dot_q[c], offset);
                 }
             }
             float mine = 0.0f;  // lane number c of a group stores column c
 #pragma unroll
             for (int c = 0; c < C; ++c) {
-                const float u = scalars.x * (v[c] - dot_k[c]);
-                const float2 uu = make_float2(u, u);
+                float o;
+                if constexpr (RULE == RULE_DELTA) {
+                    const float u = scalars.x * (v[c] - dot_k[c]);
+                    const float2 uu = make_float2(u, u);
 #pragma unroll
-                for (int i = 0; i < R / 2; ++i) s[c][i] = __ffma2_rn(row.k[i], uu, s[c][i]);
-                const float o = fmaf(scalars.y, u, dot_q[c]);
+                    for (int i = 0; i < R / 2; ++i) s[c][i] = __ffma2_rn(row.k[i], uu, s[c][i]);
+                    o = fmaf(scalars.y, u, dot_q[c]);
+                } else if constexpr (RULE == RULE_REMOVAL) {
+                    const float read = -scalars.x * dot_k[c];
+                    const float2 vv = make_float2(v[c], v[c]), rr = make_float2(read, read);
+#pragma unroll
+                    for (int i = 0; i < R / 2; ++i)
+                        s[c][i] = __ffma2_rn(row.removed[i], rr, __ffma2_rn(row.k[i], vv, __fmul2_rn(row.g[i], s[c][i])));
+                    o = fmaf(q_dot_k, v[c], fmaf(-scalars.y, dot_k[c], dot_q[c]));
+                } else {
+                    const float2 vv = make_float2(v[c], v[c]);
+#pragma unroll
+                    for (int i = 0; i < R / 2; ++i) s[c][i] = __ffma2_rn(row.g[i], s[c][i], __fmul2_rn(row.k[i], vv));
+                    o = fmaf(scalars.x, v[c], dot_q[c]);
+                }
                 if (c == 0 || part == c) mine = o;
             }
             if (part < C) results[(buffer * SC + t) * columns + local_column + part * GROUPS] = mine;
         };
-        TokenRow<R> even, odd;
+        TokenRow<R, VECTORS> even, odd;
         even.template load<L>(rows_s);
 #pragma unroll 1
         for (int t = 0; t < count; t += 2) {
-            if (t + 1 < count) odd.template load<L>(rows_s + (t + 1) * 3 * DP);
+            if (t + 1 < count) odd.template load<L>(rows_s + (t + 1) * VECTORS * DP);
             walk(even, t);
             if (t + 1 >= count) break;
-            if (t + 2 < count) even.template load<L>(rows_s + (t + 2) * 3 * DP);
+            if (t + 2 < count) even.template load<L>(rows_s + (t + 2) * VECTORS * DP);
             walk(odd, t + 1);
         }
         __syncthreads();
@@ -626,7 +787,7 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32) delta_scan_kernel(Delta
     }
 }
 
-template <int L, int R, int C, int SC>
+template <int RULE, int L, int R, int C, int SC>
 static int launch_delta_scan(const DeltaScanArgs& a, int entries, cudaStream_t stream) {
     static SharedMemoryOptIn opt_in;
     constexpr int COLUMNS = 32 / L * C;
@@ -637,11 +798,24 @@ static int launch_delta_scan(const DeltaScanArgs& a, int entries, cudaStream_t s
                          (warps / 2) * COLUMNS >= a.vdim))
         warps /= 2;
     const int columns = warps * COLUMNS;
-    const size_t smem = static_cast<size_t>(2) * SC * (3 * L * R + 2 * columns + 2) * sizeof(float);
+    const size_t smem = static_cast<size_t>(2) * SC * (Rule<RULE>::VECTORS * L * R + 2 * columns + Rule<RULE>::SCALARS) * sizeof(float);
     if (smem > 48 * 1024)
-        if (const int e = opt_in(delta_scan_kernel<L, R, C, SC>, 200 * 1024)) return e;
+        if (const int e = opt_in(delta_scan_kernel<RULE, L, R, C, SC>, 200 * 1024)) return e;
     const dim3 grid(entries, a.heads, (a.vdim + columns - 1) / columns);
-    return launch_kernel_in_order(delta_scan_kernel<L, R, C, SC>, grid, (warps + 1) * 32, smem, stream, a);
+    return launch_kernel_in_order(delta_scan_kernel<RULE, L, R, C, SC>, grid, (warps + 1) * 32, smem, stream, a);
+}
+
+template <int RULE>
+static int dispatch_delta_scan(const DeltaScanArgs& a, int entries, cudaStream_t stream) {
+    if (a.dim <= 32) return launch_delta_scan<RULE, 8, 4, 1, 16>(a, entries, stream);
+    if (a.dim <= 64) return launch_delta_scan<RULE, 8, 8, 1, 16>(a, entries, stream);
+    if (a.dim <= 128) return launch_delta_scan<RULE, 8, 16, 2, 16>(a, entries, stream);
+    if (a.dim <= 256) return launch_delta_scan<RULE, 16, 16, 2, 8>(a, entries, stream);
+    if (a.dim > MAX_DIM) return ME_ERR_UNSUPPORTED;
+    if constexpr (RULE == RULE_REMOVAL)  // four vectors per token: a lane has room for fewer channels
+        return launch_delta_scan<RULE, 32, 16, 2, 8>(a, entries, stream);
+    else
+        return launch_delta_scan<RULE, 16, 32, 1, 8>(a, entries, stream);
 }
 
 ME_EXPORT int me_delta_scan(const float* qk, const float* gv, const float* scalars, const int* cu_tokens, const int* state_slots,
@@ -653,10 +827,18 @@ ME_EXPORT int me_delta_scan(const float* qk, const float* gv, const float* scala
     const auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
     const int vector = dim % 4 == 0 && vdim % 4 == 0 && slot_floats % 4 == 0 && aligned(qk) && aligned(gv) && aligned(state);
     DeltaScanArgs a{qk, gv, scalars, cu_tokens, state_slots, fresh, state, (size_t)slot_floats, out, heads, qk_heads, dim, vdim, vector};
-    if (dim <= 32) return launch_delta_scan<8, 4, 1, 16>(a, entries, stream);
-    if (dim <= 64) return launch_delta_scan<8, 8, 1, 16>(a, entries, stream);
-    if (dim <= 128) return launch_delta_scan<8, 16, 2, 16>(a, entries, stream);
-    if (dim <= 256) return launch_delta_scan<16, 16, 2, 8>(a, entries, stream);
-    if (dim <= MAX_DIM) return launch_delta_scan<16, 32, 1, 8>(a, entries, stream);
-    return ME_ERR_UNSUPPORTED;
+    return dispatch_delta_scan<RULE_DELTA>(a, entries, stream);
+}
+
+// The other rules, on what me_state_prepare made.
+ME_EXPORT int me_state_walk(const float* rows, const float* scalars, const int* cu_tokens, const int* state_slots, const int* fresh,
+                            float* state, long long slot_floats, float* out, int rule, int entries, int heads, int dim, int vdim,
+                            cudaStream_t stream) {
+    if (entries <= 0) return 0;
+    if (dim < 1 || vdim < 1 || heads < 1 || (rule != RULE_REMOVAL && rule != RULE_BONUS)) return ME_ERR_ARGUMENT;
+    if (slot_floats < static_cast<long long>(heads) * dim * vdim) return ME_ERR_ARGUMENT;
+    const auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+    const int vector = dim % 4 == 0 && vdim % 4 == 0 && slot_floats % 4 == 0 && aligned(rows) && aligned(state);
+    DeltaScanArgs a{nullptr, rows, scalars, cu_tokens, state_slots, fresh, state, (size_t)slot_floats, out, heads, heads, dim, vdim, vector};
+    return rule == RULE_REMOVAL ? dispatch_delta_scan<RULE_REMOVAL>(a, entries, stream) : dispatch_delta_scan<RULE_BONUS>(a, entries, stream);
 }

@@ -811,7 +811,7 @@ __global__ void __launch_bounds__(QKV_WARPS * 32) qk_norm_rope_store_128_kernel(
 // (cos, sin) of position * inv_freq for every token of the step, once per step for all layers
 // (src/mini_engine/model.py:79-83,183 of YuvGev00/mini-engine builds its tables once per step too).
 __global__ void rope_table_kernel(const float* __restrict__ inv_freq, const int* __restrict__ positions,
-                                  float2* __restrict__ out, int tokens, int half) {
+                                  float2* __restrict__ out, int tokens, int half, float amplitude) {
     pdl_trigger();
     pdl_wait();
     const int idx = blockIdx.x * blockDim.x + threadIdx.x;
@@ -819,20 +819,20 @@ __global__ void rope_table_kernel(const float* __restrict__ inv_freq, const int*
     const int token = idx / half, i = idx % half;
     float sine, cosine;
     sincosf(static_cast<float>(positions[token]) * inv_freq[i], &sine, &cosine);
-    out[idx] = make_float2(cosine, sine);
+    out[idx] = make_float2(cosine * amplitude, sine * amplitude);
 }
 
-ME_EXPORT int me_rope_table(const float* inv_freq, const int* positions, float* out, int tokens, int half,
+ME_EXPORT int me_rope_table(const float* inv_freq, const int* positions, float* out, int tokens, int half, float amplitude,
                             cudaStream_t stream) {
     if (tokens <= 0) return 0;
     const int total = tokens * half;
     return launch_kernel(rope_table_kernel, (total + 255) / 256, 256, 0, stream, inv_freq, positions,
-                         reinterpret_cast<float2*>(out), tokens, half);
+                         reinterpret_cast<float2*>(out), tokens, half, amplitude);
 }
 
 // The same with the angle formed, and reduced to one turn, in double precision.
 __global__ void rope_table_double_kernel(const double* __restrict__ inv_freq, const int* __restrict__ positions,
-                                         float2* __restrict__ out, int tokens, int half) {
+                                         float2* __restrict__ out, int tokens, int half, float amplitude) {
     pdl_trigger();
     pdl_wait();
     const int idx = blockIdx.x * blockDim.x + threadIdx.x;
@@ -842,15 +842,15 @@ __global__ void rope_table_double_kernel(const double* __restrict__ inv_freq, co
     const double angle = static_cast<double>(positions[token]) * inv_freq[i];
     float sine, cosine;
     sincosf(static_cast<float>(angle - TURN * rint(angle / TURN)), &sine, &cosine);
-    out[idx] = make_float2(cosine, sine);
+    out[idx] = make_float2(cosine * amplitude, sine * amplitude);
 }
 
-ME_EXPORT int me_rope_table_double(const double* inv_freq, const int* positions, float* out, int tokens, int half,
+ME_EXPORT int me_rope_table_double(const double* inv_freq, const int* positions, float* out, int tokens, int half, float amplitude,
                                    cudaStream_t stream) {
     if (tokens <= 0) return 0;
     const int total = tokens * half;
     return launch_kernel(rope_table_double_kernel, (total + 255) / 256, 256, 0, stream, inv_freq, positions,
-                         reinterpret_cast<float2*>(out), tokens, half);
+                         reinterpret_cast<float2*>(out), tokens, half, amplitude);
 }
 
 ME_EXPORT int me_qk_norm_rope_store(const float* qkv, int splits, long long split_stride, const float* q_weight,
@@ -860,7 +860,7 @@ ME_EXPORT int me_qk_norm_rope_store(const float* qkv, int splits, long long spli
                                     int heads, int kv_heads, int head_dim, int page_size, int rotary_dim,
                                     const float* bias, int value_dim, cudaStream_t stream) {
     if (tokens <= 0) return 0;
-    if (head_dim > MAX_HEAD_DIM || (head_dim % 2 && cos_sin != nullptr)) return ME_ERR_UNSUPPORTED;
+    if (head_dim > MAX_HEAD_DIM) return ME_ERR_UNSUPPORTED;
     if (value_dim < 1 || value_dim > MAX_HEAD_DIM) return ME_ERR_UNSUPPORTED;
     if (rotary_dim < 0 || rotary_dim > head_dim || rotary_dim % 2) return ME_ERR_ARGUMENT;
     QkvArgs a{qkv, splits, (size_t)split_stride, q_weight, k_weight, eps, reinterpret_cast<const float2*>(cos_sin), positions, slot_mapping,

@@ -667,8 +667,8 @@ ME_EXPORT int me_retention_scan(const float* proj, int splits, long long split_s
     return ME_ERR_UNSUPPORTED;
 }
 
-// out[t][h][e] = weight[e] * o[t][h][e] * rsqrt(mean_e(o^2) + eps) * gate(g[t][h][e]); a null weight is all ones.  The gate
-// is silu or the sigmoid.
+// out[t][h][e] = weight[e] * o[t][h][e] * rsqrt(mean_e(o^2) + eps) * gate(g[t][h][e]); a null weight is all ones, and with
+// a weight_step of vdim every head has a weight of its own.  The gate is silu or the sigmoid.
 enum : int { FINISH_SILU = 0, FINISH_SIGMOID = 1 };
 
 __device__ __forceinline__ float finish_gate(float g, int kind) {
@@ -679,7 +679,8 @@ template <typename T>
 __global__ void __launch_bounds__(128) gla_finish_kernel(const float* __restrict__ o, const float* __restrict__ proj,
                                                          int splits, size_t split_stride, int width, int g_col,
                                                          const float* __restrict__ weight, float eps,
-                                                         T* __restrict__ out, int tokens, int heads, int vdim, int gate_kind) {
+                                                         T* __restrict__ out, int tokens, int heads, int vdim, int gate_kind,
+                                                         int weight_step) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long item = static_cast<long long>(blockIdx.x) * 4 + warp;
     pdl_trigger();
@@ -697,7 +698,7 @@ __global__ void __launch_bounds__(128) gla_finish_kernel(const float* __restrict
     for (int e = lane; e < vdim; e += 32) {
         float gate = 0.0f;
         for (int p = 0; p < splits; ++p) gate += gate_row[p * split_stride + e];
-        dst[e] = from_float<T>((weight ? weight[e] : 1.0f) * (row[e] * inv) * finish_gate(gate, gate_kind));
+        dst[e] = from_float<T>((weight ? weight[head * weight_step + e] : 1.0f) * (row[e] * inv) * finish_gate(gate, gate_kind));
     }
 }
 
@@ -765,7 +766,7 @@ __global__ void __launch_bounds__(256) projection_finish_kernel(const float* __r
 
 ME_EXPORT int me_gla_finish(const float* o, const float* proj, int splits, long long split_stride, int width,
                             int g_col, const float* weight, float eps, void* out, int type, int tokens, int heads,
-                            int vdim, int gate_kind, int whole_projection, cudaStream_t stream) {
+                            int vdim, int gate_kind, int whole_projection, int weight_step, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (gate_kind != FINISH_SILU && gate_kind != FINISH_SIGMOID) return ME_ERR_ARGUMENT;
     if (whole_projection) {
@@ -789,7 +790,7 @@ ME_EXPORT int me_gla_finish(const float* o, const float* proj, int splits, long 
     if (type == ME_BF16)
         return launch_kernel(gla_finish_kernel<__nv_bfloat16>, blocks, 128, 0, stream, o, proj, splits,
                              (size_t)split_stride, width, g_col, weight, eps, static_cast<__nv_bfloat16*>(out), tokens,
-                             heads, vdim, gate_kind);
+                             heads, vdim, gate_kind, weight_step);
     return launch_kernel(gla_finish_kernel<float>, blocks, 128, 0, stream, o, proj, splits, (size_t)split_stride, width,
-                         g_col, weight, eps, static_cast<float*>(out), tokens, heads, vdim, gate_kind);
+                         g_col, weight, eps, static_cast<float*>(out), tokens, heads, vdim, gate_kind, weight_step);
 }

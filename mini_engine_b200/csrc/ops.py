@@ -398,16 +398,16 @@ def qk_norm_rope_store(
     _check(code, "qk_norm_rope_store")
 
 
-def rope_table(inv_freq: torch.Tensor, positions: torch.Tensor, out: torch.Tensor) -> None:
-    """``out[t, i] = (cos, sin)(positions[t] * inv_freq[i])`` in float32, ``[T, rotary_dim / 2, 2]``.  With float64
+def rope_table(inv_freq: torch.Tensor, positions: torch.Tensor, out: torch.Tensor, amplitude: float = 1.0) -> None:
+    """``out[t, i] = amplitude * (cos, sin)(positions[t] * inv_freq[i])`` in float32, ``[T, rotary_dim / 2, 2]``.  With float64
     frequencies the angle is formed, and reduced to one turn, in double precision."""
     double = inv_freq.dtype == torch.float64
     _need(inv_freq, torch.float64 if double else torch.float32, "inv_freq"), _need(positions, torch.int32, "positions"), _need(out, torch.float32, "out")
     tokens, half = positions.shape[0], inv_freq.shape[0]
     if tuple(out.shape) != (tokens, half, 2):
         raise KernelError(f"rope_table: out {tuple(out.shape)} is not [{tokens}, {half}, 2]")
-    fn = _fn("elementwise", "me_rope_table_double" if double else "me_rope_table", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p])
-    _check(fn(_ptr(inv_freq), _ptr(positions), _ptr(out), tokens, half, _stream()), "rope_table")
+    fn = _fn("elementwise", "me_rope_table_double" if double else "me_rope_table", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p])
+    _check(fn(_ptr(inv_freq), _ptr(positions), _ptr(out), tokens, half, float(amplitude), _stream()), "rope_table")
 
 
 def kv_store(k_dense, v_dense, slot_mapping, k_pages, v_pages, kv_heads: int, head_dim: int, page_size: int) -> None:
@@ -470,15 +470,17 @@ def gemm_tensor_core_swiglu(plan, x: torch.Tensor, act: torch.Tensor, activation
 def paged_attention_generic(
     q, k_pages, v_pages, block_table, entry_of_token, positions, out, heads, kv_heads, head_dim, scale, window,
     value_dim: int | None = None, sink: bool = False, gate: torch.Tensor | None = None,
-    slopes: torch.Tensor | None = None, sink_values: torch.Tensor | None = None, softcap: float = 0.0,
+    slopes: torch.Tensor | None = None, sink_values: torch.Tensor | None = None, softcap: float = 0.0, chunk: int = 0,
+    sigmoid_bias: torch.Tensor | None = None,
 ) -> None:
     """One warp per (token, head), any head size; ``softcap`` > 0: a scaled score ``s`` becomes ``softcap * tanh(s /
     softcap)``; ``value_dim``: width of a value head when it differs;
     ``sink``: one more participant of score zero and no value in the softmax, or of the learned score
     ``sink_values[h]`` (float32 ``[heads]``); ``gate`` (float32 ``[T, heads]`` or ``[T, heads * value_dim]``): a
     multiplier on each head's output, or on each of its elements; ``slopes`` (float32 ``[heads]``): ``slopes[h] *
-    (p - j)`` is taken off the scaled score of query ``p`` and key ``j``.  ``v_pages=None``: the values are the first
-    ``value_dim`` elements of the key rows."""
+    (p - j)`` is taken off the scaled score of query ``p`` and key ``j``; ``chunk`` > 0: a query at ``p`` sees keys from ``p //
+    chunk * chunk`` on; ``sigmoid_bias`` (float32 ``[heads]``): a key's weight is ``sigmoid(s + bias_h)``, not normalised, in
+    the place of a softmax.  ``v_pages=None``: the values are the first ``value_dim`` elements of the key rows."""
     value_dim = head_dim if value_dim is None else value_dim
     gate_width = 1
     if gate is not None:
@@ -487,7 +489,7 @@ def paged_attention_generic(
             gate_width = value_dim
         elif gate.shape != (q.shape[0], heads):
             raise KernelError("gate must be [tokens, heads] or [tokens, heads * value_dim]")
-    for name, vector in (("slopes", slopes), ("sink_values", sink_values)):
+    for name, vector in (("slopes", slopes), ("sink_values", sink_values), ("sigmoid_bias", sigmoid_bias)):
         if vector is not None:
             _need(vector, torch.float32, name)
             if vector.shape != (heads,):
@@ -507,13 +509,13 @@ def paged_attention_generic(
     fn = _fn(
         "attention_generic",
         "me_paged_attention_generic",
-        [c_void_p] * 7 + [c_int, c_float] + [c_int] * 9 + [c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p],
+        [c_void_p] * 7 + [c_int, c_float] + [c_int] * 9 + [c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p],
     )
     code = fn(
         _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), _ptr(entry_of_token), _ptr(positions), _ptr(out),
         _type_code(q.dtype), scale, q.shape[0], heads, kv_heads, head_dim, k_pages.shape[2], block_table.shape[1],
         window, value_dim, 1 if (sink or sink_values is not None) else 0, _ptr(gate), gate_width, value_stride,
-        _ptr(slopes), _ptr(sink_values), float(softcap or 0.0), _stream(),
+        _ptr(slopes), _ptr(sink_values), float(softcap or 0.0), int(chunk), _ptr(sigmoid_bias), _stream(),
     )  # fmt: skip
     _check(code, "paged_attention_generic")
 
@@ -521,27 +523,29 @@ def paged_attention_generic(
 def paged_attention(
     *, q, k_pages, v_pages, block_table, ctx, out, heads: int, kv_heads: int, head_dim: int, scale: float, window: int,
     value_dim: int | None = None, sink: bool = False, gate: torch.Tensor | None = None,
-    slopes: torch.Tensor | None = None, sink_values: torch.Tensor | None = None, softcap: float = 0.0,
+    slopes: torch.Tensor | None = None, sink_values: torch.Tensor | None = None, softcap: float = 0.0, chunk: int = 0,
+    sigmoid_bias: torch.Tensor | None = None,
 ) -> None:  # fmt: skip
     """Causal attention of the batch's new tokens over their requests' cached keys (the new
     tokens' own keys are already in the cache).  Chooses the kernel by dtype and sizes.  ``value_dim``,
-    ``sink``, ``gate``, ``slopes`` and ``sink_values`` as in :func:`paged_attention_generic`; value heads of another
+    ``sink``, ``gate``, ``slopes``, ``sink_values``, ``chunk`` and ``sigmoid_bias`` as in :func:`paged_attention_generic`; value heads of another
     width than the key heads and values inside the key rows (``v_pages=None``) take that kernel."""
     if v_pages is None and q.dtype == torch.bfloat16 and latent_attention_supports(head_dim, value_dim, kv_heads):
-        if sink or slopes is not None or sink_values is not None or softcap:
-            raise KernelError("attention over latent rows takes a window and a gate per head, no sink, no distance bias and no cap")
+        if sink or slopes is not None or sink_values is not None or softcap or chunk or sigmoid_bias is not None:
+            raise KernelError("attention over latent rows takes a window and a gate per head, no sink, no distance bias, no cap, no chunks and a softmax")
         latent_attention_bf16(q, k_pages, block_table, ctx, out, heads, head_dim, value_dim, scale, window, gate)
         return
     if v_pages is not None and q.dtype == torch.bfloat16 and value_dim in (None, head_dim):
         if attention_bf16.supports(head_dim, heads, kv_heads):
             attention_bf16.paged_attention(
                 q, k_pages, v_pages, block_table, ctx, out, heads, kv_heads, head_dim, scale, window, sink=sink, gate=gate,
-                slopes=slopes, sink_values=sink_values, softcap=softcap,
+                slopes=slopes, sink_values=sink_values, softcap=softcap, chunk=chunk, sigmoid_bias=sigmoid_bias,
             )  # fmt: skip
             return
     paged_attention_generic(
         q, k_pages, v_pages, block_table, ctx.entry_of_token, ctx.positions, out, heads, kv_heads, head_dim,
         scale, window, value_dim=value_dim, sink=sink, gate=gate, slopes=slopes, sink_values=sink_values, softcap=softcap,
+        chunk=chunk, sigmoid_bias=sigmoid_bias,
     )  # fmt: skip
 
 
@@ -861,23 +865,25 @@ def gla_finish(
 ) -> None:  # fmt: skip
     """``out = weight * o / rms(o) * silu(gate)`` per (token, head); the gate is a column range of ``proj``;
     ``weight=None`` is a weight of ones.  ``gate="sigmoid"`` multiplies by the gate's sigmoid; ``scope="projection"`` takes
-    the root mean square over all heads of a token together, with a weight ``[heads * vdim]``."""
+    the root mean square over all heads of a token together.  The weight is ``[vdim]``, shared by the heads, or ``[heads *
+    vdim]``."""
     if gate not in FINISH_GATES or scope not in ("head", "projection"):
         raise KernelError("gla_finish: the gate is 'silu' or 'sigmoid', the scope 'head' or 'projection'")
     _need(o, torch.float32, "o"), _need(proj, torch.float32, "proj"), _need(out, None, "out")
     if weight is not None:
         _need(weight, torch.float32, "weight")
-        if weight.shape != (vdim if scope == "head" else heads * vdim,):
+        if weight.shape != (heads * vdim,) and (scope == "projection" or weight.shape != (vdim,)):
             raise KernelError("gla_finish: the weight does not fit the scope of the norm")
     tokens = o.shape[0]
     fn = _fn(
         "linear_attention",
         "me_gla_finish",
-        [c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_void_p, c_float, c_void_p] + [c_int] * 6 + [c_void_p],
+        [c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_void_p, c_float, c_void_p] + [c_int] * 7 + [c_void_p],
     )
     code = fn(
         _ptr(o), _ptr(proj), proj.shape[0], proj.stride(0), proj.shape[2], gate_column, _ptr(weight), float(eps), _ptr(out),
-        _type_code(out.dtype), tokens, heads, vdim, FINISH_GATES[gate], 1 if scope == "projection" else 0, _stream(),
+        _type_code(out.dtype), tokens, heads, vdim, FINISH_GATES[gate], 1 if scope == "projection" else 0,
+        vdim if weight is not None and weight.shape[0] == heads * vdim else 0, _stream(),
     )  # fmt: skip
     _check(code, "gla_finish")
 
@@ -1161,15 +1167,16 @@ def input_convolution(*, h: torch.Tensor, taps: torch.Tensor, ctx, state: torch.
     _check(code, "input_convolution")
 
 
-def split_halves(proj: torch.Tensor, column: int, count: int, out: torch.Tensor) -> None:
+def split_halves(proj: torch.Tensor, column: int, count: int, out: torch.Tensor, activate: bool = False) -> None:
     """The columns ``column .. column + count`` of ``sum_s proj[s]``: rounded to bfloat16, and behind them what the rounding
-    left, rounded to bfloat16 (``out [T, 2 * count]``); with a float32 ``out [T, count]`` the sums themselves."""
+    left, rounded to bfloat16 (``out [T, 2 * count]``); with a float32 ``out [T, count]`` the sums themselves.  ``activate``:
+    the tanh of the sums in their place."""
     _need(proj, torch.float32, "proj"), _need(out, None, "out")
     splits, tokens, width = proj.shape
     if out.shape != (tokens, count * (2 if out.dtype == torch.bfloat16 else 1)) or column + count > width:
         raise KernelError("split_halves: out or the columns do not fit")
-    fn = _fn("delta_rule", "me_split_halves", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p])
-    code = fn(_ptr(proj), splits, proj.stride(0), width, column, count, _ptr(out), _type_code(out.dtype), tokens, _stream())
+    fn = _fn("delta_rule", "me_split_halves", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p])
+    code = fn(_ptr(proj), splits, proj.stride(0), width, column, count, _ptr(out), _type_code(out.dtype), tokens, int(activate), _stream())
     _check(code, "split_halves")
 
 
@@ -1227,6 +1234,187 @@ def delta_scan(
         state.shape[1], _ptr(out), ctx.num_entries, heads, qk_heads, dim, vdim, _stream(),
     )  # fmt: skip
     _check(code, "delta_scan")
+
+
+STATE_RULES = {"removal": 1, "bonus": 2}
+_RULE_FLOATS = {"removal": (4, 4), "bonus": (3, 2)}  # vectors of a key head's width, numbers per token and head
+
+
+def state_rule_floats(rule: str, dim: int, vdim: int) -> tuple[int, int]:
+    """Floats per token and head of the ``rows`` and the ``scalars`` that :func:`state_prepare` makes."""
+    vectors, numbers = _RULE_FLOATS[rule]
+    return vectors * dim + vdim, numbers
+
+
+def state_prepare(
+    *, rule: str, q: tuple, k: tuple, v: tuple, logits: tuple, rate: tuple | None, decay_bias: torch.Tensor, channel: torch.Tensor,
+    rows: torch.Tensor, scalars: torch.Tensor, decay_scale: float, unit_eps: float, heads: int, dim: int, vdim: int,
+) -> None:  # fmt: skip
+    """What the recurrence of ``rule`` takes, for all tokens of the batch, in float32.  ``q``, ``k``, ``v``, ``logits`` (and ``rate``)
+    are pairs (partial sums ``[S, T, width]``, first column).  ``"removal"``: decays ``exp(-decay_scale * sigmoid(logits +
+    decay_bias))``, removal rates ``sigmoid(rate + channel)``.  ``"bonus"``: decays ``exp(-exp(logits + decay_bias))``, ``channel``
+    is the bonus.  Outputs: ``rows [T, heads, ...]`` and ``scalars [T, heads, ...]`` (:func:`state_rule_floats`)."""
+    if rule not in STATE_RULES or (rate is None) != (rule != "removal"):
+        raise KernelError("state_prepare: the rule is 'removal' (with a rate) or 'bonus' (without)")
+    ranges = [q, k, v, logits, rate if rate is not None else q]
+    tokens = q[0].shape[1]
+    for (sums, column), width in zip(ranges, (heads * dim, heads * dim, heads * vdim, heads * dim, heads * dim)):
+        _need(sums, torch.float32, "sums")
+        if sums.dim() != 3 or sums.shape[1] != tokens or column + width > sums.shape[2]:
+            raise KernelError(f"state_prepare: columns {column}..{column + width} of {tuple(sums.shape)} for {tokens} tokens")
+    for name, t in (("decay_bias", decay_bias), ("channel", channel), ("rows", rows), ("scalars", scalars)):
+        _need(t, torch.float32, name)
+    row, numbers = state_rule_floats(rule, dim, vdim)
+    if decay_bias.numel() != heads * dim or channel.numel() != heads * dim or rows.numel() < tokens * heads * row or scalars.numel() < tokens * heads * numbers:
+        raise KernelError("state_prepare: constants or outputs do not fit heads and dim")
+    pointers = (c_void_p * 5)(*[sums.data_ptr() + 4 * column for sums, column in ranges])
+    splits = (c_int * 5)(*[sums.shape[0] for sums, _ in ranges])
+    strides = (c_longlong * 5)(*[sums.stride(0) for sums, _ in ranges])
+    widths = (c_int * 5)(*[sums.shape[2] for sums, _ in ranges])
+    fn = _fn("delta_rule", "me_state_prepare", [c_void_p] * 4 + [c_int] + [c_void_p] * 4 + [c_float, c_float] + [c_int] * 4 + [c_void_p])
+    code = fn(
+        pointers, splits, strides, widths, STATE_RULES[rule], _ptr(decay_bias), _ptr(channel), _ptr(rows), _ptr(scalars),
+        float(decay_scale), float(unit_eps), tokens, heads, dim, vdim, _stream(),
+    )  # fmt: skip
+    _check(code, "state_prepare")
+
+
+def state_walk(
+    *, rule: str, rows: torch.Tensor, scalars: torch.Tensor, ctx, state: torch.Tensor, out: torch.Tensor, heads: int, dim: int, vdim: int,
+) -> None:  # fmt: skip
+    """The recurrence of ``rule`` over the batch's tokens, entry by entry, from and into each request's state slot (``state
+    [slots + 1, floats]``, a slot starts with ``[heads, vdim, dim]``), on what :func:`state_prepare` made; ``out`` is float32
+    ``[T, heads, vdim]``."""
+    for name, t in (("rows", rows), ("scalars", scalars), ("state", state), ("out", out)):
+        _need(t, torch.float32, name)
+    if state.dim() != 2 or state.shape[1] < heads * dim * vdim:
+        raise KernelError("state_walk: the state does not hold the matrix states")
+    fn = _fn("delta_rule", "me_state_walk", [c_void_p] * 6 + [c_longlong, c_void_p] + [c_int] * 5 + [c_void_p])
+    code = fn(
+        _ptr(rows), _ptr(scalars), _ptr(ctx.cu_tokens), _ptr(ctx.state_slots), _ptr(ctx.fresh), _ptr(state), state.shape[1],
+        _ptr(out), STATE_RULES[rule], ctx.num_entries, heads, dim, vdim, _stream(),
+    )  # fmt: skip
+    _check(code, "state_walk")
+
+
+def _stream_sum(x, first, second, bias, tokens: int | None, width: int) -> list:
+    """Arguments of a residual sum: the stream (or ``None``), partial sums of one or two sublayers, a bias."""
+    arguments = [_ptr(x)]
+    if x is not None:
+        _need(x, torch.float32, "x")
+        if x.shape[1] != width or (tokens is not None and x.shape[0] != tokens):
+            raise KernelError(f"x {tuple(x.shape)} is not [{tokens}, {width}]")
+    for partial in (first, second):
+        if partial is None:
+            arguments += [_ptr(None), 0, 0]
+            continue
+        _need(partial, torch.float32, "partial sums")
+        if partial.dim() != 3 or partial.shape[2] != width or (tokens is not None and partial.shape[1] != tokens):
+            raise KernelError(f"partial sums {tuple(partial.shape)} are not [S, {tokens}, {width}]")
+        arguments += [_ptr(partial), partial.shape[0], partial.stride(0)]
+    if bias is not None:
+        _need(bias, torch.float32, "bias")
+        if bias.shape != (width,):
+            raise KernelError(f"bias {tuple(bias.shape)} is not [{width}]")
+    return arguments + [_ptr(bias)]
+
+
+_STREAM_SUM = [c_void_p] + [c_void_p, c_int, c_longlong] * 2 + [c_void_p]
+
+
+def tanh_norms(
+    *, x: torch.Tensor | None, first: torch.Tensor | None, second: torch.Tensor | None, bias: torch.Tensor | None,
+    x_out: torch.Tensor | None, norms: list[tuple], rows: torch.Tensor | None = None, shift: torch.Tensor | None = None,
+    state: torch.Tensor | None = None, ctx=None,
+) -> None:  # fmt: skip
+    """``s = x + sum(first) + sum(second) + bias`` (absent terms are ``None``), written to ``x_out`` (another buffer than ``x``), and
+    one or two dynamic-tanh norms of it, ``norms = [(weight, bias, alpha, out), ...]``: ``tanh(alpha * s) * weight + bias``.
+    ``shift`` (float32 ``[width]``): the first norm's output ``h`` becomes ``h + (h' - h) * shift`` with the previous token's
+    ``h'``, from and into ``state [slots + 1, width]`` (float32; the last ``h`` of a request).  ``rows``: only those tokens."""
+    if not 1 <= len(norms) <= 2:
+        raise KernelError("tanh_norms takes one or two norms")
+    width = norms[0][0].shape[0]
+    out_type = norms[0][3].dtype
+    source = next(t for t in (x, first, second) if t is not None)
+    whole = source.shape[-2]
+    tokens = whole if rows is None else rows.shape[0]
+    pointers: list = []
+    for weight, beta, alpha, out in norms:
+        for name, t in (("weight", weight), ("bias", beta), ("alpha", alpha)):
+            _need(t, torch.float32, name)
+        _need(out, out_type, "out")
+        if weight.shape != (width,) or beta.shape != (width,) or alpha.numel() != 1 or out.shape != (tokens, width):
+            raise KernelError("tanh_norms: a norm's tensors or its output do not fit")
+        pointers += [_ptr(weight), _ptr(beta), _ptr(alpha), _ptr(out)]
+    pointers += [_ptr(None)] * (8 - len(pointers))
+    if x_out is not None:
+        _need(x_out, torch.float32, "x_out")
+        if x_out.shape != (whole, width):
+            raise KernelError("tanh_norms: x_out does not fit")
+    steps = [_ptr(None)] * 4
+    if shift is not None:
+        _need(shift, torch.float32, "shift"), _need(state, torch.float32, "state")
+        if shift.shape != (width,) or state.dim() != 2 or state.shape[1] != width:
+            raise KernelError("tanh_norms: shift or state do not fit")
+        steps = [_ptr(ctx.entry_of_token), _ptr(ctx.cu_tokens), _ptr(ctx.state_slots), _ptr(ctx.fresh)]
+    if rows is not None:
+        _need(rows, torch.int32, "rows")
+    fn = _fn("mixing", "me_tanh_norms", _STREAM_SUM + [c_void_p] + [c_void_p] * 8 + [c_void_p] * 7 + [c_int] * 3 + [c_void_p])
+    code = fn(
+        *_stream_sum(x, first, second, bias, whole, width), _ptr(x_out), *pointers, _ptr(shift), _ptr(state), *steps, _ptr(rows),
+        _type_code(out_type), tokens, width, _stream(),
+    )  # fmt: skip
+    _check(code, "tanh_norms")
+
+
+def sum_rows(*, x, first, second, bias, out: torch.Tensor, column: int = 0) -> None:
+    """``x + sum(first) + sum(second) + bias`` (absent terms are ``None``) into the columns from ``column`` on of ``out``."""
+    source = next(t for t in (x, first, second) if t is not None)
+    tokens, width = source.shape[-2], source.shape[-1]
+    _need(out, None, "out")
+    if out.dim() != 2 or out.shape[0] != tokens:
+        raise KernelError("sum_rows: out does not fit")
+    fn = _fn("mixing", "me_sum_rows", _STREAM_SUM + [c_void_p] + [c_int] * 5 + [c_void_p])
+    code = fn(*_stream_sum(x, first, second, bias, tokens, width), _ptr(out), _type_code(out.dtype), out.shape[1], column, tokens, width, _stream())
+    _check(code, "sum_rows")
+
+
+def token_mix(*, h: torch.Tensor, mu: torch.Tensor, ctx, state: torch.Tensor, out: torch.Tensor, state_column: int = 0) -> None:
+    """``out[s] = h + (h' - h) * mu[s]`` for every row of ``mu [count, width]`` (float32), with ``h'`` the previous token's ``h``
+    of the same request (zeros for its first token), from and into ``state [slots + 1, floats]`` (float32), whose columns from
+    ``state_column`` on hold the last ``h``.  ``out`` is ``[count, T, width]`` in the dtype of ``h [T, width]``."""
+    _need(h, None, "h"), _need(mu, torch.float32, "mu"), _need(state, torch.float32, "state"), _need(out, h.dtype, "out")
+    tokens, width = h.shape
+    count = mu.shape[0]
+    if mu.shape != (count, width) or out.shape != (count, tokens, width) or state.dim() != 2 or state_column + width > state.shape[1]:
+        raise KernelError("token_mix: mu, state or out do not fit")
+    fn = _fn("mixing", "me_token_mix", [c_void_p, c_int] + [c_void_p] * 3 + [c_longlong] + [c_void_p] * 4 + [c_int] * 3 + [c_void_p])
+    code = fn(
+        _ptr(h), _type_code(h.dtype), _ptr(mu), _ptr(out), c_void_p(state.data_ptr() + 4 * state_column), state.shape[1],
+        _ptr(ctx.entry_of_token), _ptr(ctx.cu_tokens), _ptr(ctx.state_slots), _ptr(ctx.fresh), tokens, width, count, _stream(),
+    )  # fmt: skip
+    _check(code, "token_mix")
+
+
+def branch_norm_sum(branches: list[tuple[torch.Tensor, float, torch.Tensor, float]], out: torch.Tensor) -> None:
+    """``out [T, width] = sum_b factor_b * weight_b * y_b / rms(y_b)`` with ``y_b`` the sum of the branch's partial sums ``[S, T,
+    width]``; branches are (partial sums, factor, weight, eps)."""
+    _need(out, torch.float32, "out")
+    count = len(branches)
+    if not 1 <= count <= 4:
+        raise KernelError("branch_norm_sum takes one to four branches")
+    for partial, _factor, weight, _eps in branches:
+        _need(partial, torch.float32, "partial"), _need(weight, torch.float32, "weight")
+        if partial.dim() != 3 or tuple(partial.shape[1:]) != tuple(out.shape) or weight.shape != (out.shape[1],):
+            raise KernelError(f"branch {tuple(partial.shape)} does not fit out {tuple(out.shape)}")
+    fn = _fn("mixing", "me_branch_norm_sum", [c_void_p] * 6 + [c_int, c_void_p, c_int, c_int, c_void_p])
+    code = fn(
+        (c_void_p * count)(*[b[0].data_ptr() for b in branches]), (c_int * count)(*[b[0].shape[0] for b in branches]),
+        (c_longlong * count)(*[b[0].stride(0) for b in branches]), (c_void_p * count)(*[b[2].data_ptr() for b in branches]),
+        (c_float * count)(*[float(b[1]) for b in branches]), (c_float * count)(*[float(b[3]) for b in branches]), count, _ptr(out),
+        out.shape[0], out.shape[1], _stream(),
+    )  # fmt: skip
+    _check(code, "branch_norm_sum")
 
 
 def pair_embedding(

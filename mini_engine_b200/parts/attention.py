@@ -46,6 +46,12 @@ And one for designs that put positions into the values as well: ``value_encoding
 head.  The value of position ``j`` is cached turned by ``j``; a head's output, the weighted sum of turned values, is turned
 back by the query's position ``i``, so that what leaves the head is the sum of values turned by ``j - i``.  It combines with
 ``qkv_bias``, ``o_bias``, ``value_dim``, ``scale``, ``window`` and a partial rotation of q and k.
+
+And two for designs that read in chunks and weigh without a softmax: with ``chunk`` the query at position ``p`` sees key ``j <= p``
+when both lie in the same chunk of positions, ``p // chunk == j // chunk`` (counted from the sequence's start; the pages of
+earlier chunks are given back); ``weights="sigmoid"`` gives a visible key the weight ``sigmoid(s + b_h)`` with a learned number
+per head (tensor ``weight_bias``), not normalised over the keys.  They combine with per-head q/k norms, ``value_dim``, ``scale``
+and a partial rotation; ``chunk`` also with a sink, gates and the linear distance bias.
 """
 
 from __future__ import annotations
@@ -100,6 +106,8 @@ class GroupedQueryAttention(Mixer):
         unit_norm_eps: float | None = None,
         score_softcap: float | None = None,
         value_encoding: PartSpec | None = None,
+        chunk: int | None = None,
+        weights: str = "softmax",
     ):
         if num_heads % kv_heads:
             raise ValueError(f"num_heads ({num_heads}) must be a multiple of kv_heads ({kv_heads})")
@@ -129,6 +137,13 @@ class GroupedQueryAttention(Mixer):
         self.unit_store = self.unit_norm_eps is not None or bool(self.softcap) or value_encoding is not None
         if self.unit_store and (qk_norm_eps is not None or head_gate or element_gate or distance_bias or talking_heads or keep_first or reads_shared_cache):
             raise ValueError("unit_norm_eps, score_softcap and value_encoding do not combine with q/k norm weights, gates, distance biases, talking heads, keep_first or a shared cache")
+        if weights not in ("softmax", "sigmoid") or (chunk is not None and chunk < 1):
+            raise ValueError(f"weights is 'softmax' or 'sigmoid' and a chunk holds at least one position, got {weights!r} and {chunk}")
+        self.chunk, self.sigmoid = chunk, weights == "sigmoid"
+        if self.sigmoid and (self.sink or head_gate or element_gate or distance_bias or self.linear_bias or self.unit_store):
+            raise ValueError("sigmoid weights do not combine with a sink, gates, distance biases, unit norms, caps or rotated values")
+        if (self.chunk or self.sigmoid) and (window or keep_first or distance_bias or talking_heads or reads_shared_cache or self.unit_store or qkv_bias):
+            raise ValueError("chunk and sigmoid weights do not combine with a window, keep_first, the logarithmic distance bias, talking heads, a shared cache, biases, unit norms, caps or rotated values")
         # Whether q, k, v (and the gates) leave the fused product through the kernel that normalises whole projections.
         self.wide_store = self.wide_norm or self.head_gate or self.element_gate or self.linear_bias
         if (self.head_gate or self.element_gate or self.linear_bias) and qk_norm_eps is not None and not self.wide_norm:
@@ -138,14 +153,14 @@ class GroupedQueryAttention(Mixer):
         if qkv_bias and self.sink and not self.wide_store and not self.unit_store:
             raise ValueError("biases with a sink need the projection-wide store (a gate, a linear bias or qk_norm_scope='projection')")
         self.extended = bool(
-            (self.value_dim != head_dim and not (self.wide_store or self.sink or self.unit_store)) or self.keep_first or distance_bias or talking_heads
+            (self.value_dim != head_dim and not (self.wide_store or self.sink or self.unit_store or self.chunk or self.sigmoid)) or self.keep_first or distance_bias or talking_heads
         )
         if self.extended:
             if reads_shared_cache or qkv_bias:
                 raise ValueError("the extended attention options do not combine with a shared cache or biases")
             if head_dim < 1 or self.value_dim < 1 or keep_first < 0:
                 raise ValueError("head sizes must be positive and keep_first must not be negative")
-        elif self.wide_store or self.sink or self.unit_store:  # these run in the kernel that takes any head size
+        elif self.wide_store or self.sink or self.unit_store or self.chunk or self.sigmoid:  # these run in the kernel that takes any head size
             if not (1 <= head_dim <= 512 and 1 <= self.value_dim <= 512):
                 raise ValueError(f"head sizes must lie between 1 and 512, got {head_dim} and {self.value_dim}")
         else:
@@ -178,6 +193,7 @@ class GroupedQueryAttention(Mixer):
             "gate": "gate_proj.weight",
             "sink": "sink",
             "o_bias": "o_proj.bias",
+            "weight_bias": "weight_bias",
         }
         self.names = {key: prefix + (names or {}).get(key, value) for key, value in defaults.items()}
         self.position = None
@@ -190,6 +206,7 @@ class GroupedQueryAttention(Mixer):
         self.gates = num_heads if self.head_gate else num_heads * self.value_dim if self.element_gate else 0
         self.slopes: torch.Tensor | None = None
         self.sink_values: torch.Tensor | None = None
+        self.weight_bias: torch.Tensor | None = None
         self.qkv: Linear | None = None
         self.out: Linear | None = None
         self.q_norm: torch.Tensor | None = None
@@ -200,7 +217,7 @@ class GroupedQueryAttention(Mixer):
 
     def paged_cache(self) -> PagedCacheSpec:
         value_dim = None if self.value_dim == self.head_dim else self.value_dim
-        return PagedCacheSpec(self.kv_heads, self.head_dim, self.window, value_dim, self.keep_first)
+        return PagedCacheSpec(self.kv_heads, self.head_dim, self.window or self.chunk, value_dim, self.keep_first, self.chunk)
 
     def weight_specs(self) -> list[WeightSpec]:
         d, n = self.head_dim, self.names
@@ -219,6 +236,8 @@ class GroupedQueryAttention(Mixer):
             specs.append(WeightSpec(n["gate"], (self.gates, self.hidden)))
         if self.learned_sink:
             specs.append(WeightSpec(n["sink"], (self.heads,), role="vector", init="wide_normal"))
+        if self.sigmoid:
+            specs.append(WeightSpec(n["weight_bias"], (self.heads,), role="vector", init="wide_normal"))
         if self.has_output_bias:
             specs.append(WeightSpec(n["o_bias"], (self.hidden,), role="vector", init="small_normal"))
         if self.qk_norm_eps is not None:
@@ -256,6 +275,8 @@ class GroupedQueryAttention(Mixer):
             self.output_bias = tensors[n["o_bias"]]
         if self.learned_sink:
             self.sink_values = tensors[n["sink"]]
+        if self.sigmoid:
+            self.weight_bias = tensors[n["weight_bias"]]
         if self.linear_bias:
             slopes = [2.0 ** (-self.linear_bias_span * (h + 1) / self.heads) for h in range(self.heads)]
             self.slopes = torch.tensor(slopes, dtype=torch.float32, device=tensors[n["q"]].device)
@@ -277,7 +298,7 @@ class GroupedQueryAttention(Mixer):
         slots = ctx.slot_mapping[cache.group]
         if self.unit_store:
             return self._forward_unit(qkv, q, table, slots, ctx, cache)
-        if self.wide_store or self.sink:
+        if self.wide_store or self.sink or self.chunk or self.sigmoid:
             return self._forward_gated(qkv, q, table, slots, ctx, cache)
         args: dict[str, Any] = dict(
             qkv=qkv, heads=self.heads, kv_heads=kv_in, head_dim=d, q_weight=self.q_norm,
@@ -363,7 +384,7 @@ class GroupedQueryAttention(Mixer):
         return self.out.forward(out, ctx, "attn.o")
 
     def _forward_gated(self, qkv, q, table, slots, ctx: StepContext, cache: LayerCache) -> torch.Tensor:
-        """The step with a projection-wide norm, a sink in the softmax or gated heads."""
+        """The step with a projection-wide norm, a sink in the softmax, gated heads, chunks or sigmoid weights."""
         tokens, d = q.shape[0], self.head_dim
         kv_in = 0 if self.reads_shared_cache else self.kv_heads
         if self.position is not None and table is None:
@@ -392,5 +413,6 @@ class GroupedQueryAttention(Mixer):
             q=q, k_pages=cache.k, v_pages=cache.v, block_table=ctx.block_tables[cache.group], ctx=ctx, out=out,
             heads=self.heads, kv_heads=self.kv_heads, head_dim=d, scale=self.scale, window=self.window or 0,
             value_dim=self.value_dim, sink=self.sink, gate=gate, slopes=self.slopes, sink_values=self.sink_values,
+            chunk=self.chunk or 0, sigmoid_bias=self.weight_bias,
         )  # fmt: skip
         return self.out.forward(out, ctx, "attn.o")

@@ -9,7 +9,8 @@ A layer is assembled from parts and an arrangement:
 * a **block** that says how they are wired (pre-norm residual here),
 
 and a mixer may own a **position encoding**.  The model's two ends are parts as well: an
-**embedding** and a **head**.  Each kind has one registry from a name to a
+**embedding** and a **head**; a **junction** is a step on the residual stream in front of an entry
+of the execution order (where a loop over layers starts a pass, say).  Each kind has one registry from a name to a
 class; a :class:`~mini_engine_b200.config.model_spec.PartSpec` names the class and carries
 its constants.  No part reads a model configuration or knows which model it is in.
 
@@ -40,7 +41,9 @@ class PagedCacheSpec:
     With a window, ``keep_first`` tokens at the start of the sequence stay readable for good (their
     pages are never given back).  ``value_dim`` is the width of a value head when it differs from
     ``head_dim``; 0 says that the values are a part of the key rows (a cache of one latent row per token
-    that serves as key and as value), so that no value pages are kept.  Mixers with an equal spec share
+    that serves as key and as value), so that no value pages are kept.  With ``chunk`` (``window`` is then equal to it) a query
+    reads the keys of its own chunk of positions only, ``p // chunk * chunk .. p``, and the pages of earlier chunks are
+    given back.  Mixers with an equal spec share
     one cache group (one page pool, one block table per request).
     """
 
@@ -49,6 +52,7 @@ class PagedCacheSpec:
     window: int | None = None
     value_dim: int | None = None
     keep_first: int = 0
+    chunk: int | None = None
 
     @property
     def v_dim(self) -> int:
@@ -90,6 +94,10 @@ class Residual:
     ``pending_gate`` (partial sums ``[S'', T, hidden]``) with ``pending_gate_bias`` (float32 ``[hidden]``) says that the
     pending output (with its bias) is first multiplied by ``sigmoid(gate + gate_bias)``, and ``pending_norm = (weight, eps)``
     that it is then RMS-normed before it is added to ``x`` (a sublayer between two norms).
+
+    ``replaced`` says that what is pending takes the stream's place: ``x`` holds nothing, the next norm writes it.  ``spare`` is a
+    second buffer of the stream's shape, for norms that write the sum to another place than they read the stream from (they
+    exchange the two).
     """
 
     x: torch.Tensor
@@ -105,6 +113,8 @@ class Residual:
     pending_gate: torch.Tensor | None = None
     pending_gate_bias: torch.Tensor | None = None
     pending_norm: tuple[torch.Tensor, float] | None = None
+    replaced: bool = False
+    spare: torch.Tensor | None = None
 
     def add(self, delta: torch.Tensor, scale: torch.Tensor | None = None, bias: torch.Tensor | None = None) -> None:
         if self.pending is not None:
@@ -123,6 +133,14 @@ class Residual:
         self.pending = self.pending_scale = self.pending_bias = self.pending_more = None
         self.stream_update = self.stream_read = None
         self.pending_gate = self.pending_gate_bias = self.pending_norm = None
+        self.replaced = False
+
+    def replace(self, whole: torch.Tensor, bias: torch.Tensor | None = None) -> None:
+        """``whole`` (partial sums ``[S, T, hidden]``) plus ``bias`` is the stream from now on."""
+        self.clear()
+        self.rounded = None
+        self.add(whole, bias=bias)
+        self.replaced = True
 
 
 @dataclass
@@ -287,6 +305,17 @@ class Head(Part):
         raise NotImplementedError
 
 
+class Junction(Part):
+    """A step on the residual stream in front of an entry of the execution order."""
+
+    def begin(self, state: Residual, ctx: StepContext) -> None:
+        """Called once per step, right behind the embedding (``state.x`` is its output)."""
+
+    def forward(self, state: Residual, ctx: StepContext, turn: int) -> None:
+        """Change the stream; ``turn`` is the entry's number among those of this junction."""
+        raise NotImplementedError
+
+
 class Block(Part):
     """Arrangement of mixer, feed-forward and norms around the residual stream.
 
@@ -345,6 +374,7 @@ POSITION_ENCODINGS: dict[str, Factory] = {}
 BLOCKS: dict[str, Factory] = {}
 EMBEDDINGS: dict[str, Factory] = {}
 HEADS: dict[str, Factory] = {}
+JUNCTIONS: dict[str, Factory] = {}
 
 _REGISTRIES = {
     "mixer": MIXERS,
@@ -354,13 +384,14 @@ _REGISTRIES = {
     "block": BLOCKS,
     "embedding": EMBEDDINGS,
     "head": HEADS,
+    "junction": JUNCTIONS,
 }
 
 
 def register(kind: str, name: str, replace: bool = False) -> Callable[[Factory], Factory]:
     """Class decorator: ``@register("mixer", "gqa_attention")``.
 
-    A mixer, feed-forward, norm or position encoding is built as ``cls(prefix, hidden_size,
+    A mixer, feed-forward, norm, position encoding or junction is built as ``cls(prefix, hidden_size,
     **PartSpec.params)`` where ``prefix`` is the checkpoint prefix of the layer; a block as
     ``cls(mixer, feed_forward, norms)`` with ``norms`` a mapping from the names in its ``NORMS``
     to norm parts; an embedding or a head as ``cls(vocab_size, hidden_size, **PartSpec.params)``.

@@ -7,6 +7,7 @@ import torch
 from mini_engine_b200.csrc import ops
 from mini_engine_b200.parts.base import Block, LayerCache, Residual, StateSpec, StepContext, register
 from mini_engine_b200.parts.linear import Linear
+from mini_engine_b200.parts.norms import DynamicTanh
 from mini_engine_b200.weights.loader import WeightSpec
 
 
@@ -308,3 +309,67 @@ class GatedSandwichMixerOnlyBlock(GatedSandwichBlock):
     """The same arrangement for a layer without a feed-forward: two norms, one gate."""
 
     NORMS = ("mixer", "mixer_out")
+
+
+@register("block", "parallel_two_norms")
+class TwoNormParallelBlock(Block):
+    """Both sublayers read the same stream through a norm of their own: ``x = x + (mixer(norm_m(x)) + feed_forward(norm_f(x)))``.
+    The mixer's input may be shifted by one token: ``h_t + (h_(t-1) - h_t) * shift``, element by element, with ``h = norm_m(x)``
+    and zeros in front of the sequence; the request's last ``h`` is then a state of the block.  The sums are 32-bit; with two
+    dynamic-tanh norms the sum, both norms and the shift are one kernel."""
+
+    capturable = True
+    adds_output_bias = True
+
+    def __init__(self, mixer, feed_forward, norms, *, prefix: str, hidden_size: int, shift: str | None = None, unused_names=()):
+        """``shift``: the name of the shift's weights ``[hidden]`` behind the layer's prefix.  ``unused_names``: tensors of the
+        layer that a checkpoint may carry although the layer has no use for them."""
+        super().__init__(mixer, feed_forward, norms)
+        self.hidden = hidden_size
+        self.shift_name = None if shift is None else prefix + shift
+        self.shift: torch.Tensor | None = None
+        self.unused = [prefix + name for name in unused_names]
+
+    def state(self) -> StateSpec | None:
+        return None if self.shift_name is None else StateSpec((self.hidden,), torch.float32)
+
+    def weight_specs(self) -> list[WeightSpec]:
+        specs = super().weight_specs()
+        if self.shift_name is not None:
+            specs.append(WeightSpec(self.shift_name, (self.hidden,), role="vector", init="small_normal"))
+        return specs + [WeightSpec(name, (), role="vector", optional=True) for name in self.unused]
+
+    def load(self, tensors) -> None:
+        super().load(tensors)
+        if self.shift_name is not None:
+            self.shift = tensors[self.shift_name]
+
+    def _inputs(self, state: Residual, ctx: StepContext, cache: LayerCache) -> tuple[torch.Tensor, torch.Tensor | None]:
+        """What the mixer and the feed-forward read."""
+        first = self.norms["mixer"]
+        second = self.norms["feed_forward"] if self.feed_forward is not None else None
+        if isinstance(first, DynamicTanh) and (second is None or isinstance(second, DynamicTanh)):
+            return first.forward_beside(second, state, ctx, ctx.dtype, self.shift, cache.block_state)
+        h = first.forward(state, ctx, ctx.dtype)
+        if self.shift is not None:
+            shifted = ctx.buffer("block.shifted", (1, *h.shape), h.dtype)
+            ops.token_mix(h=h, mu=self.shift.unsqueeze(0), ctx=ctx, state=cache.block_state, out=shifted)
+            h = shifted[0]
+        elif second is not None:  # the second norm writes where the first one did
+            kept = ctx.buffer("block.kept", tuple(h.shape), h.dtype)
+            kept.copy_(h)
+            h = kept
+        return h, None if second is None else second.forward(state, ctx, ctx.dtype)
+
+    def forward(self, state: Residual, ctx: StepContext, cache: LayerCache) -> None:
+        h, beside = self._inputs(state, ctx, cache)
+        state.add(self.mixer.forward(h, ctx, cache), bias=self.mixer.output_bias)
+        if self.feed_forward is not None:
+            state.add_beside(self.feed_forward.forward(beside, ctx))
+
+
+@register("block", "parallel_two_norms_mixer_only")
+class TwoNormParallelMixerOnlyBlock(TwoNormParallelBlock):
+    """The same arrangement for a layer without a feed-forward: one norm."""
+
+    NORMS = ("mixer",)

@@ -153,3 +153,105 @@ class GatedDeltaRule(Mixer):
             vdim=vdim, gate="sigmoid",
         )  # fmt: skip
         return self.out.forward(gated, ctx, "delta.o")
+
+
+@register("mixer", "generalized_delta_rule")
+class GeneralizedDeltaRule(Mixer):
+    """The delta rule with a removal rate per key channel: what the unit key ``u = k / sqrt(sum k^2 + unit_eps)`` reads of the old
+    state is removed channel by channel, and the key is added as it is.  From the layer's input ``h`` (``heads`` heads of ``dim``)::
+
+        r, k, v = W_r h, W_k h, W_v h        a = sigmoid(W_a h + b_a)
+        w = exp(-decay_scale * sigmoid(W_w2 tanh(W_w1 h) + w0))          (per head and key channel, like a)
+        S <- diag(w) S - (a * u) (u^T S) + k v^T        o = S^T r
+
+    Each head's ``o`` is divided by its root mean square, multiplied by a weight ``[heads * dim]`` and by ``sigmoid(W_g h)``, and
+    the concatenated heads are projected by ``W_o``.  A request's state is ``[heads, dim (values), dim (keys)]`` float32.  All
+    projections of ``h`` run as one product; the tanh of the low-rank sums enters the product with ``W_w2`` as two bfloat16
+    halves, as in :class:`GatedDeltaRule`."""
+
+    capturable = True
+    programmatic_launch = False  # the walk of the gated rule
+
+    def __init__(
+        self, prefix: str, hidden_size: int, *, num_heads: int, head_dim: int, decay_rank: int, norm_eps: float, decay_scale: float,
+        unit_eps: float = 1e-6, names: Mapping[str, str] | None = None,
+    ):  # fmt: skip
+        if min(num_heads, head_dim, decay_rank) < 1 or not decay_scale > 0:
+            raise ValueError("generalized_delta_rule: sizes and decay_scale must be positive")
+        if head_dim > ops.DELTA_MAX_DIM:
+            raise ValueError(f"generalized_delta_rule takes up to {ops.DELTA_MAX_DIM} key channels per head, got {head_dim}")
+        self.hidden, self.heads, self.dim, self.rank = hidden_size, num_heads, head_dim, decay_rank
+        self.eps, self.unit_eps, self.decay_scale = float(norm_eps), float(unit_eps), float(decay_scale)
+        defaults = {"r": "r_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "g": "g_proj.weight", "a": "a_proj.weight",
+                    "a_bias": "a_proj.bias", "w1": "decay_down.weight", "w2": "decay_up.weight", "w0": "decay_up.bias",
+                    "norm": "norm.weight", "o": "o_proj.weight"}  # fmt: skip
+        self.names = {key: prefix + (names or {}).get(key, value) for key, value in defaults.items()}
+        inner = num_heads * head_dim
+        self.columns = {key: i * inner for i, key in enumerate(("r", "k", "v", "a", "g", "w1"))}  # of the fused input projection
+        self.proj: Linear | None = None
+        self.second: Linear | None = None
+        self.out: Linear | None = None
+        self.norm_weight = self.a_bias = self.w0 = None
+
+    def state(self) -> StateSpec:
+        return StateSpec((self.heads * self.dim * self.dim,), torch.float32)
+
+    def weight_specs(self) -> list[WeightSpec]:
+        n, inner = self.names, self.heads * self.dim
+        small = dict(role="vector", init="small_normal")
+        return [
+            *[WeightSpec(n[key], (inner, self.hidden)) for key in ("r", "k", "v", "g", "a")],
+            WeightSpec(n["a_bias"], (inner,), **small),
+            WeightSpec(n["w1"], (self.rank, self.hidden)),
+            WeightSpec(n["w2"], (inner, self.rank)),
+            WeightSpec(n["w0"], (inner,), **small),
+            WeightSpec(n["norm"], (inner,), role="vector", init="ones_normal"),
+            WeightSpec(n["o"], (self.hidden, inner)),
+        ]
+
+    def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        n = self.names
+        rows = [tensors[n[key]] for key in ("r", "k", "v", "a", "g", "w1")]
+        count = sum(r.shape[0] for r in rows)
+        if count % 4:  # rows of zeros: the sums of a token then start on 16 bytes
+            rows.append(torch.zeros(4 - count % 4, self.hidden, dtype=rows[0].dtype, device=rows[0].device))
+        self.proj = Linear(torch.cat(rows, dim=0).contiguous())
+        self.second, self.halves = low_rank_second(tensors[n["w2"]])
+        self.out = Linear(tensors[n["o"]])
+        self.norm_weight, self.a_bias, self.w0 = tensors[n["norm"]], tensors[n["a_bias"]], tensors[n["w0"]]
+
+    def forward(self, h: torch.Tensor, ctx: StepContext, cache: LayerCache) -> torch.Tensor:
+        tokens, heads, dim, at = h.shape[0], self.heads, self.dim, self.columns
+        proj = self.proj.forward(h, ctx, "removal.proj")
+        low = ctx.buffer("removal.low", (tokens, self.halves * self.rank), h.dtype)
+        ops.split_halves(proj, at["w1"], self.rank, low, activate=True)
+        logits = self.second.forward(low, ctx, "removal.second")
+        raw = walk_states(
+            "removal", ctx, cache.state, heads, dim, dim, q=(proj, at["r"]), k=(proj, at["k"]), v=(proj, at["v"]), rate=(proj, at["a"]),
+            logits=(logits, 0), decay_bias=self.w0, channel=self.a_bias, decay_scale=self.decay_scale, unit_eps=self.unit_eps,
+        )  # fmt: skip
+        gated = ctx.buffer("removal.out", (tokens, heads * dim), ctx.dtype)
+        ops.gla_finish(
+            o=raw, proj=proj, gate_column=at["g"], weight=self.norm_weight, eps=self.eps, out=gated, heads=heads, vdim=dim, gate="sigmoid"
+        )
+        return self.out.forward(gated, ctx, "removal.o")
+
+
+def low_rank_second(weight: torch.Tensor) -> tuple[Linear, int]:
+    """The product with the second factor of a low-rank projection, and how many halves its input is cut into: in bfloat16 the
+    32-bit sums enter as two bfloat16 halves each, against the same weight twice."""
+    halves = 2 if weight.dtype == torch.bfloat16 else 1
+    return Linear(torch.cat([weight] * halves, dim=1).contiguous()), halves
+
+
+def walk_states(rule: str, ctx: StepContext, state: torch.Tensor, heads: int, dim: int, vdim: int, **inputs) -> torch.Tensor:
+    """Prepare and walk a recurrence of :data:`ops.STATE_RULES`; returns the heads' outputs ``[T, heads * vdim]`` float32."""
+    tokens = ctx.num_tokens
+    row, numbers = ops.state_rule_floats(rule, dim, vdim)
+    rows = ctx.buffer(f"{rule}.rows", (tokens, heads * row), torch.float32)
+    scalars = ctx.buffer(f"{rule}.scalars", (tokens, heads * numbers), torch.float32)
+    sizes = dict(heads=heads, dim=dim, vdim=vdim)
+    ops.state_prepare(rule=rule, rows=rows, scalars=scalars, **{"rate": None, "unit_eps": 0.0, "decay_scale": 1.0, **inputs}, **sizes)
+    raw = ctx.buffer(f"{rule}.raw", (tokens, heads * vdim), torch.float32)
+    ops.state_walk(rule=rule, rows=rows, scalars=scalars, ctx=ctx, state=state, out=raw, **sizes)
+    return raw

@@ -28,7 +28,7 @@ from mini_engine_b200.parts.base import (
 from mini_engine_b200.weights.loader import WeightSpec
 
 # Importing the built-in parts registers them.
-from mini_engine_b200.parts import attention, block, delta_rule, ends, latent_attention, linear_attention, mlp, moe, norms, parallel, recurrent, rotary  # noqa: F401,E402
+from mini_engine_b200.parts import attention, block, delta_rule, ends, junctions, latent_attention, linear_attention, mlp, moe, norms, parallel, recurrent, rotary, time_mixing  # noqa: F401,E402
 
 
 def build_block(spec: ModelSpec, index: int) -> Block:
@@ -53,6 +53,7 @@ class DecoderModel:
         self.spec = spec
         self.embedding = build_end("embedding", spec.embedding, spec.vocab_size, spec.hidden_size)
         self.blocks = [build_block(spec, i) for i in range(len(spec.layers))]
+        self.junctions = [build_part("junction", part, "", spec.hidden_size) for part in spec.junctions]
         self.final_norm = build_part("norm", spec.final_norm, "", spec.hidden_size)
         self.head = build_end("head", spec.head, spec.vocab_size, spec.hidden_size)
 
@@ -62,6 +63,8 @@ class DecoderModel:
         specs = list(self.embedding.weight_specs())
         for blk in self.blocks:
             specs += blk.weight_specs()
+        for junction in self.junctions:
+            specs += junction.weight_specs()
         specs += self.final_norm.weight_specs()
         specs += self.head.weight_specs()
         return specs
@@ -70,7 +73,7 @@ class DecoderModel:
     def capturable(self) -> bool:
         """Whether every part of the model says that a step of a fixed token count may be captured
         in a CUDA graph (see ``Part.capturable``)."""
-        parts = [self.embedding, self.final_norm, self.head]
+        parts = [self.embedding, self.final_norm, self.head, *self.junctions]
         for blk in self.blocks:
             parts += [blk, *blk.parts()]
             position = getattr(blk.mixer, "position", None)
@@ -81,7 +84,7 @@ class DecoderModel:
     @property
     def programmatic_launch(self) -> bool:
         """Whether every part agrees to programmatic dependent launches (see ``Part.programmatic_launch``)."""
-        parts = [self.embedding, self.final_norm, self.head]
+        parts = [self.embedding, self.final_norm, self.head, *self.junctions]
         for blk in self.blocks:
             parts += [blk, *blk.parts()]
         return all(getattr(part, "programmatic_launch", True) for part in parts)
@@ -107,6 +110,8 @@ class DecoderModel:
         self.embedding.load(tensors)
         for blk in self.blocks:
             blk.load(tensors)
+        for junction in self.junctions:
+            junction.load(tensors)
         self.final_norm.load(tensors)
         self.head.load(tensors)
 
@@ -122,7 +127,11 @@ class DecoderModel:
         x = ctx.buffer("residual", (ctx.num_tokens, self.spec.hidden_size), torch.float32)
         state = Residual(x)
         state.rounded = self.embedding.forward(ctx.token_ids, ctx, x)
+        for junction in self.junctions:
+            junction.begin(state, ctx)
         for entry, cache in zip(self.spec.order, caches, strict=True):
+            if entry.junction is not None:
+                self.junctions[entry.junction].forward(state, ctx, entry.turn)
             self.blocks[entry.layer].forward(state, ctx, cache)
         count = logits_rows.shape[0]
         if count == 0:
