@@ -1,7 +1,7 @@
-"""Prefill and decode throughput of another design (Pimezen, Molotar, Bevadra, Bizurax, Tobadra) beside Qwen3 dense at equal layer sizes.
+"""Prefill and decode throughput of another design (Pimezen, Molotar, Bevadra, Bizurax, Tobadra, Vufadra) beside Qwen3 dense at equal layer sizes.
 
-    python -m mini_engine_b200.cli.design_bench [--design pimezen|molotar|bevadra|bizurax|tobadra] [--sizes 1b,8b] [--steps K] [--warmup W]
-    (or: bench.py --design pimezen|molotar|bevadra|bizurax|tobadra)
+    python -m mini_engine_b200.cli.design_bench [--design pimezen|molotar|bevadra|bizurax|tobadra|vufadra] [--sizes 1b,8b] [--steps K] [--warmup W]
+    (or: bench.py --design pimezen|molotar|bevadra|bizurax|tobadra|vufadra)
     python -m mini_engine_b200.cli.design_bench --design bevadra --sizes 8b --capture prompt|decode   (a few eager steps, for a profiler)
 
 For each size both models get the same width, feed-forward width, head counts, head size, layer count
@@ -39,6 +39,12 @@ layers have a tanh-GELU feed-forward one and a half times as wide as Qwen3's (th
 units three eighths as wide beside 2 units that return their input, in 2 groups of which 1 is kept, of which a token uses
 2, beside a gated shared unit three quarters as wide (a token whose units both have tensors uses as many feed-forward
 weights as in Qwen3).  Every sublayer has a gate of width x width beside these.
+
+Vufadra gets four layers in the order generalized delta rule, parallel, gated linear recurrence, parallel.  Its attention branch
+has Qwen3's head counts and head size and chunks of 1,280 positions (the decode steps read 768 keys and more of their chunk);
+delta rule and time mixing have heads of 64 that fill the model's width and a decay rank of 64; the recurrence is as wide as
+the model with blocks of 128 channels and four taps; its feed-forward is Qwen3's.  The last three layers are a loop that runs
+once, so that its product of 2 x width onto width runs once in four layers.
 """
 
 from __future__ import annotations
@@ -63,12 +69,14 @@ TIMED = ("biased_attention", "mixed_attention", "gla_scan", "gla_finish", "branc
          "qk_wide_norm_rope_store", "pair_embedding", "round_rows", "gemm_tensor_core_grouped", "sort_by_unit", "gather_rows",
          "combine_rows", "add_layernorm", "latent_down_finish", "head_product", "logits_finish", "retention_scan", "hyper_step",
          "activation", "qkv_rope_unit_store", "sandwich_norm", "input_convolution", "turn_heads_back", "split_halves",
-         "delta_prepare", "delta_scan", "moe_finish", "gemm_tensor_core_activated")  # fmt: skip
+         "delta_prepare", "delta_scan", "moe_finish", "gemm_tensor_core_activated", "state_prepare", "state_walk", "tanh_norms",
+         "token_mix", "branch_norm_sum", "sum_rows")  # fmt: skip
 STREAMS, ROUTED_UNITS, ROUTED_USED = 4, 8, 2
 LATENT_RANK, LATENT_ROT = 512, 64
 UNITS, UNITS_USED, UNIT_GROUPS, UNIT_GROUPS_KEPT = 8, 2, 4, 2
 RECURRENCE_BLOCK, RECURRENCE_TAPS = 128, 4
 TAPS, PASSED_UNITS = 4, 2
+CHUNK, STATE_DIM, STATE_RANK = 1280, 64, 64
 
 
 def molotar_config(size: dict):
@@ -139,6 +147,23 @@ def tobadra_config(size: dict):
                                     "canon": {"taps": TAPS}, "logit_scale": 0.25, "layers": layers})  # fmt: skip
 
 
+def vufadra_config(size: dict):
+    from mini_engine_b200.config import VufadraConfig
+
+    d, width = size["head_dim"], size["width"]
+    left = {"heads": size["heads"], "kv_heads": size["kv_heads"], "dim": d, "vdim": d, "scale": d**-0.5, "mask": {"size": CHUNK},
+            "rot": {"base": 5e5, "dims": d, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}  # fmt: skip
+    states = {"heads": width // STATE_DIM, "dim": STATE_DIM, "decay_rank": STATE_RANK}
+    recurrence = {"width": width, "blocks": width // RECURRENCE_BLOCK, "conv": RECURRENCE_TAPS}
+    both = ("parallel", {"left": left, "right": states})
+    pattern = [("general_delta", states), both, ("rglru", recurrence), both]
+    layers = [{"type": kind, "mixer": mixer, "mlp": {"kind": "dense", "ff": size["ff"]}} for kind, mixer in (pattern * size["layers"])[: size["layers"]]]
+    return VufadraConfig.from_dict({
+        "architecture": "Vufadra", "vocab": size["vocab"], "width": width, "norm": {"eps": 1e-6}, "layers": layers,
+        "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}}, "loop": {"start": 1, "stop": size["layers"], "times": 1},
+    })  # fmt: skip
+
+
 def configs(size: dict, design: str = "pimezen"):
     from mini_engine_b200.config import PimezenConfig, Qwen3Config
 
@@ -167,6 +192,8 @@ def configs(size: dict, design: str = "pimezen"):
         return {"bizurax": bizurax_config(size), "qwen3": qwen}
     if design == "tobadra":
         return {"tobadra": tobadra_config(size), "qwen3": qwen}
+    if design == "vufadra":
+        return {"vufadra": vufadra_config(size), "qwen3": qwen}
     return {"pimezen": pimezen, "qwen3": qwen}
 
 
@@ -186,6 +213,8 @@ class KernelTimes:
             def timed(*args, _name=name, _function=function, **kwargs):
                 if _name == "paged_attention" and kwargs.get("v_pages", 0) is None:
                     _name = "latent_attention"  # the same entry point over a cache of latent rows
+                if _name.startswith("state_"):
+                    _name += "." + kwargs["rule"]
                 start, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
                 start.record()
                 result = _function(*args, **kwargs)
@@ -354,6 +383,41 @@ def rooflines(design: str, size: dict, peaks: dict) -> dict:
             factor = share[name.split(".")[1]]
             nbytes, nflops = out[name]["bytes"] * factor, out[name]["flops"] * factor
             out[name] = {"bytes": nbytes, "flops": nflops, "roofline_us": max(nbytes / bw, nflops / flops) * 1e6}
+    elif design == "vufadra":
+        n, c = width, width  # columns of the states' projections (heads x dim), channels of the recurrence
+        chunk_sum = lambda begin, end: sum(p % CHUNK + 1 for p in range(begin, end))  # noqa: E731
+        for phase, tokens, seen in (("prompt", PROMPT, chunk_sum(0, PROMPT)), ("decode", BATCH, BATCH * chunk_sum(CONTEXT, CONTEXT + 1))):
+            keys = tokens if phase == "prompt" else seen
+            bound(f"{phase}.paged_attention", (keys * 2 * g * d + tokens * 2 * h * d) * 2, seen * 4 * h * d)
+            states = (1 if phase == "prompt" else BATCH) * 2 * n * STATE_DIM * 4
+            for rule, vectors, sums in (("removal", 4, 5), ("bonus", 3, 4)):
+                bound(f"{phase}.state_prepare.{rule}", tokens * n * (sums + vectors + 1) * 4, 0)
+                bound(f"{phase}.state_walk.{rule}", tokens * n * (vectors + 2) * 4 + states, tokens * n * STATE_DIM * (8 if rule == "removal" else 6))
+            gates = 2 * c * RECURRENCE_BLOCK
+            past = 0 if phase == "prompt" else 2 * RECURRENCE_TAPS * 4
+            bound(f"{phase}.rglru", tokens * c * (2 * 4 + 4 * 4 + 2 + past) + gates * 4, 2 * tokens * gates)
+            # stream and both outputs in, the stream and both inputs out; the mixes; the two branches
+            bound(f"{phase}.tanh_norms", tokens * width * (4 + 2 * 4 + 4 + 2 * 2), 0)
+            bound(f"{phase}.token_mix", tokens * width * 6 * 2, 0)
+            bound(f"{phase}.branch_norm_sum", tokens * width * 3 * 4, 0)
+            bound(f"{phase}.sum_rows", tokens * width * (4 + 2 * 4 + 2 + 4 + 2), 0)
+            bound(f"{phase}.gla_finish", tokens * n * (4 + 4 + 2), 0)
+        attention = width * (h * d + 2 * g * d) + h * d * width
+        mixing = 5 * width * n + STATE_RANK * (width + n)
+        removal = 6 * width * n + STATE_RANK * (width + n)
+        mixer = (removal + 2 * (attention + mixing) + 3 * width * c + 2 * width * width) / 4  # and the loop's product
+        dense = 3 * width * ff
+        for phase, tokens in (("prompt", PROMPT), ("decode", BATCH)):
+            nbytes, nflops = (mixer + dense) * 2, 2 * tokens * (mixer + dense)
+            out[f"{phase}.products"] = {"bytes": nbytes, "flops": nflops, "roofline_us": max(nbytes / bw, nflops / flops) * 1e6,
+                                        "kernels": ("gemm_tensor_core", "gemm_tensor_core_swiglu", "swiglu")}  # fmt: skip
+        # kernel times are averaged over all layers: half are parallel, a quarter have the delta rule, a quarter the recurrence
+        share = {"paged_attention": 0.5, "state_prepare.bonus": 0.5, "state_walk.bonus": 0.5, "token_mix": 0.5, "branch_norm_sum": 0.5,
+                 "state_prepare.removal": 0.25, "state_walk.removal": 0.25, "rglru": 0.25, "sum_rows": 0.25, "gla_finish": 0.75}  # fmt: skip
+        for name in [k for k in out if k.split(".", 1)[1] in share]:
+            factor = share[name.split(".", 1)[1]]
+            nbytes, nflops = out[name]["bytes"] * factor, out[name]["flops"] * factor
+            out[name] = {"bytes": nbytes, "flops": nflops, "roofline_us": max(nbytes / bw, nflops / flops) * 1e6}
     elif design == "qwen3":
         mixer = width * (h * d + 2 * g * d) + h * d * width
         dense = 3 * width * ff
@@ -470,8 +534,8 @@ def layer_weight_bytes(model, layers: int) -> int:
     import math
 
     total = 0
-    for blk in model.blocks:
-        for spec in blk.weight_specs():
+    for part in [*model.blocks, *model.junctions]:
+        for spec in part.weight_specs():
             if spec.alias_of is None and not spec.optional:
                 total += math.prod(spec.shape) * (2 if spec.role == "matrix" else 4)
     return total // layers
@@ -531,7 +595,7 @@ def capture_steps(design: str, size_name: str, phase: str) -> None:
 
 def main(argv=None) -> int:
     parser = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
-    parser.add_argument("--design", choices=["pimezen", "molotar", "bevadra", "bizurax", "tobadra"], default="pimezen")
+    parser.add_argument("--design", choices=["pimezen", "molotar", "bevadra", "bizurax", "tobadra", "vufadra"], default="pimezen")
     parser.add_argument("--sizes", default="1b,8b")
     parser.add_argument("--steps", type=int, default=32)
     parser.add_argument("--warmup", type=int, default=5)

@@ -15,6 +15,7 @@ from mini_engine_b200.config.registry import (
     registered_architectures,
 )
 from mini_engine_b200.config.tobadra import TobadraConfig
+from mini_engine_b200.config.vufadra import VufadraConfig
 
 __all__ = [
     "Architecture",
@@ -29,6 +30,7 @@ __all__ = [
     "PimezenConfig",
     "Qwen3Config",
     "TobadraConfig",
+    "VufadraConfig",
     "architecture_for",
     "load_model_config",
     "register_architecture",
