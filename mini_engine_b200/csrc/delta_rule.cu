@@ -498,8 +498,98 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) state_prepare_kernel(StatePre
     }
 }
 
+// The same for key heads of 4 LANES channels and value heads as wide, with every row and range on 16 bytes: a lane takes four
+// neighbouring channels, a warp 32 / LANES heads of one token.  All loads of a lane are issued before any is used.
+template <int RULE, int LANES>
+__global__ void __launch_bounds__(PREP_WARPS * 32) state_prepare_vec_kernel(StatePrepArgs a) {
+    constexpr int VECTORS = Rule<RULE>::VECTORS, HEADS = 32 / LANES, DIM = 4 * LANES;
+    const int lane = threadIdx.x & 31, part = lane % LANES;
+    const int head = (blockIdx.y * PREP_WARPS + (threadIdx.x >> 5)) * HEADS + lane / LANES;
+    const size_t token = blockIdx.x;
+    const int column = head * DIM + part * 4;
+    const bool live = head < a.heads;
+    pdl_trigger();
+    pdl_wait();
+    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    auto fetch = [&](const Columns& range) {
+        float4 sum = zero;
+        const float* src = range.sums + token * range.width + column;
+#pragma unroll 4
+        for (int s = 0; s < range.splits; ++s) {
+            const float4 x = *reinterpret_cast<const float4*>(src + s * range.stride);
+            sum.x += x.x, sum.y += x.y, sum.z += x.z, sum.w += x.w;
+        }
+        return sum;
+    };
+    float4 q4 = zero, k4 = zero, v4 = zero, z4 = zero, r4 = zero, b4 = zero, c4 = zero;
+    if (live) {
+        q4 = fetch(a.q), k4 = fetch(a.k), v4 = fetch(a.v), z4 = fetch(a.logits);
+        if constexpr (RULE == RULE_REMOVAL) r4 = fetch(a.rate);
+        b4 = *reinterpret_cast<const float4*>(a.decay_bias + column), c4 = *reinterpret_cast<const float4*>(a.channel + column);
+    }
+    const float q[4] = {q4.x, q4.y, q4.z, q4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w};
+    const float z[4] = {z4.x + b4.x, z4.y + b4.y, z4.z + b4.z, z4.w + b4.w};
+    const float channel[4] = {r4.x + c4.x, r4.y + c4.y, r4.z + c4.z, r4.w + c4.w};
+    float decay[4], first[4], removed[4];
+    float squares = 0.0f, dot = 0.0f, weighted = 0.0f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        if constexpr (RULE == RULE_REMOVAL) {
+            decay[i] = 1.0f + expm1f(-a.decay_scale / (1.0f + expf(-z[i])));
+            removed[i] = k[i] / (1.0f + expf(-channel[i]));
+            first[i] = q[i] * decay[i];
+            squares = fmaf(k[i], k[i], squares);
+            dot = fmaf(q[i], k[i], dot);
+            weighted = fmaf(q[i], removed[i], weighted);
+        } else {
+            decay[i] = 1.0f + expm1f(-expf(z[i]));
+            first[i] = q[i];
+            weighted = fmaf(q[i] * channel[i], k[i], weighted);
+        }
+    }
+#pragma unroll
+    for (int offset = LANES / 2; offset > 0; offset >>= 1) {
+        weighted += __shfl_xor_sync(0xffffffffu, weighted, offset);
+        if constexpr (RULE == RULE_REMOVAL) {
+            squares += __shfl_xor_sync(0xffffffffu, squares, offset);
+            dot += __shfl_xor_sync(0xffffffffu, dot, offset);
+        }
+    }
+    if (!live) return;
+    float* row = a.rows + (token * a.heads + head) * ((VECTORS + 1) * DIM) + part * 4;
+    *reinterpret_cast<float4*>(row) = make_float4(first[0], first[1], first[2], first[3]);
+    *reinterpret_cast<float4*>(row + DIM) = k4;
+    *reinterpret_cast<float4*>(row + 2 * DIM) = make_float4(decay[0], decay[1], decay[2], decay[3]);
+    if constexpr (RULE == RULE_REMOVAL) *reinterpret_cast<float4*>(row + 3 * DIM) = make_float4(removed[0], removed[1], removed[2], removed[3]);
+    *reinterpret_cast<float4*>(row + VECTORS * DIM) = v4;
+    if (part) return;
+    float* scalars = a.scalars + (token * a.heads + head) * Rule<RULE>::SCALARS;
+    if constexpr (RULE == RULE_REMOVAL) {
+        const float inverse = 1.0f / (squares + a.unit_eps);
+        *reinterpret_cast<float4*>(scalars) = make_float4(inverse, inverse * weighted, dot, 0.0f);
+    } else {
+        *reinterpret_cast<float2*>(scalars) = make_float2(weighted, 0.0f);
+    }
+}
+
+static bool takes_vectors(const Columns& c) { return c.width % 4 == 0 && c.stride % 4 == 0 && reinterpret_cast<uintptr_t>(c.sums) % 16 == 0; }
+
+template <int RULE, int LANES>
+static int launch_state_prepare_vec(const StatePrepArgs& a, cudaStream_t stream) {
+    constexpr int HEADS = PREP_WARPS * 32 / LANES;
+    return launch_kernel(state_prepare_vec_kernel<RULE, LANES>, dim3(a.tokens, (a.heads + HEADS - 1) / HEADS), PREP_WARPS * 32, 0, stream, a);
+}
+
 template <int RULE>
 static int launch_state_prepare(const StatePrepArgs& a, cudaStream_t stream) {
+    const auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+    // the choice follows from the sizes and the engine's buffers alone
+    if (a.vdim == a.dim && takes_vectors(a.q) && takes_vectors(a.k) && takes_vectors(a.v) && takes_vectors(a.logits) &&
+        (RULE != RULE_REMOVAL || takes_vectors(a.rate)) && aligned(a.decay_bias) && aligned(a.channel) && aligned(a.rows) && aligned(a.scalars)) {
+        if (a.dim == 32) return launch_state_prepare_vec<RULE, 8>(a, stream);
+        if (a.dim == 64) return launch_state_prepare_vec<RULE, 16>(a, stream);
+        if (a.dim == 128) return launch_state_prepare_vec<RULE, 32>(a, stream);
+    }
     const long long items = static_cast<long long>(a.tokens) * a.heads;
     const int blocks = static_cast<int>((items + PREP_WARPS - 1) / PREP_WARPS);
     if (a.dim <= 32) return launch_kernel(state_prepare_kernel<RULE, 1>, blocks, PREP_WARPS * 32, 0, stream, a);
@@ -757,6 +847,44 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32) delta_scan_kernel(Delta
         };
         TokenRow<R, VECTORS> even, odd;
         even.template load<L>(rows_s);
+        if constexpr (RULE == RULE_BONUS && C == 2 && L == 8) {
+            // Nothing but the output waits for a token's sum over the lanes: two tokens walk, then their four sums (two
+            // columns each) are added together, each lane keeping half of what it holds: 4 + 2 + 1 lanes away.
+            auto advance = [&](const TokenRow<R, VECTORS>& row, int t, float (&sum)[C]) {
+#pragma unroll
+                for (int c = 0; c < C; ++c) {
+                    const float value = v_s[t * columns + local_column + c * GROUPS];
+                    const float2 vv = make_float2(value, value);
+                    float2 on_q[2] = {make_float2(0.0f, 0.0f), make_float2(0.0f, 0.0f)};
+#pragma unroll
+                    for (int i = 0; i < R / 2; ++i) {
+                        on_q[i & 1] = __ffma2_rn(row.q[i], s[c][i], on_q[i & 1]);
+                        s[c][i] = __ffma2_rn(row.g[i], s[c][i], __fmul2_rn(row.k[i], vv));
+                    }
+                    sum[c] = (on_q[0].x + on_q[0].y) + (on_q[1].x + on_q[1].y);
+                }
+            };
+            const bool second_token = part & 4, second_column = part & 2;
+            const int my_column = local_column + (second_column ? GROUPS : 0);
+#pragma unroll 1
+            for (int t = 0; t < count; t += 2) {
+                float first[C], second[C] = {0.0f, 0.0f};
+                const bool more = t + 1 < count;
+                if (more) odd.template load<L>(rows_s + (t + 1) * VECTORS * DP);
+                advance(even, t, first);
+                if (t + 2 < count) even.template load<L>(rows_s + (t + 2) * VECTORS * DP);
+                if (more) advance(odd, t + 1, second);
+                float kept[C];
+#pragma unroll
+                for (int c = 0; c < C; ++c)
+                    kept[c] = (second_token ? second[c] : first[c]) + __shfl_xor_sync(0xffffffffu, second_token ? first[c] : second[c], 4);
+                float sum = (second_column ? kept[1] : kept[0]) + __shfl_xor_sync(0xffffffffu, second_column ? kept[0] : kept[1], 2);
+                sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+                const int mine = t + (second_token ? 1 : 0);
+                if ((part & 1) == 0 && mine < count)
+                    results[(buffer * SC + mine) * columns + my_column] = fmaf(scalars_s[SCALARS * mine], v_s[mine * columns + my_column], sum);
+            }
+        } else
 #pragma unroll 1
         for (int t = 0; t < count; t += 2) {
             if (t + 1 < count) odd.template load<L>(rows_s + (t + 1) * VECTORS * DP);
@@ -807,8 +935,8 @@ static int launch_delta_scan(const DeltaScanArgs& a, int entries, cudaStream_t s
 
 template <int RULE>
 static int dispatch_delta_scan(const DeltaScanArgs& a, int entries, cudaStream_t stream) {
-    if (a.dim <= 32) return launch_delta_scan<RULE, 8, 4, 1, 16>(a, entries, stream);
-    if (a.dim <= 64) return launch_delta_scan<RULE, 8, 8, 1, 16>(a, entries, stream);
+    if (a.dim <= 32) return launch_delta_scan<RULE, 8, 4, 2, 16>(a, entries, stream);
+    if (a.dim <= 64) return launch_delta_scan<RULE, 8, 8, 2, 16>(a, entries, stream);
     if (a.dim <= 128) return launch_delta_scan<RULE, 8, 16, 2, 16>(a, entries, stream);
     if (a.dim <= 256) return launch_delta_scan<RULE, 16, 16, 2, 8>(a, entries, stream);
     if (a.dim > MAX_DIM) return ME_ERR_UNSUPPORTED;

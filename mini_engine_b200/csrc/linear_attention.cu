@@ -702,6 +702,62 @@ __global__ void __launch_bounds__(128) gla_finish_kernel(const float* __restrict
     }
 }
 
+// The same for heads of 4 LANES columns with every row on 16 bytes: a lane takes four neighbouring columns, a warp 32 / LANES
+// heads of one token.
+template <typename T, int LANES>
+__global__ void __launch_bounds__(128) gla_finish_vec_kernel(const float* __restrict__ o, const float* __restrict__ proj, int splits,
+                                                             size_t split_stride, int width, int g_col, const float* __restrict__ weight,
+                                                             float eps, T* __restrict__ out, int heads, int gate_kind, int weight_step) {
+    constexpr int HEADS = 32 / LANES, DIM = 4 * LANES;
+    const int lane = threadIdx.x & 31, part = lane % LANES;
+    const int head = (blockIdx.y * 4 + (threadIdx.x >> 5)) * HEADS + lane / LANES;
+    const size_t token = blockIdx.x;
+    const bool live = head < heads;
+    pdl_trigger();
+    pdl_wait();
+    float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f), g = x, w = make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+    const int column = head * DIM + part * 4;
+    if (live) {
+        x = *reinterpret_cast<const float4*>(o + token * heads * DIM + column);
+        const float* gate_row = proj + token * width + g_col + column;
+#pragma unroll 4
+        for (int p = 0; p < splits; ++p) {
+            const float4 part4 = *reinterpret_cast<const float4*>(gate_row + p * split_stride);
+            g.x += part4.x, g.y += part4.y, g.z += part4.z, g.w += part4.w;
+        }
+        if (weight) w = *reinterpret_cast<const float4*>(weight + head * weight_step + part * 4);
+    }
+    float sum_sq = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w)));
+#pragma unroll
+    for (int offset = LANES / 2; offset > 0; offset >>= 1) sum_sq += __shfl_xor_sync(0xffffffffu, sum_sq, offset);
+    if (!live) return;
+    const float inv = rsqrtf(sum_sq / static_cast<float>(DIM) + eps);
+    const float y[4] = {w.x * (x.x * inv) * finish_gate(g.x, gate_kind), w.y * (x.y * inv) * finish_gate(g.y, gate_kind),
+                        w.z * (x.z * inv) * finish_gate(g.z, gate_kind), w.w * (x.w * inv) * finish_gate(g.w, gate_kind)};
+    T* dst = out + token * heads * DIM + column;
+    if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(dst) = make_float4(y[0], y[1], y[2], y[3]);
+    } else {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(y[0], y[1]), b = __floats2bfloat162_rn(y[2], y[3]);
+        *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+    }
+}
+
+template <typename T, int LANES>
+static int launch_gla_finish_vec(const float* o, const float* proj, int splits, size_t stride, int width, int g_col, const float* weight,
+                                 float eps, void* out, int tokens, int heads, int gate_kind, int weight_step, cudaStream_t stream) {
+    constexpr int HEADS = 4 * 32 / LANES;
+    return launch_kernel(gla_finish_vec_kernel<T, LANES>, dim3(tokens, (heads + HEADS - 1) / HEADS), 128, 0, stream, o, proj, splits, stride,
+                         width, g_col, weight, eps, static_cast<T*>(out), heads, gate_kind, weight_step);
+}
+
+template <int LANES>
+static int launch_gla_finish_vec(int type, const float* o, const float* proj, int splits, size_t stride, int width, int g_col, const float* weight,
+                                 float eps, void* out, int tokens, int heads, int gate_kind, int weight_step, cudaStream_t stream) {
+    return type == ME_BF16 ? launch_gla_finish_vec<__nv_bfloat16, LANES>(o, proj, splits, stride, width, g_col, weight, eps, out, tokens, heads, gate_kind, weight_step, stream)
+                           : launch_gla_finish_vec<float, LANES>(o, proj, splits, stride, width, g_col, weight, eps, out, tokens, heads, gate_kind, weight_step, stream);
+}
+
 // The same with the root mean square over all `count` columns of a token (every head together) and a weight of that size.
 // One block per token; V columns per thread and step (4: 16-byte loads), whose squares a thread adds in ascending order.
 template <typename T, int V>
@@ -784,6 +840,15 @@ ME_EXPORT int me_gla_finish(const float* o, const float* proj, int splits, long 
         auto* dst = static_cast<float*>(out);
         return vec ? launch_kernel(projection_finish_kernel<float, 4>, tokens, 256, 0, stream, o, proj, splits, stride, width, g_col, weight, eps, dst, count, gate_kind)
                    : launch_kernel(projection_finish_kernel<float, 1>, tokens, 256, 0, stream, o, proj, splits, stride, width, g_col, weight, eps, dst, count, gate_kind);
+    }
+    {
+        const auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+        const size_t stride = static_cast<size_t>(split_stride);
+        if (width % 4 == 0 && g_col % 4 == 0 && split_stride % 4 == 0 && aligned(o) && aligned(proj) && aligned(weight) && aligned(out)) {
+            if (vdim == 32) return launch_gla_finish_vec<8>(type, o, proj, splits, stride, width, g_col, weight, eps, out, tokens, heads, gate_kind, weight_step, stream);
+            if (vdim == 64) return launch_gla_finish_vec<16>(type, o, proj, splits, stride, width, g_col, weight, eps, out, tokens, heads, gate_kind, weight_step, stream);
+            if (vdim == 128) return launch_gla_finish_vec<32>(type, o, proj, splits, stride, width, g_col, weight, eps, out, tokens, heads, gate_kind, weight_step, stream);
+        }
     }
     const long long items = static_cast<long long>(tokens) * heads;
     const int blocks = static_cast<int>((items + 3) / 4);

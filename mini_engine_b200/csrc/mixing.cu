@@ -17,6 +17,7 @@
 
 constexpr int MIX_THREADS = 128;
 constexpr int MIX_RUN = 8;            // tokens of a thread in a long step
+constexpr int TANH_RUN = 4;           // the same for the norms, which hold more of a token
 constexpr int MIX_RUN_TOKENS = 512;   // from this many tokens on
 
 template <int V>
@@ -68,10 +69,20 @@ struct StreamSum {
     const float* bias;  // [width]
     int width;
 
-    template <int V>
+    // WHOLE: there is a stream and each sublayer brings one sum (the steps of many tokens, whose products are not split).
+    template <int V, bool WHOLE = false>
     __device__ __forceinline__ void load(size_t token, int column, float (&sum)[V]) const {
         const size_t at = token * width + column;
         float part[V];
+        if constexpr (WHOLE) {
+            float y[V];
+            load_columns<V>(first + at, sum);
+            load_columns<V>(second + at, y);
+            load_columns<V>(x + at, part);
+#pragma unroll
+            for (int i = 0; i < V; ++i) sum[i] = (sum[i] + y[i]) + part[i];
+            return;
+        }
 #pragma unroll
         for (int i = 0; i < V; ++i) sum[i] = 0.0f;
         if (first) {
@@ -126,6 +137,18 @@ struct TanhArgs {
     int tokens, width;
 };
 
+// tanh from the exponential, 1 - 2 / (e^(2|z|) + 1), and below a quarter, where that difference loses digits, from its power
+// series up to z^9 (the next term is 2e-9 of the value there).
+__device__ __forceinline__ float tanh_of(float z) {
+    const float size = fabsf(z), square = z * z;
+    float series = fmaf(square, 62.0f / 2835.0f, -17.0f / 315.0f);
+    series = fmaf(series, square, 2.0f / 15.0f);
+    series = fmaf(series, square, -1.0f / 3.0f);
+    series = fmaf(series * square, z, z);
+    const float far = copysignf(1.0f - __fdividef(2.0f, __expf(fminf(2.0f * size, 80.0f)) + 1.0f), z);
+    return size < 0.25f ? series : far;
+}
+
 template <int V>
 struct TanhColumns {
     float weight[V], bias[V], alpha;
@@ -136,11 +159,11 @@ struct TanhColumns {
     }
     __device__ __forceinline__ void apply(const float (&x)[V], float (&y)[V]) const {
 #pragma unroll
-        for (int i = 0; i < V; ++i) y[i] = fmaf(tanhf(alpha * x[i]), weight[i], bias[i]);
+        for (int i = 0; i < V; ++i) y[i] = fmaf(tanh_of(alpha * x[i]), weight[i], bias[i]);
     }
 };
 
-template <typename OutT, int V, int RUN>
+template <typename OutT, int V, int RUN, bool WHOLE = false>
 __global__ void __launch_bounds__(MIX_THREADS) tanh_norms_kernel(TanhArgs a) {
     const int column = (blockIdx.y * MIX_THREADS + threadIdx.x) * V, begin = blockIdx.x * RUN;
     if (column >= a.width) return;
@@ -154,7 +177,7 @@ __global__ void __launch_bounds__(MIX_THREADS) tanh_norms_kernel(TanhArgs a) {
     float x[RUN][V];
 #pragma unroll
     for (int t = 0; t < RUN; ++t)
-        if (begin + t < a.tokens) a.sum.template load<V>(a.rows ? a.rows[begin + t] : begin + t, column, x[t]);
+        if (begin + t < a.tokens) a.sum.template load<V, WHOLE>(a.rows ? a.rows[begin + t] : begin + t, column, x[t]);
     float previous[V];
 #pragma unroll
     for (int t = 0; t < RUN; ++t) {
@@ -179,12 +202,12 @@ __global__ void __launch_bounds__(MIX_THREADS) tanh_norms_kernel(TanhArgs a) {
                 if (last == token) {
                     store_columns<V>(slot, h);
                 } else {
-                    a.sum.template load<V>(last, column, newest);
+                    a.sum.template load<V, WHOLE>(last, column, newest);
                     first.apply(newest, newest);
                     store_columns<V>(slot, newest);
                 }
             } else if (t == 0) {
-                a.sum.template load<V>(token - 1, column, previous);
+                a.sum.template load<V, WHOLE>(token - 1, column, previous);
                 first.apply(previous, previous);
             }
 #pragma unroll
@@ -214,11 +237,13 @@ static int launch_tanh_norms(const TanhArgs& a, cudaStream_t stream) {
     // the choice of vectors follows from the sizes and the engine's buffers alone
     bool vector = sum_takes_vectors(a.sum) && aligned(a.x_out) && aligned(a.shift) && aligned(a.state);
     for (const TanhNorm& n : a.norms) vector = vector && aligned(n.weight) && aligned(n.bias) && aligned(n.out);
-    const int columns = MIX_THREADS * (vector ? 4 : 1), run = a.tokens >= MIX_RUN_TOKENS && vector ? MIX_RUN : 1;
+    const int columns = MIX_THREADS * (vector ? 4 : 1), run = a.tokens >= MIX_RUN_TOKENS && vector ? TANH_RUN : 1;
     const dim3 grid((a.tokens + run - 1) / run, (a.width + columns - 1) / columns);
     if (!vector) return launch_kernel(tanh_norms_kernel<OutT, 1, 1>, grid, MIX_THREADS, 0, stream, a);
     if (run == 1) return launch_kernel(tanh_norms_kernel<OutT, 4, 1>, grid, MIX_THREADS, 0, stream, a);
-    return launch_kernel(tanh_norms_kernel<OutT, 4, MIX_RUN>, grid, MIX_THREADS, 0, stream, a);
+    if (a.sum.x && a.sum.first && a.sum.first_splits == 1 && a.sum.second && a.sum.second_splits == 1 && !a.sum.bias)
+        return launch_kernel(tanh_norms_kernel<OutT, 4, TANH_RUN, true>, grid, MIX_THREADS, 0, stream, a);
+    return launch_kernel(tanh_norms_kernel<OutT, 4, TANH_RUN>, grid, MIX_THREADS, 0, stream, a);
 }
 
 ME_EXPORT int me_tanh_norms(const float* x, const float* first, int first_splits, long long first_stride, const float* second,
