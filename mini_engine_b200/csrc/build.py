@@ -41,6 +41,7 @@ LIBRARIES = {
     "sandwich": "sandwich.cu",
     "delta_rule": "delta_rule.cu",
     "mixing": "mixing.cu",
+    "state_chunks": "state_chunks.cu",
     "recurrent": "recurrent.cu",
     "routing": "routing.cu",
     "gemm_tcgen05": "gemm_tcgen05.cu",

@@ -637,6 +637,7 @@ struct DeltaScanArgs {
     size_t slot_floats;
     float* out;  // [tokens][heads][vdim]
     int heads, qk_heads, dim, vdim, vector;  // vector: 16-byte loads are aligned
+    int max_count = 0;                       // > 0: entries with more tokens than this are left to the chunked kernels
 };
 
 __device__ __forceinline__ void copy_async_16(float* shared_dst, const float* global_src) {
@@ -694,6 +695,7 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32) delta_scan_kernel(Delta
         staged[stage * stage_floats + (j / (DP - dim)) * DP + dim + j % (DP - dim)] = 0.0f;
     }
     const int begin = a.cu_tokens[entry], end = a.cu_tokens[entry + 1];
+    if (a.max_count > 0 && end - begin > a.max_count) return;
     float* state = a.state + static_cast<size_t>(a.state_slots[entry]) * a.slot_floats +
                    (static_cast<size_t>(head) * a.vdim + first_column + local_column) * dim;
 
@@ -847,44 +849,6 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32) delta_scan_kernel(Delta
         };
         TokenRow<R, VECTORS> even, odd;
         even.template load<L>(rows_s);
-        if constexpr (RULE == RULE_BONUS && C == 2 && L == 8) {
-            // Nothing but the output waits for a token's sum over the lanes: two tokens walk, then their four sums (two
-            // columns each) are added together, each lane keeping half of what it holds: 4 + 2 + 1 lanes away.
-            auto advance = [&](const TokenRow<R, VECTORS>& row, int t, float (&sum)[C]) {
-#pragma unroll
-                for (int c = 0; c < C; ++c) {
-                    const float value = v_s[t * columns + local_column + c * GROUPS];
-                    const float2 vv = make_float2(value, value);
-                    float2 on_q[2] = {make_float2(0.0f, 0.0f), make_float2(0.0f, 0.0f)};
-#pragma unroll
-                    for (int i = 0; i < R / 2; ++i) {
-                        on_q[i & 1] = __ffma2_rn(row.q[i], s[c][i], on_q[i & 1]);
-                        s[c][i] = __ffma2_rn(row.g[i], s[c][i], __fmul2_rn(row.k[i], vv));
-                    }
-                    sum[c] = (on_q[0].x + on_q[0].y) + (on_q[1].x + on_q[1].y);
-                }
-            };
-            const bool second_token = part & 4, second_column = part & 2;
-            const int my_column = local_column + (second_column ? GROUPS : 0);
-#pragma unroll 1
-            for (int t = 0; t < count; t += 2) {
-                float first[C], second[C] = {0.0f, 0.0f};
-                const bool more = t + 1 < count;
-                if (more) odd.template load<L>(rows_s + (t + 1) * VECTORS * DP);
-                advance(even, t, first);
-                if (t + 2 < count) even.template load<L>(rows_s + (t + 2) * VECTORS * DP);
-                if (more) advance(odd, t + 1, second);
-                float kept[C];
-#pragma unroll
-                for (int c = 0; c < C; ++c)
-                    kept[c] = (second_token ? second[c] : first[c]) + __shfl_xor_sync(0xffffffffu, second_token ? first[c] : second[c], 4);
-                float sum = (second_column ? kept[1] : kept[0]) + __shfl_xor_sync(0xffffffffu, second_column ? kept[0] : kept[1], 2);
-                sum += __shfl_xor_sync(0xffffffffu, sum, 1);
-                const int mine = t + (second_token ? 1 : 0);
-                if ((part & 1) == 0 && mine < count)
-                    results[(buffer * SC + mine) * columns + my_column] = fmaf(scalars_s[SCALARS * mine], v_s[mine * columns + my_column], sum);
-            }
-        } else
 #pragma unroll 1
         for (int t = 0; t < count; t += 2) {
             if (t + 1 < count) odd.template load<L>(rows_s + (t + 1) * VECTORS * DP);
@@ -935,8 +899,8 @@ static int launch_delta_scan(const DeltaScanArgs& a, int entries, cudaStream_t s
 
 template <int RULE>
 static int dispatch_delta_scan(const DeltaScanArgs& a, int entries, cudaStream_t stream) {
-    if (a.dim <= 32) return launch_delta_scan<RULE, 8, 4, 2, 16>(a, entries, stream);
-    if (a.dim <= 64) return launch_delta_scan<RULE, 8, 8, 2, 16>(a, entries, stream);
+    if (a.dim <= 32) return launch_delta_scan<RULE, 8, 4, 1, 16>(a, entries, stream);
+    if (a.dim <= 64) return launch_delta_scan<RULE, 8, 8, 1, 16>(a, entries, stream);
     if (a.dim <= 128) return launch_delta_scan<RULE, 8, 16, 2, 16>(a, entries, stream);
     if (a.dim <= 256) return launch_delta_scan<RULE, 16, 16, 2, 8>(a, entries, stream);
     if (a.dim > MAX_DIM) return ME_ERR_UNSUPPORTED;
@@ -958,15 +922,15 @@ ME_EXPORT int me_delta_scan(const float* qk, const float* gv, const float* scala
     return dispatch_delta_scan<RULE_DELTA>(a, entries, stream);
 }
 
-// The other rules, on what me_state_prepare made.
+// The other rules, on what me_state_prepare made.  `max_count` > 0: entries with more tokens are left to me_state_chunks.
 ME_EXPORT int me_state_walk(const float* rows, const float* scalars, const int* cu_tokens, const int* state_slots, const int* fresh,
                             float* state, long long slot_floats, float* out, int rule, int entries, int heads, int dim, int vdim,
-                            cudaStream_t stream) {
+                            int max_count, cudaStream_t stream) {
     if (entries <= 0) return 0;
     if (dim < 1 || vdim < 1 || heads < 1 || (rule != RULE_REMOVAL && rule != RULE_BONUS)) return ME_ERR_ARGUMENT;
     if (slot_floats < static_cast<long long>(heads) * dim * vdim) return ME_ERR_ARGUMENT;
     const auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
     const int vector = dim % 4 == 0 && vdim % 4 == 0 && slot_floats % 4 == 0 && aligned(rows) && aligned(state);
-    DeltaScanArgs a{nullptr, rows, scalars, cu_tokens, state_slots, fresh, state, (size_t)slot_floats, out, heads, heads, dim, vdim, vector};
+    DeltaScanArgs a{nullptr, rows, scalars, cu_tokens, state_slots, fresh, state, (size_t)slot_floats, out, heads, heads, dim, vdim, vector, max_count};
     return rule == RULE_REMOVAL ? dispatch_delta_scan<RULE_REMOVAL>(a, entries, stream) : dispatch_delta_scan<RULE_BONUS>(a, entries, stream);
 }

@@ -1246,6 +1246,23 @@ def state_rule_floats(rule: str, dim: int, vdim: int) -> tuple[int, int]:
     return vectors * dim + vdim, numbers
 
 
+STATE_CHUNK = 16  # tokens of a chunk of the chunked recurrences
+
+
+def state_chunks_support(dim: int, vdim: int) -> bool:
+    """Whether the chunked kernels take these head sizes."""
+    fn = load_library("state_chunks").me_state_chunks_supports
+    fn.argtypes, fn.restype = [c_int, c_int], c_int
+    return bool(fn(int(dim), int(vdim)))
+
+
+def state_record_floats(rule: str, dim: int) -> int:
+    """Floats of a chunk's record per head."""
+    fn = load_library("state_chunks").me_state_chunks_record_floats
+    fn.argtypes, fn.restype = [c_int, c_int], c_int
+    return int(fn(STATE_RULES[rule], int(dim)))
+
+
 def state_prepare(
     *, rule: str, q: tuple, k: tuple, v: tuple, logits: tuple, rate: tuple | None, decay_bias: torch.Tensor, channel: torch.Tensor,
     rows: torch.Tensor, scalars: torch.Tensor, decay_scale: float, unit_eps: float, heads: int, dim: int, vdim: int,
@@ -1281,18 +1298,31 @@ def state_prepare(
 
 def state_walk(
     *, rule: str, rows: torch.Tensor, scalars: torch.Tensor, ctx, state: torch.Tensor, out: torch.Tensor, heads: int, dim: int, vdim: int,
+    chunk_min: int = 0, records: torch.Tensor | None = None,
 ) -> None:  # fmt: skip
     """The recurrence of ``rule`` over the batch's tokens, entry by entry, from and into each request's state slot (``state
     [slots + 1, floats]``, a slot starts with ``[heads, vdim, dim]``), on what :func:`state_prepare` made; ``out`` is float32
-    ``[T, heads, vdim]``."""
+    ``[T, heads, vdim]``.  ``chunk_min`` > 0: entries of at least that many tokens run in chunks of ``STATE_CHUNK`` tokens
+    (:func:`state_chunks_support` says for which sizes), with ``records [chunks, floats]`` as scratch for all of their chunks
+    (:func:`state_record_floats` floats per head); the other entries walk token by token."""
     for name, t in (("rows", rows), ("scalars", scalars), ("state", state), ("out", out)):
         _need(t, torch.float32, name)
     if state.dim() != 2 or state.shape[1] < heads * dim * vdim:
         raise KernelError("state_walk: the state does not hold the matrix states")
-    fn = _fn("delta_rule", "me_state_walk", [c_void_p] * 6 + [c_longlong, c_void_p] + [c_int] * 5 + [c_void_p])
+    if chunk_min:
+        _need(records, torch.float32, "records")
+        if not state_chunks_support(dim, vdim) or records.dim() != 2 or records.shape[1] != heads * state_record_floats(rule, dim):
+            raise KernelError("state_walk: the chunks' records or the head sizes do not fit")
+        fn = _fn("state_chunks", "me_state_chunks", [c_void_p] * 6 + [c_longlong, c_void_p, c_void_p] + [c_int] * 7 + [c_void_p])
+        code = fn(
+            _ptr(rows), _ptr(scalars), _ptr(ctx.cu_tokens), _ptr(ctx.state_slots), _ptr(ctx.fresh), _ptr(state), state.shape[1],
+            _ptr(out), _ptr(records), STATE_RULES[rule], ctx.num_entries, heads, dim, vdim, int(chunk_min), records.shape[0], _stream(),
+        )  # fmt: skip
+        _check(code, "state_chunks")
+    fn = _fn("delta_rule", "me_state_walk", [c_void_p] * 6 + [c_longlong, c_void_p] + [c_int] * 6 + [c_void_p])
     code = fn(
         _ptr(rows), _ptr(scalars), _ptr(ctx.cu_tokens), _ptr(ctx.state_slots), _ptr(ctx.fresh), _ptr(state), state.shape[1],
-        _ptr(out), STATE_RULES[rule], ctx.num_entries, heads, dim, vdim, _stream(),
+        _ptr(out), STATE_RULES[rule], ctx.num_entries, heads, dim, vdim, max(int(chunk_min) - 1, 0), _stream(),
     )  # fmt: skip
     _check(code, "state_walk")
 

@@ -244,6 +244,11 @@ def low_rank_second(weight: torch.Tensor) -> tuple[Linear, int]:
     return Linear(torch.cat([weight] * halves, dim=1).contiguous()), halves
 
 
+# An entry of at least this many tokens runs in chunks; decoded tokens and short portions walk and keep the bits of a
+# token-by-token run.
+CHUNKED_MIN_TOKENS = 33
+
+
 def walk_states(rule: str, ctx: StepContext, state: torch.Tensor, heads: int, dim: int, vdim: int, **inputs) -> torch.Tensor:
     """Prepare and walk a recurrence of :data:`ops.STATE_RULES`; returns the heads' outputs ``[T, heads * vdim]`` float32."""
     tokens = ctx.num_tokens
@@ -253,5 +258,10 @@ def walk_states(rule: str, ctx: StepContext, state: torch.Tensor, heads: int, di
     sizes = dict(heads=heads, dim=dim, vdim=vdim)
     ops.state_prepare(rule=rule, rows=rows, scalars=scalars, **{"rate": None, "unit_eps": 0.0, "decay_scale": 1.0, **inputs}, **sizes)
     raw = ctx.buffer(f"{rule}.raw", (tokens, heads * vdim), torch.float32)
-    ops.state_walk(rule=rule, rows=rows, scalars=scalars, ctx=ctx, state=state, out=raw, **sizes)
+    chunk_min, records = 0, None
+    if ctx.max_query_len >= CHUNKED_MIN_TOKENS and ops.state_chunks_support(dim, vdim):  # a step's longest entry is known on the host
+        chunk_min = CHUNKED_MIN_TOKENS
+        chunks = tokens // ops.STATE_CHUNK + ctx.num_entries
+        records = ctx.workspace.growing(f"{rule}.records", (chunks, heads * ops.state_record_floats(rule, dim)), torch.float32)
+    ops.state_walk(rule=rule, rows=rows, scalars=scalars, ctx=ctx, state=state, out=raw, chunk_min=chunk_min, records=records, **sizes)
     return raw

@@ -247,8 +247,9 @@ def test_the_test_weights_show_every_mechanism(folders, what):
 
 @pytest.mark.parametrize("block_size", [4, 16, 32])
 def test_float32_hardly_depends_on_the_cut_or_the_batch(folders, block_size):
-    """In float32 every kernel's sums for a token depend on that token's position alone: portions, single tokens, mixed batches
-    and other page sizes give the whole prompt's logits up to rounding."""
+    """In float32 every kernel's sums for a token depend on that token's position alone, except that the matrix states run long
+    portions in chunks, whose sums are ordered by a token's place in its portion: portions, single tokens, mixed batches and
+    other page sizes give the whole prompt's logits up to rounding."""
     requests = {name: toks for name, toks in list(requests_for("S").items())[:5]}
     whole = replay(folders["S"], "float32", schedules.whole(requests), block_size)
     for maker in (schedules.changing_portions, schedules.mixed, lambda r: schedules.tail_one_by_one(r, 40)):

@@ -318,7 +318,7 @@ class StateRun:
         self.__dict__.update(rule=rule, heads=heads, dim=dim, vdim=vdim, inputs=inputs, decay_scale=decay_scale)
         self.state = torch.full((5, heads * dim * vdim + 4), 7.0, dtype=torch.float32, device="cuda")
 
-    def step(self, spans, slots):
+    def step(self, spans, slots, chunk_min=0):
         """``spans``: (first, count) per entry, all of the same sequence."""
         from mini_engine_b200.csrc import ops
 
@@ -339,7 +339,10 @@ class StateRun:
         )  # fmt: skip
         out = torch.empty(count, self.heads * self.vdim, device="cuda")
         ctx = Context([n for _, n in spans], [a for a, _ in spans], slots)
-        ops.state_walk(rule=self.rule, rows=held[0], scalars=held[1], ctx=ctx, state=self.state, out=out, **sizes)
+        records = None
+        if chunk_min:
+            records = torch.full((count // ops.STATE_CHUNK + len(spans), self.heads * ops.state_record_floats(self.rule, self.dim)), float("nan"), device="cuda")
+        ops.state_walk(rule=self.rule, rows=held[0], scalars=held[1], ctx=ctx, state=self.state, out=out, chunk_min=chunk_min, records=records, **sizes)
         return out.cpu()
 
 
@@ -365,6 +368,37 @@ def test_states_whole_in_portions_token_by_token_and_side_by_side(rule, heads, d
     both = run.step([(0, 2), (33, 37)], [3, 2])
     assert torch.equal(both[:2], whole[:2]) and torch.equal(both[2:], whole[33:])
     assert torch.equal(run.state[2], run.state[0])
+
+
+@pytest.mark.parametrize("rule", ["removal", "bonus"])
+@pytest.mark.parametrize("heads,dim,vdim", [(2, 16, 8), (3, 24, 40), (1, 4, 4), (2, 64, 64), (2, 128, 128), (1, 100, 36), (3, 48, 48), (1, 32, 68)])
+@pytest.mark.parametrize("decays", ["mixed", "strong", "none"])
+def test_states_in_chunks(rule, heads, dim, vdim, decays):
+    """Long entries in chunks of 16 tokens: whole, from a carried state, whole chunks and a rest of one token and of fifteen,
+    beside entries that walk and beside each other, with decays that leave nothing of a channel within a token, and with none."""
+    tokens = 150
+    q, k, v, z, rate, decay_bias, channel = state_inputs(rule, heads, dim, vdim, tokens)
+    z, scale = {"mixed": (2.0 * z, 0.6), "strong": (z + (3.0 if rule == "bonus" else 9.0), 40.0), "none": (z - 60.0, 0.6)}[decays]
+    if rule == "removal":
+        k = k / math.sqrt(dim)
+    inputs = (q, k, v, z, rate, decay_bias, channel)
+    run = StateRun(rule, heads, dim, vdim, inputs, decay_scale=scale)
+    want, state = plain_states(rule, heads, dim, vdim, *inputs, scale)
+    want = want.reshape(tokens, -1)
+    states_of = lambda slot: run.state[slot, : heads * dim * vdim].view(heads, vdim, dim)  # noqa: E731
+    for cuts in ([0, tokens], [0, 49, 97, tokens], [0, 5, 38, 101, 103, tokens], [0, 33, 112, tokens]):
+        run.state.fill_(7.0)
+        got = torch.cat([run.step([(a, b - a)], [1], chunk_min=33) for a, b in zip(cuts, cuts[1:])])
+        close(got, want, 3e-5)
+        close(states_of(1), state.transpose(1, 2), 3e-5)
+        assert float(run.state[0].min()) == 7.0 and float(run.state[1, heads * dim * vdim :].min()) == 7.0
+    # in one batch: a single token, a long entry, a walking portion, another long entry
+    run.step([(0, 60)], [0], chunk_min=33)
+    run.step([(0, 20)], [2], chunk_min=33)
+    got = run.step([(60, 1), (0, tokens), (20, 32), (0, 35)], [0, 3, 2, 4], chunk_min=33)
+    for rows, first in ((got[:1], 60), (got[1 : 1 + tokens], 0), (got[1 + tokens : 33 + tokens], 20), (got[33 + tokens :], 0)):
+        close(rows, want[first : first + rows.shape[0]], 3e-5)
+    close(states_of(3), state.transpose(1, 2), 3e-5)
 
 
 def test_a_key_is_removed_channel_by_channel_hundreds_of_tokens_later():
