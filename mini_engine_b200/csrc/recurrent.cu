@@ -16,7 +16,8 @@
 // that starts its sequence starts from zeros.
 //
 // Three kernels.  `conv`: a thread per (token, channel), one token per grid column, forms u (the convolution reaches back into the entry's
-// earlier tokens of this step or into the state) and leaves it in scratch.  `gates`: a CTA takes 16 tokens of one
+// earlier tokens of this step or into the state) and leaves it in scratch; in long steps a thread takes four channels of eight
+// tokens, whose inputs slide through its registers.  `gates`: a CTA takes 16 tokens of one
 // block, holds their u in shared memory and forms 64 channels' two gates, reading each weight once for the 16
 // tokens; it leaves a_t and the driven term in scratch.  `scan`: a CTA per
 // (entry, 32 channels) walks the entry's tokens in order, then leaves S and the convolution's history in the
@@ -83,6 +84,50 @@ __global__ void __launch_bounds__(256) rglru_conv_kernel(RecurrentArgs a) {
         u = fmaf(a.taps[static_cast<size_t>(c) * K + (K - 1 - back)], x, u);
     }
     a.conv[static_cast<size_t>(t) * a.channels + c] = u;
+}
+
+// The same bits for a long step whose projection is not split, with rows on 16 bytes and KC taps.
+constexpr int CONV_RUN = 8;            // tokens of a thread
+constexpr int CONV_RUN_TOKENS = 512;   // from this many tokens on
+
+template <int KC>
+__global__ void __launch_bounds__(128) rglru_conv_runs_kernel(RecurrentArgs a) {
+    const int c = (blockIdx.y * 128 + threadIdx.x) * 4, run_begin = blockIdx.x * CONV_RUN;
+    pdl_trigger();
+    pdl_wait();
+    if (c >= a.channels) return;
+    const float4 bias4 = *reinterpret_cast<const float4*>(a.in_bias + a.channels + c);
+    float taps[4][KC];  // [channel][taps], the last one the current token's
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < KC; ++j) taps[i][j] = a.taps[static_cast<size_t>(c + i) * KC + j];
+    const float4 conv_bias4 = *reinterpret_cast<const float4*>(a.conv_bias + c);
+    float4 x[CONV_RUN + KC - 1];  // the run's inputs behind the KC - 1 in front of it (as rows of this step; an entry's start looks elsewhere)
+#pragma unroll
+    for (int i = 0; i < CONV_RUN + KC - 1; ++i) {
+        const int t = run_begin - (KC - 1) + i;
+        x[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (t >= 0 && t < a.tokens) x[i] = *reinterpret_cast<const float4*>(a.proj + static_cast<size_t>(t) * 2 * a.channels + a.channels + c);
+    }
+#pragma unroll
+    for (int i = 0; i < CONV_RUN + KC - 1; ++i) x[i] = make_float4(x[i].x + bias4.x, x[i].y + bias4.y, x[i].z + bias4.z, x[i].w + bias4.w);
+#pragma unroll
+    for (int i = 0; i < CONV_RUN; ++i) {
+        const int t = run_begin + i;
+        if (t >= a.tokens) break;
+        const int entry = a.entry_of_token[t], n = t - a.cu_tokens[entry];
+        const float* history = n < KC - 1 && !a.fresh[entry] ? a.state + (static_cast<size_t>(a.state_slots[entry]) * KC + 1) * a.channels : nullptr;
+        float4 u = conv_bias4;
+#pragma unroll
+        for (int back = 0; back < KC; ++back) {
+            float4 y = x[i + KC - 1 - back];
+            if (n - back < 0) y = history ? *reinterpret_cast<const float4*>(history + static_cast<size_t>(n - back + KC - 1) * a.channels + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            u.x = fmaf(taps[0][KC - 1 - back], y.x, u.x), u.y = fmaf(taps[1][KC - 1 - back], y.y, u.y);
+            u.z = fmaf(taps[2][KC - 1 - back], y.z, u.z), u.w = fmaf(taps[3][KC - 1 - back], y.w, u.w);
+        }
+        *reinterpret_cast<float4*>(a.conv + static_cast<size_t>(t) * a.channels + c) = u;
+    }
 }
 
 __global__ void __launch_bounds__(GATE_THREADS) rglru_gates_kernel(RecurrentArgs a) {
@@ -276,7 +321,17 @@ ME_EXPORT int me_rglru(const float* proj, int splits, long long split_stride, co
     const int chunks = (width + GATE_THREADS - 1) / GATE_THREADS;
     const dim3 gate_grid((tokens + GATE_TOKENS - 1) / GATE_TOKENS, blocks * chunks);
     const dim3 conv_grid(tokens, (channels + 255) / 256);
-    int status = launch_kernel(rglru_conv_kernel, conv_grid, 256, 0, stream, a);
+    const auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+    int status;
+    if (tokens >= CONV_RUN_TOKENS && taps_count >= 2 && taps_count <= 4 && splits == 1 && channels % 4 == 0 && aligned(proj) && aligned(in_bias) &&
+        aligned(conv_bias) && aligned(conv) && aligned(state)) {
+        const dim3 runs_grid((tokens + CONV_RUN - 1) / CONV_RUN, (channels + 511) / 512);
+        status = taps_count == 2   ? launch_kernel(rglru_conv_runs_kernel<2>, runs_grid, 128, 0, stream, a)
+                 : taps_count == 3 ? launch_kernel(rglru_conv_runs_kernel<3>, runs_grid, 128, 0, stream, a)
+                                   : launch_kernel(rglru_conv_runs_kernel<4>, runs_grid, 128, 0, stream, a);
+    } else {
+        status = launch_kernel(rglru_conv_kernel, conv_grid, 256, 0, stream, a);
+    }
     if (status) return status;
     status = launch_kernel(rglru_gates_kernel, gate_grid, GATE_THREADS, smem, stream, a);
     if (status) return status;

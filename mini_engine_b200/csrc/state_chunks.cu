@@ -32,6 +32,7 @@ enum : int { RULE_REMOVAL = 1, RULE_BONUS = 2 };
 constexpr int CHUNK = 16;
 constexpr int COLUMNS = 32;  // value columns of a walking block
 constexpr int THREADS = 128;
+constexpr int STAGES = 3;  // records that a walking block holds: two are on their way
 
 template <int RULE>
 struct Rule;
@@ -55,8 +56,8 @@ struct ChunkArgs {
     float* state;  // [slots + 1][slot_floats], a slot starts with [heads][vdim][dim]
     size_t slot_floats;
     float* out;      // [tokens][heads][vdim]
-    float* records;  // [chunks][heads][record_floats]
-    int entries, heads, dim, vdim, min_count;
+    float* records;  // [heads][max_chunks][record floats]: a walking block reads its records one after the other
+    int entries, heads, dim, vdim, min_count, max_chunks;
 };
 
 // The entry that chunk number `chunk` belongs to (entries of at least min_count tokens, cut in order).
@@ -155,7 +156,7 @@ __global__ void __launch_bounds__(THREADS) chunk_record_kernel(ChunkArgs a) {
         }
     }
     __syncthreads();
-    float* record = a.records + (static_cast<size_t>(blockIdx.x) * a.heads + head) * Record<RULE, DIM>::FLOATS;
+    float* record = a.records + (static_cast<size_t>(head) * a.max_chunks + blockIdx.x) * Record<RULE, DIM>::FLOATS;
     float* writing = record + (DIM + CHUNK) * ROWS;
     // One column per thread: a key channel of A and R, or a token of AK and RK.
     for (int column = threadIdx.x; column < DIM + CHUNK; column += THREADS) {
@@ -212,21 +213,25 @@ __device__ __forceinline__ void copy_async_16(float* shared_dst, const float* gl
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(global_src) : "memory");
 }
 __device__ __forceinline__ void copy_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-__device__ __forceinline__ void copy_async_wait() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+__device__ __forceinline__ void copy_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory"); }
 
-// One block per (entry, head, 32 value columns).  A thread owns a tile of 4 channels x 4 columns of the state (two of them at
-// 128 channels) in registers, and shares it with the block through shared memory.
+// One block of four warps per (entry, head, 32 value columns).  A thread owns a tile of 4 channels x 4 columns of the state (two
+// of them at 128 channels) in registers, and shares it with the block through shared memory.  Shared memory's bandwidth is what
+// the two products of a chunk are bound by, so that a thread takes tiles as large as its registers hold: in the reading product
+// every warp adds up a quarter of the terms for all of the outputs, ROWS / 4 rows x 4 columns to a lane, and the quarters meet in
+// shared memory.
 template <int RULE, int DIM>
 __global__ void __launch_bounds__(THREADS) chunk_walk_kernel(ChunkArgs a) {
     constexpr int VECTORS = Rule<RULE>::VECTORS, ROWS = Rule<RULE>::ROWS, RECORD = Record<RULE, DIM>::FLOATS;
     constexpr bool REMOVES = RULE == RULE_REMOVAL;
     constexpr int STAGE = RECORD + CHUNK * COLUMNS;
     constexpr int TILES = DIM > 64 ? DIM / 64 : 1;
-    constexpr int TALL = ROWS / 8;  // rows of a thread's part of the reading product
+    constexpr int TALL = ROWS / 4;  // rows of a lane's part of the reading product
     extern __shared__ __align__(16) float chunk_smem[];
-    float* stages = chunk_smem;               // [2]: record, values [CHUNK][COLUMNS]
-    float* held = chunk_smem + 2 * STAGE;     // the state [DIM][COLUMNS]
-    float* minus_y = held + DIM * COLUMNS;    // [CHUNK][COLUMNS]
+    float* stages = chunk_smem;                  // [STAGES]: record, values [CHUNK][COLUMNS]
+    float* held = chunk_smem + STAGES * STAGE;   // the state [DIM][COLUMNS]
+    float* minus_y = held + DIM * COLUMNS;       // [CHUNK][COLUMNS]
+    float* partial = minus_y + CHUNK * COLUMNS;  // [4 warps][ROWS][COLUMNS]
     const int entry = blockIdx.x, head = blockIdx.y, first_column = blockIdx.z * COLUMNS;
     pdl_trigger();
     pdl_wait();
@@ -240,10 +245,10 @@ __global__ void __launch_bounds__(THREADS) chunk_walk_kernel(ChunkArgs a) {
     const int chunks = (count + CHUNK - 1) / CHUNK;
     const int row_floats = VECTORS * a.dim + a.vdim;
     const float* values = a.rows + (static_cast<size_t>(begin) * a.heads + head) * row_floats + VECTORS * a.dim + first_column;
-    const size_t row_step = static_cast<size_t>(a.heads) * row_floats, record_step = static_cast<size_t>(a.heads) * RECORD;
-    const float* records = a.records + (static_cast<size_t>(first_chunk) * a.heads + head) * RECORD;
+    const size_t row_step = static_cast<size_t>(a.heads) * row_floats;
+    const float* records = a.records + (static_cast<size_t>(head) * a.max_chunks + first_chunk) * RECORD;
     auto fetch = [&](int chunk, float* stage) {
-        const float* record = records + chunk * record_step;
+        const float* record = records + static_cast<size_t>(chunk) * RECORD;
         for (int i = threadIdx.x; i < RECORD / 4; i += THREADS) copy_async_16(stage + 4 * i, record + 4 * i);
         for (int i = threadIdx.x; i < CHUNK * COLUMNS / 4; i += THREADS) {
             const int t = chunk * CHUNK + i / (COLUMNS / 4), column = i % (COLUMNS / 4) * 4;
@@ -251,11 +256,14 @@ __global__ void __launch_bounds__(THREADS) chunk_walk_kernel(ChunkArgs a) {
             if (t < count && first_column + column < a.vdim) copy_async_16(dst, values + t * row_step + column);
             else *reinterpret_cast<float4*>(dst) = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         }
-        copy_async_commit();
     };
-    fetch(0, stages);
+#pragma unroll
+    for (int i = 0; i < STAGES - 1; ++i) {  // a group per chunk, empty behind the last one
+        if (i < chunks) fetch(i, stages + i * STAGE);
+        copy_async_commit();
+    }
 
-    // The state's tile: channels [4 quad, +4), columns [4 strip, +4).
+    // The state's tile: channels [4 (thread / 8), +4), columns [4 strip, +4).
     const int strip = threadIdx.x % 8;
     float4 s[TILES][4];  // [channel] of four columns
     float* state = a.state + static_cast<size_t>(a.state_slots[entry]) * a.slot_floats + (static_cast<size_t>(head) * a.vdim + first_column + 4 * strip) * a.dim;
@@ -275,73 +283,86 @@ __global__ void __launch_bounds__(THREADS) chunk_walk_kernel(ChunkArgs a) {
         }
     }
 
-    const int group = threadIdx.x / 16, pair = threadIdx.x % 16;  // rows [TALL group, +TALL), columns [2 pair, +2) of the reading product
+    const int warp = threadIdx.x / 32, group = threadIdx.x % 32 / 8;  // rows [TALL group, +TALL) of the reading product, columns as above
     for (int chunk = 0; chunk < chunks; ++chunk) {
-        float* stage = stages + (chunk & 1) * STAGE;
+        float* stage = stages + chunk % STAGES * STAGE;
         copy_async_wait();
-        __syncthreads();  // the record has landed, the state is in shared memory and nobody reads the other stage any more
-        if (chunk + 1 < chunks) fetch(chunk + 1, stages + ((chunk + 1) & 1) * STAGE);
+        __syncthreads();  // the record has landed, the state is in shared memory and nobody reads the oldest stage any more
+        if (chunk + STAGES - 1 < chunks) fetch(chunk + STAGES - 1, stages + (chunk + STAGES - 1) % STAGES * STAGE);
+        copy_async_commit();
         const float* v = stage + RECORD;
-        float2 z[TALL];
+        float2 low[TALL], high[TALL];
 #pragma unroll
-        for (int i = 0; i < TALL; ++i) z[i] = make_float2(0.0f, 0.0f);
-        auto add_row = [&](const float* reading, const float* operand) {
-            const float2 x = *reinterpret_cast<const float2*>(operand + 2 * pair);
-            if constexpr (TALL == 4) {
-                const float4 w = *reinterpret_cast<const float4*>(reading + 4 * group);
-                z[0] = __ffma2_rn(make_float2(w.x, w.x), x, z[0]), z[1] = __ffma2_rn(make_float2(w.y, w.y), x, z[1]);
-                z[2] = __ffma2_rn(make_float2(w.z, w.z), x, z[2]), z[3] = __ffma2_rn(make_float2(w.w, w.w), x, z[3]);
-            } else {
-                const float2 w = *reinterpret_cast<const float2*>(reading + 2 * group);
-                z[0] = __ffma2_rn(make_float2(w.x, w.x), x, z[0]), z[1] = __ffma2_rn(make_float2(w.y, w.y), x, z[1]);
-            }
-        };
-#pragma unroll 8
-        for (int d = 0; d < DIM; ++d) add_row(stage + d * ROWS, held + d * COLUMNS);
-#pragma unroll 8
-        for (int t = 0; t < CHUNK; ++t) add_row(stage + (DIM + t) * ROWS, v + t * COLUMNS);
+        for (int i = 0; i < TALL; ++i) low[i] = high[i] = make_float2(0.0f, 0.0f);
+        // A warp's quarter of the terms: channels of the state, then tokens' values.
+        constexpr int TERMS = (DIM + CHUNK) / 4;
+#pragma unroll 4
+        for (int n = 0; n < TERMS; ++n) {
+            const int term = warp * TERMS + n;
+            const float* reading = stage + term * ROWS + TALL * group;
+            const float4 x = *reinterpret_cast<const float4*>((term < DIM ? held + term * COLUMNS : v + (term - DIM) * COLUMNS) + 4 * strip);
+            const float2 left = make_float2(x.x, x.y), right = make_float2(x.z, x.w);
 #pragma unroll
-        for (int i = 0; i < TALL; ++i) {
-            const int row = TALL * group + i, t = row - (ROWS - CHUNK);
-            if (REMOVES && row < CHUNK) {
-                *reinterpret_cast<float2*>(minus_y + row * COLUMNS + 2 * pair) = make_float2(-z[i].x, -z[i].y);
-            } else if (chunk * CHUNK + t < count && first_column + 2 * pair < a.vdim) {
-                float* out = a.out + (static_cast<size_t>(begin + chunk * CHUNK + t) * a.heads + head) * a.vdim + first_column + 2 * pair;
-                *reinterpret_cast<float2*>(out) = z[i];
+            for (int q = 0; q < TALL; q += 4) {
+                const float4 w = *reinterpret_cast<const float4*>(reading + q);
+                low[q] = __ffma2_rn(make_float2(w.x, w.x), left, low[q]), high[q] = __ffma2_rn(make_float2(w.x, w.x), right, high[q]);
+                low[q + 1] = __ffma2_rn(make_float2(w.y, w.y), left, low[q + 1]), high[q + 1] = __ffma2_rn(make_float2(w.y, w.y), right, high[q + 1]);
+                low[q + 2] = __ffma2_rn(make_float2(w.z, w.z), left, low[q + 2]), high[q + 2] = __ffma2_rn(make_float2(w.z, w.z), right, high[q + 2]);
+                low[q + 3] = __ffma2_rn(make_float2(w.w, w.w), left, low[q + 3]), high[q + 3] = __ffma2_rn(make_float2(w.w, w.w), right, high[q + 3]);
             }
         }
-        __syncthreads();  // every thread has read the state, and the reads y are there
+#pragma unroll
+        for (int i = 0; i < TALL; ++i)
+            *reinterpret_cast<float4*>(partial + (warp * ROWS + TALL * group + i) * COLUMNS + 4 * strip) = make_float4(low[i].x, low[i].y, high[i].x, high[i].y);
+        __syncthreads();  // the quarters are there, and nobody reads the state any more
+#pragma unroll
+        for (int n = 0; n < ROWS / 16; ++n) {
+            const int row = n * 16 + threadIdx.x / 8, t = row - (ROWS - CHUNK);
+            float4 z = *reinterpret_cast<const float4*>(partial + row * COLUMNS + 4 * strip);
+#pragma unroll
+            for (int part = 1; part < 4; ++part) {
+                const float4 x = *reinterpret_cast<const float4*>(partial + (part * ROWS + row) * COLUMNS + 4 * strip);
+                z.x += x.x, z.y += x.y, z.z += x.z, z.w += x.w;
+            }
+            if (REMOVES && n == 0) {
+                *reinterpret_cast<float4*>(minus_y + row * COLUMNS + 4 * strip) = make_float4(-z.x, -z.y, -z.z, -z.w);
+            } else if (chunk * CHUNK + t < count && first_column + 4 * strip < a.vdim) {
+                float* out = a.out + (static_cast<size_t>(begin + chunk * CHUNK + t) * a.heads + head) * a.vdim + first_column + 4 * strip;
+                *reinterpret_cast<float4*>(out) = z;
+            }
+        }
+        if (REMOVES) __syncthreads();  // the reads y are there
         const float* writing = stage + (DIM + CHUNK) * ROWS;
 #pragma unroll
         for (int tile = 0; tile < TILES; ++tile) {
             const int d = 4 * (threadIdx.x / 8 + 16 * tile);
             if (d >= DIM) continue;
             const float4 g = *reinterpret_cast<const float4*>(writing + ROWS * DIM + d);
-            float2 low[4], high[4];
+            float2 first[4], second[4];
             const float decay[4] = {g.x, g.y, g.z, g.w};
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
-                low[i] = make_float2(s[tile][i].x * decay[i], s[tile][i].y * decay[i]);
-                high[i] = make_float2(s[tile][i].z * decay[i], s[tile][i].w * decay[i]);
+                first[i] = make_float2(s[tile][i].x * decay[i], s[tile][i].y * decay[i]);
+                second[i] = make_float2(s[tile][i].z * decay[i], s[tile][i].w * decay[i]);
             }
             auto add_outer = [&](const float* written, const float* operand) {
                 const float4 w = *reinterpret_cast<const float4*>(written + d), x = *reinterpret_cast<const float4*>(operand + 4 * strip);
                 const float weights[4] = {w.x, w.y, w.z, w.w};
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
-                    low[i] = __ffma2_rn(make_float2(weights[i], weights[i]), make_float2(x.x, x.y), low[i]);
-                    high[i] = __ffma2_rn(make_float2(weights[i], weights[i]), make_float2(x.z, x.w), high[i]);
+                    first[i] = __ffma2_rn(make_float2(weights[i], weights[i]), make_float2(x.x, x.y), first[i]);
+                    second[i] = __ffma2_rn(make_float2(weights[i], weights[i]), make_float2(x.z, x.w), second[i]);
                 }
             };
-#pragma unroll 4
+#pragma unroll 8
             for (int t = 0; t < CHUNK; ++t) add_outer(writing + t * DIM, v + t * COLUMNS);
             if constexpr (REMOVES) {
-#pragma unroll 4
+#pragma unroll 8
                 for (int t = 0; t < CHUNK; ++t) add_outer(writing + (CHUNK + t) * DIM, minus_y + t * COLUMNS);
             }
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
-                s[tile][i] = make_float4(low[i].x, low[i].y, high[i].x, high[i].y);
+                s[tile][i] = make_float4(first[i].x, first[i].y, second[i].x, second[i].y);
                 *reinterpret_cast<float4*>(held + (d + i) * COLUMNS + 4 * strip) = s[tile][i];
             }
         }
@@ -374,7 +395,7 @@ template <int RULE, int DIM>
 static int launch_chunks(const ChunkArgs& a, int max_chunks, cudaStream_t stream) {
     static SharedMemoryOptIn record_opt_in, walk_opt_in;
     constexpr int RECORD_SMEM = (Rule<RULE>::VECTORS * CHUNK * DIM + 4 * CHUNK * CHUNK) * sizeof(float);
-    constexpr int WALK_SMEM = (2 * (Record<RULE, DIM>::FLOATS + CHUNK * COLUMNS) + DIM * COLUMNS + CHUNK * COLUMNS) * sizeof(float);
+    constexpr int WALK_SMEM = (STAGES * (Record<RULE, DIM>::FLOATS + CHUNK * COLUMNS) + DIM * COLUMNS + (CHUNK + 4 * Rule<RULE>::ROWS) * COLUMNS) * sizeof(float);
     if (RECORD_SMEM > 48 * 1024)
         if (const int e = record_opt_in(chunk_record_kernel<RULE, DIM>, RECORD_SMEM)) return e;
     if (WALK_SMEM > 48 * 1024)
@@ -401,6 +422,6 @@ ME_EXPORT int me_state_chunks(const float* rows, const float* scalars, const int
     if (!me_state_chunks_supports(dim, vdim) || slot_floats % 4 || !aligned(rows) || !aligned(state) || !aligned(out) || !aligned(records))
         return ME_ERR_UNSUPPORTED;
     if (slot_floats < static_cast<long long>(heads) * dim * vdim) return ME_ERR_ARGUMENT;
-    ChunkArgs a{rows, scalars, cu_tokens, state_slots, fresh, state, (size_t)slot_floats, out, records, entries, heads, dim, vdim, min_count};
+    ChunkArgs a{rows, scalars, cu_tokens, state_slots, fresh, state, (size_t)slot_floats, out, records, entries, heads, dim, vdim, min_count, max_chunks};
     return rule == RULE_REMOVAL ? dispatch_chunks<RULE_REMOVAL>(a, max_chunks, stream) : dispatch_chunks<RULE_BONUS>(a, max_chunks, stream);
 }
