@@ -31,7 +31,9 @@ enum : int { RULE_REMOVAL = 1, RULE_BONUS = 2 };
 
 constexpr int CHUNK = 16;
 constexpr int COLUMNS = 32;  // value columns of a walking block
-constexpr int THREADS = 128;
+constexpr int THREADS = 128;       // of a recording block
+constexpr int WALK_THREADS = 256;  // of a walking block
+constexpr int WALK_WARPS = WALK_THREADS / 32;
 constexpr int STAGES = 3;  // records that a walking block holds: two are on their way
 
 template <int RULE>
@@ -215,13 +217,13 @@ __device__ __forceinline__ void copy_async_16(float* shared_dst, const float* gl
 __device__ __forceinline__ void copy_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void copy_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory"); }
 
-// One block of four warps per (entry, head, 32 value columns).  A thread owns a tile of 4 channels x 4 columns of the state (two
-// of them at 128 channels) in registers, and shares it with the block through shared memory.  Shared memory's bandwidth is what
-// the two products of a chunk are bound by, so that a thread takes tiles as large as its registers hold: in the reading product
-// every warp adds up a quarter of the terms for all of the outputs, ROWS / 4 rows x 4 columns to a lane, and the quarters meet in
-// shared memory.
+// One block of eight warps per (entry, head, 32 value columns).  A thread of the first four warps owns a tile of 4 channels x 4
+// columns of the state (two of them at 128 channels) in registers, and shares it with the block through shared memory.  What
+// the two products of a chunk read from shared memory is what they cost, so that a thread takes tiles as large as its registers
+// hold and the warps share the terms and not the outputs: in the reading product every warp adds up an eighth of the terms for all
+// outputs, ROWS / 4 rows x 4 columns to a lane; of what is written the other four warps add up half.
 template <int RULE, int DIM>
-__global__ void __launch_bounds__(THREADS) chunk_walk_kernel(ChunkArgs a) {
+__global__ void __launch_bounds__(WALK_THREADS) chunk_walk_kernel(ChunkArgs a) {
     constexpr int VECTORS = Rule<RULE>::VECTORS, ROWS = Rule<RULE>::ROWS, RECORD = Record<RULE, DIM>::FLOATS;
     constexpr bool REMOVES = RULE == RULE_REMOVAL;
     constexpr int STAGE = RECORD + CHUNK * COLUMNS;
@@ -231,7 +233,8 @@ __global__ void __launch_bounds__(THREADS) chunk_walk_kernel(ChunkArgs a) {
     float* stages = chunk_smem;                  // [STAGES]: record, values [CHUNK][COLUMNS]
     float* held = chunk_smem + STAGES * STAGE;   // the state [DIM][COLUMNS]
     float* minus_y = held + DIM * COLUMNS;       // [CHUNK][COLUMNS]
-    float* partial = minus_y + CHUNK * COLUMNS;  // [4 warps][ROWS][COLUMNS]
+    float* partial = minus_y + CHUNK * COLUMNS;  // [warps][ROWS][COLUMNS]
+    float* added = partial + WALK_WARPS * ROWS * COLUMNS;  // [DIM][COLUMNS]: the other warps' half of what is written
     const int entry = blockIdx.x, head = blockIdx.y, first_column = blockIdx.z * COLUMNS;
     pdl_trigger();
     pdl_wait();
@@ -249,8 +252,8 @@ __global__ void __launch_bounds__(THREADS) chunk_walk_kernel(ChunkArgs a) {
     const float* records = a.records + (static_cast<size_t>(head) * a.max_chunks + first_chunk) * RECORD;
     auto fetch = [&](int chunk, float* stage) {
         const float* record = records + static_cast<size_t>(chunk) * RECORD;
-        for (int i = threadIdx.x; i < RECORD / 4; i += THREADS) copy_async_16(stage + 4 * i, record + 4 * i);
-        for (int i = threadIdx.x; i < CHUNK * COLUMNS / 4; i += THREADS) {
+        for (int i = threadIdx.x; i < RECORD / 4; i += WALK_THREADS) copy_async_16(stage + 4 * i, record + 4 * i);
+        for (int i = threadIdx.x; i < CHUNK * COLUMNS / 4; i += WALK_THREADS) {
             const int t = chunk * CHUNK + i / (COLUMNS / 4), column = i % (COLUMNS / 4) * 4;
             float* dst = stage + RECORD + 4 * i;
             if (t < count && first_column + column < a.vdim) copy_async_16(dst, values + t * row_step + column);
@@ -263,21 +266,22 @@ __global__ void __launch_bounds__(THREADS) chunk_walk_kernel(ChunkArgs a) {
         copy_async_commit();
     }
 
-    // The state's tile: channels [4 (thread / 8), +4), columns [4 strip, +4).
-    const int strip = threadIdx.x % 8;
+    // The state's tile: channels [4 quad, +4), columns [4 strip, +4).
+    const int strip = threadIdx.x % 8, quad = threadIdx.x % 128 / 8;
+    const bool owner = threadIdx.x < 128;
     float4 s[TILES][4];  // [channel] of four columns
     float* state = a.state + static_cast<size_t>(a.state_slots[entry]) * a.slot_floats + (static_cast<size_t>(head) * a.vdim + first_column + 4 * strip) * a.dim;
     auto columns_of = [](float4& row, int c) -> float& { return c == 0 ? row.x : c == 1 ? row.y : c == 2 ? row.z : row.w; };
 #pragma unroll
     for (int tile = 0; tile < TILES; ++tile) {
-        const int d = 4 * (threadIdx.x / 8 + 16 * tile);
+        const int d = 4 * (quad + 16 * tile);
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
             float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
             if (d < a.dim && first_column + 4 * strip + c < a.vdim && a.fresh[entry] == 0) x = *reinterpret_cast<const float4*>(state + static_cast<size_t>(c) * a.dim + d);
             columns_of(s[tile][0], c) = x.x, columns_of(s[tile][1], c) = x.y, columns_of(s[tile][2], c) = x.z, columns_of(s[tile][3], c) = x.w;
         }
-        if (d < DIM) {
+        if (owner && d < DIM) {
 #pragma unroll
             for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(held + (d + i) * COLUMNS + 4 * strip) = s[tile][i];
         }
@@ -294,9 +298,9 @@ __global__ void __launch_bounds__(THREADS) chunk_walk_kernel(ChunkArgs a) {
         float2 low[TALL], high[TALL];
 #pragma unroll
         for (int i = 0; i < TALL; ++i) low[i] = high[i] = make_float2(0.0f, 0.0f);
-        // A warp's quarter of the terms: channels of the state, then tokens' values.
-        constexpr int TERMS = (DIM + CHUNK) / 4;
-#pragma unroll 4
+        // A warp's share of the terms: channels of the state, then tokens' values.
+        constexpr int TERMS = (DIM + CHUNK) / WALK_WARPS;
+#pragma unroll (TERMS % 5 == 0 ? 5 : 6)
         for (int n = 0; n < TERMS; ++n) {
             const int term = warp * TERMS + n;
             const float* reading = stage + term * ROWS + TALL * group;
@@ -314,17 +318,16 @@ __global__ void __launch_bounds__(THREADS) chunk_walk_kernel(ChunkArgs a) {
 #pragma unroll
         for (int i = 0; i < TALL; ++i)
             *reinterpret_cast<float4*>(partial + (warp * ROWS + TALL * group + i) * COLUMNS + 4 * strip) = make_float4(low[i].x, low[i].y, high[i].x, high[i].y);
-        __syncthreads();  // the quarters are there, and nobody reads the state any more
-#pragma unroll
-        for (int n = 0; n < ROWS / 16; ++n) {
-            const int row = n * 16 + threadIdx.x / 8, t = row - (ROWS - CHUNK);
+        __syncthreads();  // every warp's sums are there, and nobody reads the state any more
+        if (threadIdx.x / 8 < ROWS) {
+            const int row = threadIdx.x / 8, t = row - (ROWS - CHUNK);
             float4 z = *reinterpret_cast<const float4*>(partial + row * COLUMNS + 4 * strip);
 #pragma unroll
-            for (int part = 1; part < 4; ++part) {
+            for (int part = 1; part < WALK_WARPS; ++part) {
                 const float4 x = *reinterpret_cast<const float4*>(partial + (part * ROWS + row) * COLUMNS + 4 * strip);
                 z.x += x.x, z.y += x.y, z.z += x.z, z.w += x.w;
             }
-            if (REMOVES && n == 0) {
+            if (REMOVES && row < CHUNK) {
                 *reinterpret_cast<float4*>(minus_y + row * COLUMNS + 4 * strip) = make_float4(-z.x, -z.y, -z.z, -z.w);
             } else if (chunk * CHUNK + t < count && first_column + 4 * strip < a.vdim) {
                 float* out = a.out + (static_cast<size_t>(begin + chunk * CHUNK + t) * a.heads + head) * a.vdim + first_column + 4 * strip;
@@ -333,46 +336,56 @@ __global__ void __launch_bounds__(THREADS) chunk_walk_kernel(ChunkArgs a) {
         }
         if (REMOVES) __syncthreads();  // the reads y are there
         const float* writing = stage + (DIM + CHUNK) * ROWS;
+        // The owners add the first half of the written terms to their decayed tiles, the others add up the second half: the removals,
+        // or the last tokens' keys and values.
+        float2 first[TILES][4], second[TILES][4];
 #pragma unroll
         for (int tile = 0; tile < TILES; ++tile) {
-            const int d = 4 * (threadIdx.x / 8 + 16 * tile);
-            if (d >= DIM) continue;
+            const int d = min(4 * (quad + 16 * tile), DIM - 4);
             const float4 g = *reinterpret_cast<const float4*>(writing + ROWS * DIM + d);
-            float2 first[4], second[4];
             const float decay[4] = {g.x, g.y, g.z, g.w};
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
-                first[i] = make_float2(s[tile][i].x * decay[i], s[tile][i].y * decay[i]);
-                second[i] = make_float2(s[tile][i].z * decay[i], s[tile][i].w * decay[i]);
+                first[tile][i] = owner ? make_float2(s[tile][i].x * decay[i], s[tile][i].y * decay[i]) : make_float2(0.0f, 0.0f);
+                second[tile][i] = owner ? make_float2(s[tile][i].z * decay[i], s[tile][i].w * decay[i]) : make_float2(0.0f, 0.0f);
             }
-            auto add_outer = [&](const float* written, const float* operand) {
-                const float4 w = *reinterpret_cast<const float4*>(written + d), x = *reinterpret_cast<const float4*>(operand + 4 * strip);
+            const float* written = writing + (owner ? 0 : ROWS / 2 * DIM) + d;
+            const float* operand = (owner ? v : REMOVES ? minus_y : v + ROWS / 2 * COLUMNS) + 4 * strip;
+#pragma unroll 8
+            for (int n = 0; n < ROWS / 2; ++n) {
+                const float4 w = *reinterpret_cast<const float4*>(written + n * DIM), x = *reinterpret_cast<const float4*>(operand + n * COLUMNS);
                 const float weights[4] = {w.x, w.y, w.z, w.w};
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
-                    first[i] = __ffma2_rn(make_float2(weights[i], weights[i]), make_float2(x.x, x.y), first[i]);
-                    second[i] = __ffma2_rn(make_float2(weights[i], weights[i]), make_float2(x.z, x.w), second[i]);
+                    first[tile][i] = __ffma2_rn(make_float2(weights[i], weights[i]), make_float2(x.x, x.y), first[tile][i]);
+                    second[tile][i] = __ffma2_rn(make_float2(weights[i], weights[i]), make_float2(x.z, x.w), second[tile][i]);
                 }
-            };
-#pragma unroll 8
-            for (int t = 0; t < CHUNK; ++t) add_outer(writing + t * DIM, v + t * COLUMNS);
-            if constexpr (REMOVES) {
-#pragma unroll 8
-                for (int t = 0; t < CHUNK; ++t) add_outer(writing + (CHUNK + t) * DIM, minus_y + t * COLUMNS);
             }
+            if (!owner && 4 * (quad + 16 * tile) < DIM) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+                    *reinterpret_cast<float4*>(added + (d + i) * COLUMNS + 4 * strip) = make_float4(first[tile][i].x, first[tile][i].y, second[tile][i].x, second[tile][i].y);
+            }
+        }
+        __syncthreads();  // the second half is there
+#pragma unroll
+        for (int tile = 0; tile < TILES && owner; ++tile) {
+            const int d = 4 * (quad + 16 * tile);
+            if (d >= DIM) continue;
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
-                s[tile][i] = make_float4(first[i].x, first[i].y, second[i].x, second[i].y);
+                const float4 x = *reinterpret_cast<const float4*>(added + (d + i) * COLUMNS + 4 * strip);
+                s[tile][i] = make_float4(first[tile][i].x + x.x, first[tile][i].y + x.y, second[tile][i].x + x.z, second[tile][i].y + x.w);
                 *reinterpret_cast<float4*>(held + (d + i) * COLUMNS + 4 * strip) = s[tile][i];
             }
         }
     }
 #pragma unroll
     for (int tile = 0; tile < TILES; ++tile) {
-        const int d = 4 * (threadIdx.x / 8 + 16 * tile);
+        const int d = 4 * (quad + 16 * tile);
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
-            if (d < a.dim && first_column + 4 * strip + c < a.vdim)
+            if (owner && d < a.dim && first_column + 4 * strip + c < a.vdim)
                 *reinterpret_cast<float4*>(state + static_cast<size_t>(c) * a.dim + d) =
                     make_float4(columns_of(s[tile][0], c), columns_of(s[tile][1], c), columns_of(s[tile][2], c), columns_of(s[tile][3], c));
         }
@@ -395,14 +408,14 @@ template <int RULE, int DIM>
 static int launch_chunks(const ChunkArgs& a, int max_chunks, cudaStream_t stream) {
     static SharedMemoryOptIn record_opt_in, walk_opt_in;
     constexpr int RECORD_SMEM = (Rule<RULE>::VECTORS * CHUNK * DIM + 4 * CHUNK * CHUNK) * sizeof(float);
-    constexpr int WALK_SMEM = (STAGES * (Record<RULE, DIM>::FLOATS + CHUNK * COLUMNS) + DIM * COLUMNS + (CHUNK + 4 * Rule<RULE>::ROWS) * COLUMNS) * sizeof(float);
+    constexpr int WALK_SMEM = (STAGES * (Record<RULE, DIM>::FLOATS + CHUNK * COLUMNS) + 2 * DIM * COLUMNS + (CHUNK + WALK_WARPS * Rule<RULE>::ROWS) * COLUMNS) * sizeof(float);
     if (RECORD_SMEM > 48 * 1024)
         if (const int e = record_opt_in(chunk_record_kernel<RULE, DIM>, RECORD_SMEM)) return e;
     if (WALK_SMEM > 48 * 1024)
         if (const int e = walk_opt_in(chunk_walk_kernel<RULE, DIM>, WALK_SMEM)) return e;
     const int code = launch_kernel_in_order(chunk_record_kernel<RULE, DIM>, dim3(max_chunks, a.heads), THREADS, RECORD_SMEM, stream, a);
     if (code) return code;
-    return launch_kernel_in_order(chunk_walk_kernel<RULE, DIM>, dim3(a.entries, a.heads, (a.vdim + COLUMNS - 1) / COLUMNS), THREADS, WALK_SMEM, stream, a);
+    return launch_kernel_in_order(chunk_walk_kernel<RULE, DIM>, dim3(a.entries, a.heads, (a.vdim + COLUMNS - 1) / COLUMNS), WALK_THREADS, WALK_SMEM, stream, a);
 }
 
 template <int RULE>
