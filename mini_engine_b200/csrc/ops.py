@@ -1249,11 +1249,11 @@ def state_rule_floats(rule: str, dim: int, vdim: int) -> tuple[int, int]:
 STATE_CHUNK = 16  # tokens of a chunk of the chunked recurrences
 
 
-def state_chunks_support(dim: int, vdim: int) -> bool:
-    """Whether the chunked kernels take these head sizes."""
+def state_chunks_support(dim: int, vdim: int, slot_floats: int) -> bool:
+    """Whether the chunked kernels take these head sizes and slots that are ``slot_floats`` apart."""
     fn = load_library("state_chunks").me_state_chunks_supports
     fn.argtypes, fn.restype = [c_int, c_int], c_int
-    return bool(fn(int(dim), int(vdim)))
+    return bool(fn(int(dim), int(vdim))) and slot_floats % 4 == 0
 
 
 def state_record_floats(rule: str, dim: int) -> int:
@@ -1311,7 +1311,7 @@ def state_walk(
         raise KernelError("state_walk: the state does not hold the matrix states")
     if chunk_min:
         _need(records, torch.float32, "records")
-        if not state_chunks_support(dim, vdim) or records.dim() != 2 or records.shape[1] != heads * state_record_floats(rule, dim):
+        if not state_chunks_support(dim, vdim, state.shape[1]) or records.dim() != 2 or records.shape[1] != heads * state_record_floats(rule, dim):
             raise KernelError("state_walk: the chunks' records or the head sizes do not fit")
         fn = _fn("state_chunks", "me_state_chunks", [c_void_p] * 6 + [c_longlong, c_void_p, c_void_p] + [c_int] * 7 + [c_void_p])
         code = fn(

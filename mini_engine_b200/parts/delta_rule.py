@@ -259,7 +259,8 @@ def walk_states(rule: str, ctx: StepContext, state: torch.Tensor, heads: int, di
     ops.state_prepare(rule=rule, rows=rows, scalars=scalars, **{"rate": None, "unit_eps": 0.0, "decay_scale": 1.0, **inputs}, **sizes)
     raw = ctx.buffer(f"{rule}.raw", (tokens, heads * vdim), torch.float32)
     chunk_min, records = 0, None
-    if ctx.max_query_len >= CHUNKED_MIN_TOKENS and ops.state_chunks_support(dim, vdim):  # a step's longest entry is known on the host
+    # a step's longest entry is known on the host
+    if ctx.max_query_len >= CHUNKED_MIN_TOKENS and ops.state_chunks_support(dim, vdim, state.shape[1]):
         chunk_min = CHUNKED_MIN_TOKENS
         chunks = tokens // ops.STATE_CHUNK + ctx.num_entries
         records = ctx.workspace.growing(f"{rule}.records", (chunks, heads * ops.state_record_floats(rule, dim)), torch.float32)

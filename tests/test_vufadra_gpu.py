@@ -368,6 +368,17 @@ def test_a_model_of_one_mixer(kind, tmp_path):
             replay_and_compare(folder, dtype_name, maker(requests), requests)
 
 
+def test_states_in_slots_of_an_odd_length(tmp_path):
+    """Time mixing keeps its last input behind its matrix states: with a width of 54 the slots of heads that the chunks would
+    take start on no 16 bytes, and long portions walk token by token."""
+    raw = model(80, 54, 0.1, [both(attention(2, 1, 32, 32, 50, 0.2, 3000.0, 16), states(2, 32, 6), 40), delta(2, 32, 6, None)], bigram=(40, 9, 4))
+    folder = write_model(tmp_path, raw, seed=8)
+    requests = {"a": random_ids(3, 160, 80), "b": random_ids(4, 47, 80), "c": random_ids(5, 1, 80)}
+    for dtype_name in ("float32", "bfloat16"):
+        for maker in (schedules.whole, schedules.changing_portions, schedules.mixed):
+            replay_and_compare(folder, dtype_name, maker(requests), requests)
+
+
 def test_the_block_with_another_norm(monkeypatch):
     """The arrangement with layer norms in the place of dynamic tanh: three kernels in the place of one, the same layer."""
     from mini_engine_b200.cache.manager import CacheManager
